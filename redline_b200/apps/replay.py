@@ -7,7 +7,7 @@ from typing import Any, Dict, List, Optional, Sequence
 
 import numpy as np
 
-MAX_LIVE_REQUESTS = 8          # the trace format allows up to four live requests
+MAX_LIVE_REQUESTS = 4          # the most requests a trace may hold live at any time
 MAX_STEP_TOKENS = 8192         # larger steps are run as several batches
 MAX_LOGITS_BYTES = 1 << 30
 

@@ -1014,3 +1014,244 @@ class VenezenConfig(ModelConfig):
         if self.eos_token_ids:
             out["eos_token_id"] = list(self.eos_token_ids)
         return out
+
+
+# ------------------------------------------------------------------------------------------------ Lakatar
+
+@dataclass(frozen=True)
+class LakatarScaling:
+    """YaRN scaling of a rotation's frequencies."""
+
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
+class LakatarRotation:
+    base: float
+    dims: int
+    scaling: Optional[LakatarScaling] = None
+
+
+@dataclass(frozen=True)
+class LakatarTimeMix:
+    """A 'wkv' mixer.  The inner size of the decays' two products is not in config.json: it is the checkpoint's tensor
+    shape (``decay_rank`` may be given for a model without a file)."""
+
+    heads: int
+    dim: int
+    decay_rank: int
+
+
+@dataclass(frozen=True)
+class LakatarRetention:
+    heads: int
+    dim: int
+    vdim: int
+    decay: Tuple[float, ...]       # one per head
+    rot: Optional[LakatarRotation]     # entry i of the first ``dims`` turns with entry i + dims / 2
+
+
+@dataclass(frozen=True)
+class LakatarLatent:
+    """A 'latent_attention' mixer; with ``kv_from`` it attends over the rows that layer has cached."""
+
+    heads: int
+    dim: int                  # unrotated entries of a head's query and key
+    rot_dim: int              # rotated entries (the key's are one vector for all heads), neighbours turn together
+    vdim: int
+    kv_rank: int              # size of the cached latent
+    q_rank: int               # size of the latent the queries come from
+    scale: float
+    rot: Optional[LakatarRotation]
+    kv_from: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class LakatarMLP:
+    """Routed experts with a shared one."""
+
+    ff: int                   # of one expert
+    experts: int
+    top: int
+    groups: int = 1
+    group_keep: int = 1
+    scale: float = 1.0        # factor on the chosen experts' weights
+    shared_ff: int = 0        # 0: no shared expert
+
+
+@dataclass(frozen=True)
+class LakatarLayer:
+    type: str                 # wkv | retention | latent_attention
+    mixer: Any
+    mlp: Optional[LakatarMLP]
+
+
+@dataclass(frozen=True)
+class LakatarConfig(ModelConfig):
+    """``Lakatar``: layers that norm the stream after every sum, x = norm(alpha x + s * sublayer(x)) with a vector s
+    per sublayer.  Mixers: RWKV-style time mixing, retention with rotated queries and keys, attention over a cached
+    latent whose queries come from a latent of their own (a layer may share an earlier one's cache).
+    Feed-forwards: routed experts chosen within the best groups, with a gated shared expert.  The head has a matrix
+    of its own.  config.json lists the layers under ``layers``."""
+
+    norm_eps: float = 1e-6
+    alpha: float = 1.0
+    layers: Tuple[LakatarLayer, ...] = ()
+
+    @staticmethod
+    def _rotation(rot: Optional[Dict[str, Any]], where: str) -> Optional[LakatarRotation]:
+        if not rot:
+            return None
+        sc = rot.get("scaling")
+        w = where + ".scaling"
+        return LakatarRotation(
+            float(_need(rot, "base", where)), int(_need(rot, "dims", where)),
+            LakatarScaling(float(_need(sc, "factor", w)), float(_need(sc, "original", w)), float(_need(sc, "fast", w)),
+                           float(_need(sc, "slow", w))) if sc else None)
+
+    @classmethod
+    def from_hf(cls, cfg: Dict[str, Any], model_dir: Optional[str] = None) -> "LakatarConfig":
+        shapes = _safetensors_shapes(model_dir)
+        layers: List[LakatarLayer] = []
+        for i, entry in enumerate(_need(cfg, "layers")):
+            where = f"layers[{i}]"
+            kind = _need(entry, "type", where)
+            m = _need(entry, "mixer", where)
+            mw = where + ".mixer"
+            heads = int(_need(m, "heads", mw))
+            dim = int(_need(m, "dim", mw))
+            if kind == "wkv":
+                name = f"l{i}.mix.w1"
+                if name in shapes:
+                    rank = int(shapes[name][0])
+                elif m.get("decay_rank") is not None:
+                    rank = int(m["decay_rank"])
+                else:
+                    raise ConfigError(f"{mw}: the inner size of the decay's products is neither a tensor shape of the "
+                                      f"checkpoint nor given as 'decay_rank'")
+                mixer: Any = LakatarTimeMix(heads, dim, rank)
+            elif kind == "retention":
+                mixer = LakatarRetention(heads, dim, int(_need(m, "vdim", mw)),
+                                         tuple(float(d) for d in _need(m, "decay", mw)), cls._rotation(m.get("rot"), mw + ".rot"))
+            elif kind == "latent_attention":
+                src = m.get("kv_from")
+                mixer = LakatarLatent(
+                    heads=heads, dim=dim, rot_dim=int(_need(m, "rot_dim", mw)), vdim=int(_need(m, "vdim", mw)),
+                    kv_rank=int(_need(m, "kv_rank", mw)), q_rank=int(_need(m, "q_rank", mw)), scale=float(_need(m, "scale", mw)),
+                    rot=cls._rotation(m.get("rot"), mw + ".rot"), kv_from=int(src) if src is not None else None)
+            else:
+                raise ConfigError(f"{where}: mixer type '{kind}' is not supported (wkv, retention, latent_attention)")
+            mlp = entry.get("mlp")
+            ff: Optional[LakatarMLP] = None
+            if mlp is not None:
+                fw = where + ".mlp"
+                if _need(mlp, "kind", fw) != "moe":
+                    raise ConfigError(f"{fw}: kind '{mlp['kind']}' is not supported (moe)")
+                r = _need(mlp, "router", fw)
+                groups = r.get("groups") or {"count": 1, "keep": 1}
+                sh = mlp.get("shared")
+                ff = LakatarMLP(
+                    ff=int(_need(_need(mlp, "expert", fw), "ff", fw + ".expert")), experts=int(_need(r, "experts", fw + ".router")),
+                    top=int(_need(r, "top", fw + ".router")), groups=int(_need(groups, "count", fw + ".router.groups")),
+                    group_keep=int(_need(groups, "keep", fw + ".router.groups")), scale=float(r.get("scale", 1.0)),
+                    shared_ff=int(_need(sh, "ff", fw + ".shared")) if sh else 0)
+            layers.append(LakatarLayer(kind, mixer, ff))
+        eos = cfg.get("eos_token_id")
+        eos = [] if eos is None else ([eos] if isinstance(eos, int) else list(eos))
+        bos = cfg.get("bos_token_id")
+        c = cls(architecture="Lakatar", vocab_size=int(_need(cfg, "vocab")), hidden_size=int(_need(cfg, "width")),
+                max_position_embeddings=int(cfg.get("max_positions", 1 << 30)),
+                bos_token_id=int(bos) if bos is not None else -1, eos_token_ids=tuple(int(e) for e in eos),
+                norm_eps=float(_need(_need(cfg, "norm"), "eps", "norm")), alpha=float(_need(cfg, "postln_alpha")),
+                layers=tuple(layers))
+        c.validate()
+        return c
+
+    def validate(self) -> None:
+        if self.vocab_size <= 0 or self.hidden_size <= 0 or not self.layers:
+            raise ConfigError("vocab, width and the number of layers must be positive")
+        if not self.norm_eps > 0:
+            raise ConfigError(f"norm.eps must be positive, got {self.norm_eps}")
+        for i, layer in enumerate(self.layers):
+            m = layer.mixer
+            mw = f"layers[{i}].mixer"
+            if m.heads <= 0 or m.dim <= 0:
+                raise ConfigError(f"{mw}: heads and dim must be positive")
+            rot = getattr(m, "rot", None)
+            if rot is not None:
+                if rot.dims <= 0 or rot.dims % 2 != 0 or not rot.base > 0:
+                    raise ConfigError(f"{mw}: rot.dims must be even and positive, rot.base positive")
+                if rot.dims > (m.rot_dim if layer.type == "latent_attention" else m.dim):
+                    raise ConfigError(f"{mw}: rot.dims must be at most the size of what is rotated")
+                s = rot.scaling
+                if s is not None and not (s.factor > 0 and s.original > 0 and s.fast > 0 and s.slow > 0 and rot.base > 1):
+                    raise ConfigError(f"{mw}: rot.scaling needs positive factor, original, fast and slow")
+            if layer.type == "wkv":
+                if m.decay_rank <= 0:
+                    raise ConfigError(f"{mw}: the inner size of the decay's products must be positive")
+            elif layer.type == "retention":
+                if m.vdim <= 0 or len(m.decay) != m.heads:
+                    raise ConfigError(f"{mw}: vdim must be positive, decay list one number per head")
+            else:
+                if min(m.vdim, m.kv_rank, m.q_rank) <= 0 or m.rot_dim < 0:
+                    raise ConfigError(f"{mw}: vdim, kv_rank and q_rank must be positive")
+                if m.rot_dim > 0 and rot is None:
+                    raise ConfigError(f"{mw} has no 'rot'")
+                if m.kv_from is not None:
+                    src = self.layers[m.kv_from] if 0 <= m.kv_from < i else None
+                    if src is None or src.type != "latent_attention" or src.mixer.kv_from is not None:
+                        raise ConfigError(f"{mw}: kv_from must name an earlier latent_attention layer with a latent of its own")
+                    if (src.mixer.kv_rank, src.mixer.rot_dim, src.mixer.rot) != (m.kv_rank, m.rot_dim, m.rot):
+                        raise ConfigError(f"{mw}: kv_rank, rot_dim and rot must equal those of layer {m.kv_from}")
+            f = layer.mlp
+            fw = f"layers[{i}].mlp"
+            if f is None:
+                continue
+            if f.ff <= 0 or f.shared_ff < 0 or f.experts <= 0:
+                raise ConfigError(f"{fw}: ff and experts must be positive")
+            if f.groups <= 0 or f.experts % f.groups != 0 or not 1 <= f.group_keep <= f.groups:
+                raise ConfigError(f"{fw}: the experts must form groups.count equal groups of which groups.keep stay")
+            if not 1 <= f.top <= f.group_keep * (f.experts // f.groups):
+                raise ConfigError(f"{fw}: top must lie between 1 and the experts of the kept groups")
+
+    def to_hf(self) -> Dict[str, Any]:
+        def rotation(r: Optional[LakatarRotation]) -> Dict[str, Any]:
+            if r is None:
+                return {}
+            out: Dict[str, Any] = {"base": r.base, "dims": r.dims}
+            if r.scaling is not None:
+                s = r.scaling
+                out["scaling"] = {"factor": s.factor, "original": s.original, "fast": s.fast, "slow": s.slow}
+            return {"rot": out}
+
+        layers = []
+        for layer in self.layers:
+            m = layer.mixer
+            if layer.type == "wkv":
+                mixer: Dict[str, Any] = {"heads": m.heads, "dim": m.dim, "decay_rank": m.decay_rank}
+            elif layer.type == "retention":
+                mixer = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "decay": list(m.decay), **rotation(m.rot)}
+            else:
+                mixer = {"heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank,
+                         "q_rank": m.q_rank, "scale": m.scale, **rotation(m.rot)}
+                if m.kv_from is not None:
+                    mixer["kv_from"] = m.kv_from
+            f = layer.mlp
+            mlp = None
+            if f is not None:
+                mlp = {"kind": "moe", "expert": {"ff": f.ff},
+                       "router": {"experts": f.experts, "top": f.top, "scale": f.scale,
+                                  "groups": {"count": f.groups, "keep": f.group_keep}}}
+                if f.shared_ff > 0:
+                    mlp["shared"] = {"ff": f.shared_ff}
+            layers.append({"type": layer.type, "mixer": mixer, "mlp": mlp})
+        out: Dict[str, Any] = {"architecture": "Lakatar", "vocab": self.vocab_size, "width": self.hidden_size,
+                               "norm": {"eps": self.norm_eps}, "postln_alpha": self.alpha, "layers": layers}
+        if self.bos_token_id >= 0:
+            out["bos_token_id"] = self.bos_token_id
+        if self.eos_token_ids:
+            out["eos_token_id"] = list(self.eos_token_ids)
+        return out

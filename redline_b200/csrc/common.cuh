@@ -47,6 +47,19 @@ __device__ __forceinline__ void store16(bf16* p, const float* in) {
   *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
 }
 
+// Four neighbouring elements as one access (a 16-byte piece of floats, an 8-byte piece of bfloat16).
+__device__ __forceinline__ void load4(const float* p, float* out) { load16(p, out); }
+__device__ __forceinline__ void load4(const bf16* p, float* out) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  out[0] = __uint_as_float(v.x << 16); out[1] = __uint_as_float(v.x & 0xFFFF0000u);
+  out[2] = __uint_as_float(v.y << 16); out[3] = __uint_as_float(v.y & 0xFFFF0000u);
+}
+__device__ __forceinline__ void store4(float* p, const float* in) { store16(p, in); }
+__device__ __forceinline__ void store4(bf16* p, const float* in) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(in[0], in[1]), b = __floats2bfloat162_rn(in[2], in[3]);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
 __device__ __forceinline__ float to_float(float x) { return x; }
 __device__ __forceinline__ float to_float(bf16 x) { return __bfloat162float(x); }
 template <typename T>

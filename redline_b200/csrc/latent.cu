@@ -8,9 +8,13 @@
 // attention runs over the cached rows [c | k_r] themselves, one key head for all query heads, with the query
 // [W_uk,h^T q_n | q_r] and the row's first `rank` entries as the value; W_uv,h is applied to its result.
 //
+// The queries may come from a latent of their own (RMS-normed, then a product), and a layer may attend over
+// the rows another layer has cached; the three jobs of latent_prep can then be asked for one by one.
+//
 //   latent_prep   per token: c (RMS norm in float32, weight w), k_r and every head's q_r turned by the
-//                 token's position (entry i with entry i + dims/2 of the first `dims` rotated entries, cos
-//                 and sin from tables), [c | k_r] into the paged cache, q_r into the attention's query rows
+//                 token's position (entry i with entry i + dims/2 of the first `dims` rotated entries, or
+//                 neighbours, cos and sin from tables), [c | k_r] into the paged cache, q_r into the
+//                 attention's query rows; the norm of the queries' latent
 //   head_linear   y[t, h, :] = W_h x[t, h, :] for every head h, W [heads, n, k], float32 sums in ascending k
 //                 (a row's result does not depend on what else is in the launch); FFMA for float32, and
 //                 mma.sync.m16n8k16 for bfloat16 operands whose sizes allow it
@@ -19,29 +23,45 @@
 namespace rl {
 
 struct LatentPrepArgs {
-  int ld;            // row length of the projection buffer
+  int q_src_ld;      // row length of the buffer the queries lie in
+  int c_ld;          // row length of the buffer the raw latent lies in
   int heads, dn, dr, rank, rot_dims;
   int q_ld;          // row length of the attention's query buffer: heads * (rank + dr)
   float eps;
   int page_size;
   long long num_slots;
   int max_pos;       // rows of the tables
+  int pairs;         // rotated entries 2i and 2i + 1 turn together (else i and i + rot_dims / 2)
+  int dq_ld, dq_rank, dq_out_ld;     // a latent of the queries, normed for the product behind it
 };
 
-// One CTA per token.  A position beyond the tables sets bit 1 of *status, a slot beyond the pool bit 2
-// (negative slot: no write).
+// Entry d of a rotated part, turned.
+template <typename TA>
+__device__ __forceinline__ float rotated(const TA* __restrict__ src, int d, int rot_dims, int pairs,
+                                         const float* __restrict__ cs, const float* __restrict__ sn) {
+  const float v = to_float(src[d]);
+  if (d >= rot_dims) return v;
+  const int half = rot_dims / 2;
+  const bool first = pairs ? (d & 1) == 0 : d < half;
+  const int i = pairs ? d >> 1 : (first ? d : d - half), gap = pairs ? 1 : half;
+  return first ? v * cs[i] - to_float(src[d + gap]) * sn[i] : v * cs[i] + to_float(src[d - gap]) * sn[i];
+}
+
+// One CTA per token; each of the three jobs is done where its buffers are given: the heads' rotated query
+// parts (q), the norm of the queries' latent (dq), the latent and the shared key part into the cache (craw and
+// slots).  A position beyond the tables sets bit 1 of *status, a slot beyond the pool bit 2 (negative slot: no
+// write).
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(128)
-latent_prep_kernel(const TA* __restrict__ proj, const int32_t* __restrict__ positions, const TW* __restrict__ w,
-                   const float* __restrict__ cos_t, const float* __restrict__ sin_t, TA* __restrict__ qa,
-                   const int32_t* __restrict__ slots, TA* __restrict__ cache, int* status, const LatentPrepArgs a) {
+latent_prep_kernel(const TA* __restrict__ q, const TA* __restrict__ craw, const int32_t* __restrict__ positions,
+                   const TW* __restrict__ w, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                   TA* __restrict__ qa, const int32_t* __restrict__ slots, TA* __restrict__ cache,
+                   const TA* __restrict__ dq, const TW* __restrict__ dq_w, TA* __restrict__ dq_out, int* status,
+                   const LatentPrepArgs a) {
   pdl_launch();
   pdl_wait();
   __shared__ float scratch[32];
   const int t = blockIdx.x;
-  const int qsize = a.heads * (a.dn + a.dr);
-  const TA* row = proj + static_cast<size_t>(t) * a.ld;
-  const TA* craw = row + qsize;
   const int half = a.rot_dims / 2;
   int pos = positions[t];
   if (a.dr > 0 && (pos < 0 || pos >= a.max_pos)) {
@@ -50,38 +70,47 @@ latent_prep_kernel(const TA* __restrict__ proj, const int32_t* __restrict__ posi
   }
   const float* cs = cos_t + static_cast<size_t>(pos) * half;
   const float* sn = sin_t + static_cast<size_t>(pos) * half;
-  // ---- the heads' rotated query parts
-  TA* qrow = qa + static_cast<size_t>(t) * a.q_ld;
-  for (int i = threadIdx.x; i < a.heads * a.dr; i += blockDim.x) {
-    const int h = i / a.dr, d = i - h * a.dr;
-    const TA* src = row + h * (a.dn + a.dr) + a.dn;
-    float v = to_float(src[d]);
-    if (d < half) v = v * cs[d] - to_float(src[d + half]) * sn[d];
-    else if (d < a.rot_dims) v = v * cs[d - half] + to_float(src[d - half]) * sn[d - half];
-    qrow[h * (a.rank + a.dr) + a.rank + d] = from_float<TA>(v);
+  if (q != nullptr) {
+    // ---- the heads' rotated query parts
+    const TA* row = q + static_cast<size_t>(t) * a.q_src_ld;
+    TA* qrow = qa + static_cast<size_t>(t) * a.q_ld;
+    for (int i = threadIdx.x; i < a.heads * a.dr; i += blockDim.x) {
+      const int h = i / a.dr, d = i - h * a.dr;
+      qrow[h * (a.rank + a.dr) + a.rank + d] =
+          from_float<TA>(rotated(row + h * (a.dn + a.dr) + a.dn, d, a.rot_dims, a.pairs, cs, sn));
+    }
   }
+  if (dq != nullptr) {
+    // ---- the queries' latent, normed
+    const TA* src = dq + static_cast<size_t>(t) * a.dq_ld;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < a.dq_rank; i += blockDim.x) {
+      const float v = to_float(src[i]);
+      ss += v * v;
+    }
+    const float r = rsqrtf(block_sum(ss, scratch) / static_cast<float>(a.dq_rank) + a.eps);
+    TA* dst = dq_out + static_cast<size_t>(t) * a.dq_out_ld;
+    for (int i = threadIdx.x; i < a.dq_rank; i += blockDim.x) dst[i] = from_float<TA>(to_float(src[i]) * r * to_float(dq_w[i]));
+  }
+  if (craw == nullptr || slots == nullptr) return;
   // ---- the latent and the shared key part into the cache
-  float q = 0.f;
+  const TA* c = craw + static_cast<size_t>(t) * a.c_ld;
+  float ss = 0.f;
   for (int i = threadIdx.x; i < a.rank; i += blockDim.x) {
-    const float v = to_float(craw[i]);
-    q += v * v;
+    const float v = to_float(c[i]);
+    ss += v * v;
   }
-  const float r = rsqrtf(block_sum(q, scratch) / static_cast<float>(a.rank) + a.eps);
-  const int slot = slots != nullptr ? slots[t] : -1;
+  const float r = rsqrtf(block_sum(ss, scratch) / static_cast<float>(a.rank) + a.eps);
+  const int slot = slots[t];
   if (slot < 0) return;
   if (slot >= a.num_slots) {
     if (threadIdx.x == 0) atomicOr(status, 4);
     return;
   }
   TA* dst = cache + static_cast<size_t>(slot) * (a.rank + a.dr);     // one key head: [pages, 1, page, rank + dr]
-  for (int i = threadIdx.x; i < a.rank; i += blockDim.x) dst[i] = from_float<TA>(to_float(craw[i]) * r * to_float(w[i]));
-  for (int d = threadIdx.x; d < a.dr; d += blockDim.x) {
-    const TA* src = craw + a.rank;
-    float v = to_float(src[d]);
-    if (d < half) v = v * cs[d] - to_float(src[d + half]) * sn[d];
-    else if (d < a.rot_dims) v = v * cs[d - half] + to_float(src[d - half]) * sn[d - half];
-    dst[a.rank + d] = from_float<TA>(v);
-  }
+  for (int i = threadIdx.x; i < a.rank; i += blockDim.x) dst[i] = from_float<TA>(to_float(c[i]) * r * to_float(w[i]));
+  for (int d = threadIdx.x; d < a.dr; d += blockDim.x)
+    dst[a.rank + d] = from_float<TA>(rotated(c + a.rank, d, a.rot_dims, a.pairs, cs, sn));
 }
 
 // ------------------------------------------------------------------ per-head products
@@ -199,13 +228,15 @@ using namespace rl;
 
 extern "C" {
 
-int rl_latent_prep(int act_dtype, int w_dtype, const void* proj, int ld, const int32_t* positions, int tokens, int heads,
-                   int dn, int dr, int rank, int rot_dims, const void* w, float eps, const float* cos_t,
-                   const float* sin_t, int max_pos, void* qa, int q_ld, const int32_t* slots, void* cache, int page_size,
-                   long long num_slots, int* status, cudaStream_t stream) {
+int rl_latent_prep(int act_dtype, int w_dtype, const void* q, int q_src_ld, const void* craw, int c_ld,
+                   const int32_t* positions, int tokens, int heads, int dn, int dr, int rank, int rot_dims, int pairs,
+                   const void* w, float eps, const float* cos_t, const float* sin_t, int max_pos, void* qa, int q_ld,
+                   const int32_t* slots, void* cache, int page_size, long long num_slots, const void* dq, int dq_ld,
+                   int dq_rank, const void* dq_w, void* dq_out, int dq_out_ld, int* status, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   LatentPrepArgs a;
-  a.ld = ld;
+  a.q_src_ld = q_src_ld;
+  a.c_ld = c_ld;
   a.heads = heads;
   a.dn = dn;
   a.dr = dr;
@@ -216,10 +247,15 @@ int rl_latent_prep(int act_dtype, int w_dtype, const void* proj, int ld, const i
   a.page_size = page_size;
   a.num_slots = num_slots;
   a.max_pos = max_pos;
-#define RL_CASE(TA, TW)                                                                                          \
-  launch_kernel(latent_prep_kernel<TA, TW>, dim3(tokens), dim3(128), 0, stream, static_cast<const TA*>(proj),    \
-                positions, static_cast<const TW*>(w), cos_t, sin_t, static_cast<TA*>(qa), slots,                  \
-                static_cast<TA*>(cache), status, a)
+  a.pairs = pairs;
+  a.dq_ld = dq_ld;
+  a.dq_rank = dq_rank;
+  a.dq_out_ld = dq_out_ld;
+#define RL_CASE(TA, TW)                                                                                            \
+  launch_kernel(latent_prep_kernel<TA, TW>, dim3(tokens), dim3(128), 0, stream, static_cast<const TA*>(q),         \
+                static_cast<const TA*>(craw), positions, static_cast<const TW*>(w), cos_t, sin_t,                  \
+                static_cast<TA*>(qa), slots, static_cast<TA*>(cache), static_cast<const TA*>(dq),                  \
+                static_cast<const TW*>(dq_w), static_cast<TA*>(dq_out), status, a)
   if (act_dtype == 0) RL_CASE(float, float);
   else if (w_dtype == 0) RL_CASE(bf16, float);
   else RL_CASE(bf16, bf16);

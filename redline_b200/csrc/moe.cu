@@ -3,7 +3,7 @@
 //
 //   router:   z = W_r x (float32 sums; in this kernel, or handed in as float32 logits), score = sigmoid(z) (or softmax over the experts); experts lie in
 //             `groups` equal groups of neighbours; a group's score is the sum of its `group_top` best
-//             scores; only experts of the best `keep` groups can be chosen; the `top` best of those are
+//             choice scores; only experts of the best `keep` groups can be chosen; the `top` best of those are
 //             the token's experts, weighted by their scores (optionally divided by their sum);
 //             a choice bias per expert may be added to the scores for the choice alone (the weights are the
 //             scores without it); the weights may be multiplied by a constant
@@ -13,7 +13,8 @@
 //             `tile_begin` / `tile_rows` cut every expert's pairs into tiles of up to 64 rows
 //   products: up:   act[p, :]  = f(W_up[e]   x[token(p), :])      f = activation
 //             down: y[p, :]    =   W_down[e] act[p, :]
-//   combine:  out[t, :] = sum_k weight[t, k] * y[t * top + k, :] (+ shared[t, :]), k in order
+//   combine:  out[t, :] = sum_k weight[t, k] * y[t * top + k, :] (+ shared[t, :], times sigmoid(gate_t) where
+//             the shared expert has a gate), k in order
 //
 // A pair's results do not depend on which other pairs share its tile or on the order within the
 // expert's list: every output element is one thread's sum over k in a fixed order.  All sums are float32.
@@ -105,7 +106,7 @@ __global__ void moe_route_kernel(const TA* __restrict__ x, int ld, const TW* __r
   __syncwarp();
   const int per = experts / groups;
   if (groups > 1 && keep < groups) {
-    // a group's score: the sum of its group_top best scores
+    // a group's score: the sum of its group_top best choice scores
     for (int g = lane; g < groups; g += 32) {
       float total = 0.f;
       int taken_a = -1;                    // (group_top is small: the best, then the best of the rest, ...)
@@ -114,7 +115,7 @@ __global__ void moe_route_kernel(const TA* __restrict__ x, int ld, const TW* __r
         float best = -INFINITY;
         int bi = -1;
         for (int e = 0; e < per; ++e) {
-          const float v = score[g * per + e];
+          const float v = work[g * per + e];
           // next in the order (value descending, index ascending) after (last, taken_a)
           const bool after = v < last || (v == last && e > taken_a);
           if (after && (v > best || bi < 0)) {
@@ -494,10 +495,11 @@ template <typename TA>
 __global__ void moe_combine_kernel(const TA* __restrict__ y, const float* __restrict__ weight,
                                    const TA* __restrict__ shared, TA* __restrict__ out, int width, int top,
                                    const int32_t* __restrict__ choice, int real_experts, const TA* __restrict__ x,
-                                   int ld_x) {
+                                   int ld_x, const float* __restrict__ shared_gate, int ld_gate) {
   pdl_launch();
   pdl_wait();
   const int t = blockIdx.y;
+  const float sg = shared_gate != nullptr ? 1.f / (1.f + expf(-shared_gate[static_cast<size_t>(t) * ld_gate])) : 1.f;
   for (int c = blockIdx.x * blockDim.x + threadIdx.x; c < width; c += gridDim.x * blockDim.x) {
     float s = 0.f;
     for (int k = 0; k < top; ++k) {
@@ -506,7 +508,7 @@ __global__ void moe_combine_kernel(const TA* __restrict__ y, const float* __rest
       const bool same = choice != nullptr && choice[pair] >= real_experts;
       s = fmaf(weight[pair], same ? to_float(x[static_cast<size_t>(t) * ld_x + c]) : to_float(y[pair * width + c]), s);
     }
-    if (shared != nullptr) s += to_float(shared[static_cast<size_t>(t) * width + c]);
+    if (shared != nullptr) s = fmaf(sg, to_float(shared[static_cast<size_t>(t) * width + c]), s);
     out[static_cast<size_t>(t) * width + c] = from_float<TA>(s);
   }
 }
@@ -586,17 +588,17 @@ int rl_moe_gemm(int act_dtype, const void* src, int ld_src, int src_div, const v
 
 int rl_moe_combine(int act_dtype, const void* y, const float* weight, const void* shared, void* out, int tokens,
                    int width, int top, const int32_t* choice, int real_experts, const void* x, int ld_x,
-                   cudaStream_t stream) {
+                   const float* shared_gate, int ld_gate, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   dim3 grid(min((width + 255) / 256, 32), tokens);
   if (act_dtype == 0)
     launch_kernel(moe_combine_kernel<float>, grid, dim3(256), 0, stream, static_cast<const float*>(y), weight,
                   static_cast<const float*>(shared), static_cast<float*>(out), width, top, choice, real_experts,
-                  static_cast<const float*>(x), ld_x);
+                  static_cast<const float*>(x), ld_x, shared_gate, ld_gate);
   else
     launch_kernel(moe_combine_kernel<bf16>, grid, dim3(256), 0, stream, static_cast<const bf16*>(y), weight,
                   static_cast<const bf16*>(shared), static_cast<bf16*>(out), width, top, choice, real_experts,
-                  static_cast<const bf16*>(x), ld_x);
+                  static_cast<const bf16*>(x), ld_x, shared_gate, ld_gate);
   RL_LAUNCH_END();
 }
 

@@ -1,5 +1,6 @@
 // Row-wise kernels for blocks that norm a sublayer's input AND its output: layer norm (weight, no
-// bias) fused with the add to the float32 residual stream and with the norm that follows; bias +
+// bias) fused with the add to the float32 residual stream and with the norm that follows; the norm of the
+// weighted sum of stream and output, for blocks that norm after the sum; bias +
 // activation over a range of columns; the write of any per-token tensor into its paged cache; the
 // gated unit-RMS norm that closes a linear-attention mixer; a gated activation act(gate) * up; and what
 // attention heads may need between their projection and the cache: an RMS norm of queries and keys
@@ -14,7 +15,7 @@
 namespace rl {
 
 enum { ACT_NONE = 0, ACT_RELU_SQ = 1, ACT_GELU_ERF = 2, ACT_SILU = 3, ACT_GELU_TANH = 4, ACT_SIGMOID = 5,
-       ACT_CLAMPED_SWISH = 6 };
+       ACT_CLAMPED_SWISH = 6, ACT_TANH = 7 };
 
 __device__ __forceinline__ float activate(float z, int mode) {
   switch (mode) {
@@ -23,6 +24,7 @@ __device__ __forceinline__ float activate(float z, int mode) {
     case ACT_SILU: return z / (1.f + expf(-z));
     case ACT_GELU_TANH: return 0.5f * z * (1.f + tanhf(0.79788456080286536f * (z + 0.044715f * z * z * z)));
     case ACT_SIGMOID: return 1.f / (1.f + expf(-z));
+    case ACT_TANH: return tanhf(z);
     default: return z;
   }
 }
@@ -178,6 +180,97 @@ __global__ void sandwich_norm_reg_kernel(float* __restrict__ residual, const TA*
   }
 }
 
+// ------------------------------------------------ residual = RMS(alpha * residual + scale * delta) * w
+// The norm after the sum: the stream itself is what comes out of the norm, and with `out` also goes there in
+// the activation type for a sublayer that reads it.  One CTA per row.  delta null: nothing is summed or
+// normed, out is the stream row as it is.  w float32 [hidden]; scale float32 [hidden] or null (ones).
+// The row lives in registers, NV pieces of four neighbouring elements per thread (VEC: rows start on 16-byte
+// boundaries and hidden is a multiple of 4; else the elements are handled one by one).
+template <typename TA, int NV, bool VEC>
+__global__ void sum_norm_kernel(float* __restrict__ residual, const TA* __restrict__ delta, int ld_delta,
+                                const float* __restrict__ w, const float* __restrict__ scale, float alpha, float eps,
+                                TA* __restrict__ out, int ld_out, int hidden) {
+  __shared__ float scratch[32];
+  const int r = blockIdx.x;
+  float* res = residual + static_cast<size_t>(r) * hidden;
+  const TA* d = delta != nullptr ? delta + static_cast<size_t>(r) * ld_delta : nullptr;
+  // (weights come from no earlier kernel of the step: asked for before the wait)
+  float wv[NV][4], sv[NV][4], v[NV][4];
+  auto piece = [&](int i) { return (threadIdx.x + i * blockDim.x) * 4; };
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = piece(i);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { wv[i][j] = 0.f; sv[i][j] = 1.f; v[i][j] = 0.f; }
+    if (d == nullptr) continue;
+    if (VEC) {
+      if (c < hidden) {
+        load4(w + c, wv[i]);
+        if (scale != nullptr) load4(scale + c, sv[i]);
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < hidden) {
+          wv[i][j] = w[c + j];
+          if (scale != nullptr) sv[i][j] = scale[c + j];
+        }
+    }
+  }
+  pdl_launch();
+  pdl_wait();
+  float q = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = piece(i);
+    float dv[4] = {0.f, 0.f, 0.f, 0.f};
+    if (VEC) {
+      if (c < hidden) {
+        load4(res + c, v[i]);
+        if (d != nullptr) load4(d + c, dv);
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < hidden) {
+          v[i][j] = res[c + j];
+          if (d != nullptr) dv[j] = to_float(d[c + j]);
+        }
+    }
+    if (d != nullptr) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        v[i][j] = fmaf(sv[i][j], dv[j], alpha * v[i][j]);
+        q = fmaf(v[i][j], v[i][j], q);
+      }
+    }
+  }
+  if (d != nullptr) {
+    const float rstd = rsqrtf(block_sum(q, scratch) / static_cast<float>(hidden) + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[i][j] = v[i][j] * rstd * wv[i][j];
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = piece(i);
+    if (VEC) {
+      if (c < hidden) {
+        if (d != nullptr) store4(res + c, v[i]);
+        if (out != nullptr) store4(out + static_cast<size_t>(r) * ld_out + c, v[i]);
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < hidden) {
+          if (d != nullptr) res[c + j] = v[i][j];
+          if (out != nullptr) out[static_cast<size_t>(r) * ld_out + c + j] = from_float<TA>(v[i][j]);
+        }
+    }
+  }
+}
+
 // ------------------------------------------------ x[r, c] = act(x[r, c] + bias[c]) for c < cols
 template <typename TA>
 __global__ void bias_act_kernel(TA* __restrict__ x, int ld, const float* __restrict__ bias, int cols, int mode,
@@ -204,6 +297,15 @@ __global__ void bias_act_kernel(TA* __restrict__ x, int ld, const float* __restr
     if (bias != nullptr) v = to_float(from_float<TA>(v + bias[c]));   // (the biased projection is what is stored)
     p[c] = from_float<TA>(activate(v, mode));
   }
+}
+
+// ------------------------------------------------ y[i] = act(x[i]): a float32 product into the activation type
+template <typename TA>
+__global__ void act_cast_kernel(const float* __restrict__ x, TA* __restrict__ y, int n, int mode) {
+  pdl_launch();
+  pdl_wait();
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) y[i] = from_float<TA>(activate(x[i], mode));
 }
 
 // ------------------------------------------------ cache[page, head, offset, :] = src[t, col + head * dim : ...]
@@ -488,6 +590,35 @@ int rl_sandwich_norm(float* residual, const void* delta, int ld_delta, const voi
   RL_LAUNCH_END();
 }
 
+// Rows of up to 16 x 1,024 elements (cudaErrorInvalidValue beyond).
+int rl_sum_norm(float* residual, const void* delta, int ld_delta, const float* w, const float* scale, float alpha,
+                float eps, void* out, int ld_out, int act_dtype, int rows, int hidden, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  const int pieces = (hidden + 3) / 4, nv = pieces <= 1024 ? 1 : (pieces <= 2048 ? 2 : 4);
+  if (pieces > 4096) return static_cast<int>(cudaErrorInvalidValue);
+  const int th = max(32, ((pieces + nv - 1) / nv + 31) / 32 * 32);
+  const size_t act = act_dtype == RL_F32 ? 16 : 8;
+  const bool vec = hidden % 4 == 0 && ld_delta % 4 == 0 && ld_out % 4 == 0 && reinterpret_cast<uintptr_t>(residual) % 16 == 0 &&
+                   reinterpret_cast<uintptr_t>(w) % 16 == 0 && reinterpret_cast<uintptr_t>(scale) % 16 == 0 &&
+                   reinterpret_cast<uintptr_t>(delta) % act == 0 && reinterpret_cast<uintptr_t>(out) % act == 0;
+#define RL_CASE(TA, NV)                                                                                            \
+  do {                                                                                                             \
+    if (vec) launch_kernel(sum_norm_kernel<TA, NV, true>, dim3(rows), dim3(th), 0, stream, residual,               \
+                           static_cast<const TA*>(delta), ld_delta, w, scale, alpha, eps, static_cast<TA*>(out),   \
+                           ld_out, hidden);                                                                        \
+    else launch_kernel(sum_norm_kernel<TA, NV, false>, dim3(rows), dim3(th), 0, stream, residual,                  \
+                       static_cast<const TA*>(delta), ld_delta, w, scale, alpha, eps, static_cast<TA*>(out),       \
+                       ld_out, hidden);                                                                            \
+  } while (0)
+  if (act_dtype == RL_F32) {
+    if (nv == 1) RL_CASE(float, 1); else if (nv == 2) RL_CASE(float, 2); else RL_CASE(float, 4);
+  } else {
+    if (nv == 1) RL_CASE(bf16, 1); else if (nv == 2) RL_CASE(bf16, 2); else RL_CASE(bf16, 4);
+  }
+#undef RL_CASE
+  RL_LAUNCH_END();
+}
+
 int rl_bias_act(void* x, int act_dtype, int ld, const float* bias, int rows, int cols, int mode, cudaStream_t stream) {
   if (rows <= 0 || cols <= 0) return 0;
   const int th = 256;
@@ -499,6 +630,14 @@ int rl_bias_act(void* x, int act_dtype, int ld, const float* bias, int rows, int
     launch_kernel(bias_act_kernel<float>, grid, dim3(th), 0, stream, static_cast<float*>(x), ld, bias, cols, mode, vec_ok);
   else
     launch_kernel(bias_act_kernel<bf16>, grid, dim3(th), 0, stream, static_cast<bf16*>(x), ld, bias, cols, mode, vec_ok);
+  RL_LAUNCH_END();
+}
+
+int rl_act_cast(const float* x, void* y, int act_dtype, int n, int mode, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  const dim3 grid((n + 255) / 256);
+  if (act_dtype == RL_F32) launch_kernel(act_cast_kernel<float>, grid, dim3(256), 0, stream, x, static_cast<float*>(y), n, mode);
+  else launch_kernel(act_cast_kernel<bf16>, grid, dim3(256), 0, stream, x, static_cast<bf16*>(y), n, mode);
   RL_LAUNCH_END();
 }
 

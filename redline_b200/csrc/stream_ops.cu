@@ -253,6 +253,82 @@ __global__ void short_conv_state_kernel(const ConvArgs a, const TA* __restrict__
   }
 }
 
+// ------------------------------------------------------------------ token shift
+// Each of `groups` outputs mixes a token's row with the row of the token before it in its sequence, entry by
+// entry: y_g[t] = x_t + (x_(t-1) - x_t) * mu_g.  What comes before the step's portion is the sequence's slot of
+// the state ([slots, width] float32, zeros for a new request), which then receives the portion's last row.
+// One CTA per token.  The CTA of a sequence's first token alone touches the slot: it reads it, and when all
+// its threads have read, writes the last token's row there.
+struct ShiftArgs {
+  int ld_x, groups, width, tokens;
+  long long group_stride, slot_stride;       // elements between the outputs of two groups; floats between slots
+  const float* mu;                           // [groups, width]
+  const int32_t* seq_of_token;
+  const int32_t* state_slot;
+  float* state;
+  int vec;                                   // rows start on 16-byte boundaries, width is a multiple of 4
+};
+
+template <typename TX, typename TA>
+__global__ void __launch_bounds__(256)
+token_shift_kernel(const ShiftArgs a, const TX* __restrict__ x, TA* __restrict__ y) {
+  pdl_launch();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const int seq = a.seq_of_token[t];
+  const bool first = t == 0 || a.seq_of_token[t - 1] != seq;
+  const TX* row = x + static_cast<size_t>(t) * a.ld_x;
+  float* slot = a.state + static_cast<size_t>(a.state_slot[seq]) * a.slot_stride;
+  int last = t;                              // the sequence's last token of the step (asked for by its first)
+  if (first) {
+    int lo = t, hi = a.tokens;
+    while (lo + 1 < hi) {
+      const int mid = (lo + hi) >> 1;
+      if (a.seq_of_token[mid] == seq) lo = mid;
+      else hi = mid;
+    }
+    last = lo;
+  }
+  const TX* next = x + static_cast<size_t>(last) * a.ld_x;
+  TA* out = y + static_cast<size_t>(t) * a.width;
+  // (each thread reads and writes its own entries of the slot only: no thread waits for another)
+  if (a.vec) {
+    for (int c = threadIdx.x * 4; c < a.width; c += blockDim.x * 4) {
+      float v[4], p[4];
+      load4(row + c, v);
+      if (first) {
+        float n[4];
+        load4(slot + c, p);
+        load4(next + c, n);
+        store4(slot + c, n);
+      } else {
+        load4(row + c - a.ld_x, p);
+      }
+#pragma unroll 5
+      for (int g = 0; g < a.groups; ++g) {
+        float m[4];
+        load4(a.mu + static_cast<size_t>(g) * a.width + c, m);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) m[j] = fmaf(p[j] - v[j], m[j], v[j]);
+        store4(out + g * a.group_stride + c, m);
+      }
+    }
+    return;
+  }
+  for (int c = threadIdx.x; c < a.width; c += blockDim.x) {
+    const float v = to_float(row[c]);
+    float p;
+    if (first) {
+      p = slot[c];
+      slot[c] = to_float(next[c]);
+    } else {
+      p = to_float(row[c - a.ld_x]);
+    }
+    for (int g = 0; g < a.groups; ++g)
+      out[g * a.group_stride + c] = from_float<TA>(fmaf(p - v, a.mu[static_cast<size_t>(g) * a.width + c], v));
+  }
+}
+
 }  // namespace rl
 
 using namespace rl;
@@ -328,6 +404,28 @@ int rl_short_conv(int act_dtype, const void* x, int ld_x, int col_x, const void*
   } while (0)
   if (act_dtype == RL_F32) RL_CASE(float, float);
   else if (w_dtype == RL_F32) RL_CASE(bf16, float);
+  else RL_CASE(bf16, bf16);
+#undef RL_CASE
+  RL_LAUNCH_END();
+}
+
+// x float32 (x_dtype 0) or the activation type.
+int rl_token_shift(int x_dtype, int act_dtype, const void* x, int ld_x, const float* mu, int groups, void* y,
+                   long long group_stride, const int32_t* seq_of_token, const int32_t* state_slot, float* state,
+                   long long slot_stride, int tokens, int width, cudaStream_t stream) {
+  if (tokens <= 0 || groups <= 0) return 0;
+  ShiftArgs a;
+  a.ld_x = ld_x; a.groups = groups; a.width = width; a.tokens = tokens; a.group_stride = group_stride;
+  a.slot_stride = slot_stride; a.mu = mu; a.seq_of_token = seq_of_token; a.state_slot = state_slot; a.state = state;
+  a.vec = width % 4 == 0 && slot_stride % 4 == 0 && ld_x % 4 == 0 && group_stride % 4 == 0 &&
+          ((reinterpret_cast<uintptr_t>(state) | reinterpret_cast<uintptr_t>(mu) | reinterpret_cast<uintptr_t>(x) |
+            reinterpret_cast<uintptr_t>(y)) & 15) == 0;
+  const int th = width >= 1024 ? 256 : (width >= 256 ? 128 : 64);
+#define RL_CASE(TX, TA)                                                                                       \
+  launch_kernel(token_shift_kernel<TX, TA>, dim3(tokens), dim3(th), 0, stream, a, static_cast<const TX*>(x), \
+                static_cast<TA*>(y))
+  if (act_dtype == RL_F32) RL_CASE(float, float);
+  else if (x_dtype == RL_F32) RL_CASE(float, bf16);
   else RL_CASE(bf16, bf16);
 #undef RL_CASE
   RL_LAUNCH_END();

@@ -571,6 +571,7 @@ def attn_prefill(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcache: t
 
 ACT_NONE, ACT_RELU_SQ, ACT_GELU_ERF, ACT_SILU, ACT_GELU_TANH, ACT_SIGMOID = 0, 1, 2, 3, 4, 5
 ACT_CLAMPED_SWISH = 6      # gated_act only: min / clamp of gate and up, g * sigmoid(slope * g) * (up + 1)
+ACT_TANH = 7               # act_cast and bias_act
 ACTIVATIONS = {"none": ACT_NONE, "relu_squared": ACT_RELU_SQ, "gelu": ACT_GELU_ERF, "silu": ACT_SILU,
                "gelu_tanh": ACT_GELU_TANH}
 NORM_LAYER, NORM_RMS = 0, 1
@@ -609,6 +610,36 @@ def sandwich_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], post_w:
              _ptr(rows_idx), n, residual.shape[-1], float(eps), kind, _stream()), "sandwich_norm")
 
 
+SUM_NORM_MAX_WIDTH = 16384
+
+
+def sum_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: Optional[torch.Tensor],
+             scale: Optional[torch.Tensor], alpha: float, eps: float, out: Optional[torch.Tensor],
+             rows: Optional[int] = None) -> None:
+    """residual (float32 stream) = rmsnorm(alpha * residual + scale * delta) * weight, out = the new rows in out's
+    type (out given); without ``delta`` only the copy.  weight and scale float32 [width] (scale None: ones)."""
+    _need_cuda(residual, delta, weight, scale, out)
+    n = rows if rows is not None else residual.shape[0]
+    act = out if out is not None else delta
+    if act is None:
+        return
+    width = residual.shape[1]
+    if residual.dtype != torch.float32 or not residual.is_contiguous() or width > SUM_NORM_MAX_WIDTH:
+        raise KernelError(f"sum_norm: the stream must be contiguous float32 rows of up to {SUM_NORM_MAX_WIDTH} entries")
+    for t in (weight, scale):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != width or not t.is_contiguous()):
+            raise KernelError("sum_norm: weight and scale are contiguous float32 [width]")
+    if (delta is not None and (weight is None or delta.stride(1) != 1 or delta.shape[1] != width)) \
+            or (out is not None and (out.stride(1) != 1 or out.dtype != act.dtype)) \
+            or (delta is not None and out is not None and delta.dtype != out.dtype):
+        raise KernelError("sum_norm: delta (with a weight) and out have one type and contiguous rows")
+    f = _fn(_rw(), "rl_sum_norm", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p, c_int, c_int,
+                                   c_int, c_int, c_void_p])
+    _check(f(_ptr(residual), _ptr(delta), delta.stride(0) if delta is not None else 0, _ptr(weight), _ptr(scale),
+             float(alpha), float(eps), _ptr(out), out.stride(0) if out is not None else 0, _code(act.dtype), n, width,
+             _stream()), "sum_norm")
+
+
 def bias_act(x: torch.Tensor, bias: Optional[torch.Tensor], act: int, cols: Optional[int] = None,
              rows: Optional[int] = None) -> None:
     """In place: x[r, c] = act(x[r, c] + bias[c]) for c < cols (x may be a row-strided view; bias float32)."""
@@ -620,6 +651,15 @@ def bias_act(x: torch.Tensor, bias: Optional[torch.Tensor], act: int, cols: Opti
     f = _fn(_rw(), "rl_bias_act", [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p])
     _check(f(_ptr(x), _code(x.dtype), x.stride(0), _ptr(bias), rows if rows is not None else x.shape[0],
              cols if cols is not None else x.shape[1], act, _stream()), "bias_act")
+
+
+def act_cast(x: torch.Tensor, y: torch.Tensor, act: int) -> None:
+    """y = act(x) element by element: x contiguous float32, y contiguous of any engine type."""
+    _need_cuda(x, y)
+    if x.dtype != torch.float32 or not x.is_contiguous() or not y.is_contiguous() or x.numel() != y.numel():
+        raise KernelError("act_cast: a contiguous float32 tensor and a contiguous output of its size")
+    f = _fn(_rw(), "rl_act_cast", [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(x), _ptr(y), _code(y.dtype), x.numel(), act, _stream()), "act_cast")
 
 
 def cache_store(src: torch.Tensor, col: int, heads: int, dim: int, slots: torch.Tensor, cache: torch.Tensor,
@@ -817,32 +857,51 @@ def _latent() -> ctypes.CDLL:
     return _lib("latent", "latent.cu")
 
 
-def latent_prep(proj: torch.Tensor, positions: torch.Tensor, tokens: int, heads: int, dn: int, dr: int, rank: int,
-                rot_dims: int, norm_w: torch.Tensor, eps: float, cos: Optional[torch.Tensor], sin: Optional[torch.Tensor],
-                qa: torch.Tensor, slots: Optional[torch.Tensor], cache: torch.Tensor, page_size: int,
-                status: torch.Tensor) -> None:
-    """Rows of ``proj``: per head a query [dn unrotated | dr rotated], then [latent of ``rank`` | key part of dr].
-    The latent is RMS-normed (float32, weight ``norm_w``); the key part and every head's rotated query part turn
-    by the token's position (the first ``rot_dims`` rotated entries, entry i with i + rot_dims/2; cos / sin
-    float32 [positions, rot_dims/2]); [latent | key part] goes into ``cache`` [pages, 1, page, rank + dr] at the
-    token's slot (negative: not written), the rotated query parts into columns [rank, rank + dr) of every
-    head of ``qa`` [tokens, heads * (rank + dr)] (csrc/latent.cu)."""
-    _need_cuda(proj, positions, norm_w, cos, sin, qa, slots, cache)
-    if proj.dtype != qa.dtype or proj.dtype != cache.dtype or proj.stride(1) != 1 or qa.stride(1) != 1 \
-            or not cache.is_contiguous() or norm_w.numel() != rank:
-        raise KernelError("latent_prep: projection, query rows and cache have one type and contiguous rows")
-    if dr > 0 and (cos is None or sin is None or cos.dtype != torch.float32 or cos.shape[1] * 2 != rot_dims
-                   or rot_dims > dr or not cos.is_contiguous() or not sin.is_contiguous()):
+def latent_prep(q: Optional[torch.Tensor], latent: Optional[torch.Tensor], positions: torch.Tensor, tokens: int,
+                heads: int, dn: int, dr: int, rank: int, rot_dims: int, norm_w: Optional[torch.Tensor], eps: float,
+                cos: Optional[torch.Tensor], sin: Optional[torch.Tensor], qa: Optional[torch.Tensor],
+                slots: Optional[torch.Tensor], cache: Optional[torch.Tensor], page_size: int, status: torch.Tensor,
+                pairs: bool = False, dq: Optional[torch.Tensor] = None, dq_w: Optional[torch.Tensor] = None,
+                dq_out: Optional[torch.Tensor] = None) -> None:
+    """Three jobs of csrc/latent.cu, each done where its tensors are given (all row-strided views of one type).
+    ``q``, rows of per head [dn unrotated | dr rotated]: every head's rotated part turns by the token's position
+    into columns [rank, rank + dr) of the head in ``qa`` [tokens, heads * (rank + dr)].  ``latent``, rows of
+    [latent of ``rank`` | key part of dr]: the latent is RMS-normed (float32, weight ``norm_w``), the key part
+    turns, both go into ``cache`` [pages, 1, page, rank + dr] at the token's slot (negative: not written).
+    ``dq`` [tokens, n]: dq_out = rmsnorm(dq) * dq_w.  The first ``rot_dims`` rotated entries turn, entry i with
+    entry i + rot_dims/2 or (``pairs``) 2i with 2i + 1; cos / sin float32 [positions, rot_dims/2]."""
+    _need_cuda(q, latent, positions, norm_w, cos, sin, qa, slots, cache, dq, dq_w, dq_out)
+    given = [t for t in (q, latent, dq, qa, cache, dq_out) if t is not None]
+    if any(t.dtype != given[0].dtype for t in given) or any(t is not None and t.stride(1) != 1 for t in (q, latent, dq, qa, dq_out)):
+        raise KernelError("latent_prep: the buffers have one type and contiguous rows")
+    if latent is not None and (cache is None or norm_w is None or not cache.is_contiguous() or norm_w.numel() != rank
+                               or latent.shape[1] < rank + dr):
+        raise KernelError("latent_prep: a latent comes with its norm's weight and a contiguous cache")
+    if q is not None and (qa is None or q.shape[1] < heads * (dn + dr) or qa.shape[1] < heads * (rank + dr)):
+        raise KernelError("latent_prep: rows too short for the heads")
+    if dq is not None and (dq_w is None or dq_out is None or dq_w.numel() != dq.shape[1] or dq_out.shape[1] != dq.shape[1]
+                           or (norm_w is not None and norm_w.dtype != dq_w.dtype)):
+        raise KernelError("latent_prep: the queries' latent comes with a weight (of the other weight's type) and a buffer")
+    if dr > 0 and (q is not None or latent is not None) and (
+            cos is None or sin is None or cos.dtype != torch.float32 or cos.shape[1] * 2 != rot_dims
+            or rot_dims > dr or not cos.is_contiguous() or not sin.is_contiguous()):
         raise KernelError("latent_prep: cos / sin are float32 [positions, rot_dims / 2], rot_dims at most dr")
-    if proj.shape[1] < heads * (dn + dr) + rank + dr or qa.shape[1] < heads * (rank + dr):
-        raise KernelError("latent_prep: rows too short for the heads and the latent")
+    turns = dr > 0 and (q is not None or latent is not None)
+    w = norm_w if norm_w is not None else dq_w
     f = _fn(_latent(), "rl_latent_prep",
-            [c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_float,
-             c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p])
-    _check(f(_code(proj.dtype), _code(norm_w.dtype), _ptr(proj), proj.stride(0), _ptr(positions), tokens, heads, dn, dr,
-             rank, rot_dims if dr > 0 else 0, _ptr(norm_w), float(eps), _ptr(cos), _ptr(sin),
-             cos.shape[0] if cos is not None else 0, _ptr(qa), qa.stride(0), _ptr(slots), _ptr(cache), page_size,
-             cache.shape[0] * page_size, _ptr(status), _stream()), "latent_prep")
+            [c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+             c_void_p, c_float, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_longlong,
+             c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p])
+
+    def ld(t):
+        return t.stride(0) if t is not None else 0
+
+    _check(f(_code(given[0].dtype), _code(w.dtype) if w is not None else 0, _ptr(q), ld(q), _ptr(latent), ld(latent),
+             _ptr(positions), tokens, heads, dn, dr if turns else 0, rank, rot_dims if turns else 0, 1 if pairs else 0,
+             _ptr(norm_w), float(eps), _ptr(cos), _ptr(sin), cos.shape[0] if cos is not None else 0, _ptr(qa), ld(qa),
+             _ptr(slots), _ptr(cache), page_size, cache.shape[0] * page_size if cache is not None else 0, _ptr(dq),
+             ld(dq), dq.shape[1] if dq is not None else 0, _ptr(dq_w), _ptr(dq_out), ld(dq_out), _ptr(status),
+             _stream()), "latent_prep")
 
 
 def head_linear(x: torch.Tensor, x_col: int, x_head: int, w: torch.Tensor, y: torch.Tensor, y_col: int, y_head: int,
@@ -877,31 +936,104 @@ def linear_attention_chunks(longest: int) -> Tuple[int, int]:
     return chunk, (longest + chunk - 1) // chunk
 
 
-def linear_attention(qkv: torch.Tensor, q_col: int, k_col: int, v_col: int, seq_of_token: torch.Tensor,
-                     state_slot: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
-                     tokens: int, sequences: int, heads: int, dim: int, vdim: int,
-                     chunk_state: Optional[torch.Tensor] = None, chunk: int = 0, max_chunks: int = 1) -> None:
-    """S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head over every sequence of the step, from and
-    into the sequences' state slots (csrc/linear_attention.cu).  qkv [tokens, *] holds q, k (heads x dim)
-    and v (heads x vdim) at the given columns; state float32 [slots, heads, dim, vdim]; out float32
-    [tokens, heads * vdim].  With ``chunk_state`` (float32, sequences * max_chunks * heads * dim * vdim)
-    sequences are cut into chunks of ``chunk`` tokens that run side by side."""
-    _need_cuda(qkv, state, out)
-    if state.dtype != torch.float32 or out.dtype != torch.float32 or decay.dtype != torch.float32 \
-            or not state.is_contiguous() or not out.is_contiguous() or qkv.stride(1) != 1:
-        raise KernelError("linear_attention: state, decay and out are contiguous float32")
+GATE_NONE, GATE_SIGMOID, GATE_SILU = 0, 1, 2
+
+
+def _lin(dim: int) -> ctypes.CDLL:
     if not 1 <= dim <= 256:
         raise KernelError(f"linear_attention takes key sizes up to 256; got {dim}")
-    if chunk_state is not None and max_chunks > 1 and \
-            chunk_state.numel() < sequences * max_chunks * heads * dim * vdim:
-        raise KernelError("linear_attention: chunk workspace too small")
-    f = _fn(_lib(f"linear_attention_d{dim}", "linear_attention.cu", {"RL_LIN_DIM": dim}), "rl_linear_attention",
-            [c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-             c_int, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    return _lib(f"linear_attention_d{dim}", "linear_attention.cu", {"RL_LIN_DIM": dim})
+
+
+def linear_attention_finishes(dim: int, vdim: int) -> bool:
+    """Whether the recurrence's kernel can also norm, weigh and gate the heads (``y`` of ``linear_attention``)."""
+    return bool(_fn(_lin(dim), "rl_linear_one_block", [c_int])(vdim))
+
+
+def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, seq_of_token: torch.Tensor,
+                     state_slot: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: Optional[torch.Tensor],
+                     tokens: int, sequences: int, heads: int, dim: int, vdim: int,
+                     chunk_state: Optional[torch.Tensor] = None, chunk: int = 0, max_chunks: int = 1,
+                     k_scale: float = 1.0, cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None,
+                     positions: Optional[torch.Tensor] = None, decay_bias: Optional[torch.Tensor] = None,
+                     bonus: Optional[torch.Tensor] = None, chunk_decay: Optional[torch.Tensor] = None,
+                     y: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_mode: int = GATE_NONE,
+                     norm_w: Optional[torch.Tensor] = None, eps: float = 0.0,
+                     status: Optional[torch.Tensor] = None) -> None:
+    """A recurrence per head over every sequence of the step, from and into the sequences' state slots
+    (csrc/linear_attention.cu).  q, k [tokens, heads * dim] and v [tokens, heads * vdim] are row-strided views of
+    one type; state float32 [slots, heads * dim * vdim] (or [slots, heads, dim, vdim]).
+
+    ``bonus`` None: S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, ``decay`` float32 [heads].  Otherwise, per
+    key channel, o_t = S_(t-1)^T q_t + (sum q u k) v_t, S_t = diag(a_t) S_(t-1) + k_t v_t^T with
+    a_t = exp(-exp(decay_t + decay_bias)): ``decay`` float32 [tokens, heads * dim], ``decay_bias`` and ``bonus`` u
+    float32 [heads * dim].  q and k are rotated first (``cos``, ``sin`` [positions, pairs]: entry i with entry
+    i + pairs), k multiplied by ``k_scale``.
+
+    ``out`` receives o (float32 [tokens, heads * vdim]); or ``y`` (where ``linear_attention_finishes``) the
+    finished heads, o / sqrt(mean over the head (o^2) + eps) * norm_w * act(gate), in the activation type.
+    With ``chunk_state`` (float32, sequences * max_chunks * heads * dim * vdim; per channel also ``chunk_decay``,
+    sequences * max_chunks * heads * dim) sequences are cut into chunks of ``chunk`` tokens that run side by
+    side."""
+    _need_cuda(q, k, v, state, out, y, gate, decay, decay_bias, bonus, chunk_state, chunk_decay, norm_w)
+    channel = bonus is not None
+    for t in (decay, decay_bias, bonus, out, norm_w, chunk_state, chunk_decay):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
+            raise KernelError("linear_attention: decays, bonus, weights and float outputs are contiguous float32")
+    flat = state.view(state.shape[0], -1) if state.is_contiguous() else state
+    if state.dtype != torch.float32 or flat.stride(1) != 1 or flat.shape[1] < heads * dim * vdim:
+        raise KernelError("linear_attention: the state is float32 [slots, heads * dim * vdim]")
+    if any(t.dtype != q.dtype or t.stride(1) != 1 for t in (k, v)) or q.stride(1) != 1 or q.shape[1] != heads * dim \
+            or k.shape[1] != heads * dim or v.shape[1] != heads * vdim:
+        raise KernelError("linear_attention: q, k [tokens, heads * dim] and v [tokens, heads * vdim] of one type")
+    if channel and (decay_bias is None or decay_bias.numel() != heads * dim or bonus.numel() != heads * dim
+                    or decay.numel() < tokens * heads * dim):
+        raise KernelError("linear_attention: decays per channel come with a bias and a bonus of [heads * dim]")
+    if not channel and decay.numel() != heads:
+        raise KernelError("linear_attention: one decay per head")
+    if (out is None) == (y is None) or (y is not None and (y.dtype != q.dtype or y.stride(1) != 1
+                                                           or not linear_attention_finishes(dim, vdim))):
+        raise KernelError("linear_attention: either float32 sums or (where one CTA has a head) the finished heads")
+    if gate is not None and (gate.dtype != q.dtype or gate.stride(1) != 1 or gate.shape[1] != heads * vdim):
+        raise KernelError("linear_attention: the gate has one entry per output and the activation type")
+    pairs = 0
+    if cos is not None:
+        pairs = cos.shape[1]
+        if sin is None or positions is None or status is None or cos.dtype != torch.float32 or not cos.is_contiguous() \
+                or not sin.is_contiguous() or 2 * pairs > dim:
+            raise KernelError("linear_attention: a rotation needs float32 tables, positions and a status word")
     chunked = chunk_state is not None and max_chunks > 1
-    _check(f(_code(qkv.dtype), _ptr(qkv), qkv.stride(0), q_col, k_col, v_col, _ptr(seq_of_token), _ptr(state_slot),
-             _ptr(decay), _ptr(state), _ptr(out), _ptr(chunk_state) if chunked else None, tokens, sequences, heads,
-             vdim, chunk, max_chunks if chunked else 1, _stream()), "linear_attention", 3 if chunked else 1)
+    if chunked and (chunk_state.numel() < sequences * max_chunks * heads * dim * vdim
+                    or (channel and (chunk_decay is None or chunk_decay.numel() < sequences * max_chunks * heads * dim))):
+        raise KernelError("linear_attention: chunk workspace too small")
+    f = _fn(_lin(dim), "rl_linear_attention",
+            [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int,
+             c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p,
+             c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+             c_void_p])
+    _check(f(_code(q.dtype), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), float(k_scale), _ptr(cos),
+             _ptr(sin), _ptr(positions), pairs, cos.shape[0] if cos is not None else 0, _ptr(seq_of_token),
+             _ptr(state_slot), _ptr(decay), _ptr(decay_bias), _ptr(bonus), _ptr(state), flat.stride(0), _ptr(out), _ptr(y),
+             y.stride(0) if y is not None else 0, _ptr(gate), gate.stride(0) if gate is not None else 0,
+             gate_mode if gate is not None else GATE_NONE, _ptr(norm_w), float(eps),
+             _ptr(chunk_state) if chunked else None, _ptr(chunk_decay) if chunked and channel else None, _ptr(status), tokens,
+             sequences, heads, vdim, chunk, max_chunks if chunked else 1, _stream()), "linear_attention", 3 if chunked else 1)
+
+
+def linear_output(o: torch.Tensor, gate: Optional[torch.Tensor], gate_mode: int, norm_w: Optional[torch.Tensor],
+                  y: torch.Tensor, tokens: int, heads: int, dim: int, vdim: int, eps: float) -> None:
+    """y = o / sqrt(mean over the head (o^2) + eps) (* norm_w) (* act(gate)): o float32 [tokens, heads * vdim],
+    gate and y row-strided views of the activation type, norm_w float32 [heads * vdim]."""
+    _need_cuda(o, gate, norm_w, y)
+    if o.dtype != torch.float32 or not o.is_contiguous() or y.stride(1) != 1 \
+            or (gate is not None and (gate.dtype != y.dtype or gate.stride(1) != 1)) \
+            or (norm_w is not None and (norm_w.dtype != torch.float32 or norm_w.numel() != heads * vdim)):
+        raise KernelError("linear_output: bad shapes")
+    f = _fn(_lin(dim), "rl_linear_output", [c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
+                                            c_int, c_int, c_float, c_void_p])
+    _check(f(_code(y.dtype), _ptr(o), _ptr(gate), gate.stride(0) if gate is not None else 0,
+             gate_mode if gate is not None else GATE_NONE, _ptr(norm_w), _ptr(y), y.stride(0), tokens, heads, vdim,
+             float(eps), _stream()), "linear_output")
 
 
 # ------------------------------------------------------- matrix memory with exponential gates
@@ -1059,6 +1191,24 @@ def short_conv(x: torch.Tensor, col_x: int, w: torch.Tensor, bias: Optional[torc
              1 if single else 0, _stream()), "short_conv", 2 if (taps > 1 and not single) else 1)
 
 
+def token_shift(x: torch.Tensor, mu: torch.Tensor, y: torch.Tensor, seq_of_token: torch.Tensor,
+                state_slot: torch.Tensor, state: torch.Tensor, tokens: int) -> None:
+    """y[g, t] = x_t + (x_(t-1) - x_t) * mu[g] for every row g of ``mu`` (float32 [groups, width]), x_(t-1) the row
+    of the token before in t's own sequence; what lies before the step's portion comes from the sequence's slot of
+    ``state`` (float32 [slots, width], zeros for a new request), which then receives the portion's last row
+    (csrc/stream_ops.cu).  x [tokens, width] is float32 or y's type; y [groups, *, width]."""
+    _need_cuda(x, mu, y, state)
+    groups, width = mu.shape
+    if mu.dtype != torch.float32 or not mu.is_contiguous() or state.dtype != torch.float32 or state.stride(1) != 1 \
+            or state.shape[1] < width or x.stride(1) != 1 or x.shape[1] != width or y.shape[0] != groups \
+            or y.shape[2] != width or y.stride(2) != 1 or y.stride(1) != width or x.dtype not in (torch.float32, y.dtype):
+        raise KernelError("token_shift: bad shapes or types")
+    f = _fn(_so(), "rl_token_shift", [c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_longlong, c_void_p,
+                                      c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p])
+    _check(f(_code(x.dtype), _code(y.dtype), _ptr(x), x.stride(0), _ptr(mu), groups, _ptr(y), y.stride(0),
+             _ptr(seq_of_token), _ptr(state_slot), _ptr(state), state.stride(0), tokens, width, _stream()), "token_shift")
+
+
 # ------------------------------------------------------------------- the gated delta rule
 
 def _delta(dim: int) -> ctypes.CDLL:
@@ -1211,8 +1361,9 @@ def moe_gemm(src: torch.Tensor, src_div: int, w: torch.Tensor, dst: torch.Tensor
 
 def moe_combine(y: torch.Tensor, weight: torch.Tensor, shared: Optional[torch.Tensor], out: torch.Tensor,
                 tokens: int, top: int, choice: Optional[torch.Tensor] = None, real_experts: int = 0,
-                x: Optional[torch.Tensor] = None) -> None:
+                x: Optional[torch.Tensor] = None, shared_gate: Optional[torch.Tensor] = None) -> None:
     """out[t] = sum_k weight[t, k] * y[t * top + k] (+ shared[t]), k in order; y, shared and out contiguous.
+    ``shared_gate`` (a column [tokens] or [tokens, 1] of a float32 buffer): shared[t] counts sigmoid(gate_t) times.
     With ``choice`` and ``x`` (the experts' input [tokens, width]) a pair whose chosen index is at least
     ``real_experts`` stands for the identity: its term is weight[t, k] * x[t]."""
     _need_cuda(y, weight, out, choice, x)
@@ -1220,10 +1371,13 @@ def moe_combine(y: torch.Tensor, weight: torch.Tensor, shared: Optional[torch.Te
         raise KernelError("moe_combine: contiguous tensors")
     if (choice is None) != (x is None) or (x is not None and (x.dtype != out.dtype or x.stride(1) != 1)):
         raise KernelError("moe_combine: identity experts need the choices and the experts' input in out's type")
+    if shared_gate is not None and (shared is None or shared_gate.dtype != torch.float32):
+        raise KernelError("moe_combine: a shared expert's gate is float32")
     f = _fn(_moe(), "rl_moe_combine", [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p,
-                                        c_int, c_void_p, c_int, c_void_p])
+                                        c_int, c_void_p, c_int, c_void_p, c_int, c_void_p])
     _check(f(_code(out.dtype), _ptr(y), _ptr(weight), _ptr(shared), _ptr(out), tokens, out.shape[1], top, _ptr(choice),
-             real_experts, _ptr(x), x.stride(0) if x is not None else 0, _stream()), "moe_combine")
+             real_experts, _ptr(x), x.stride(0) if x is not None else 0, _ptr(shared_gate),
+             shared_gate.stride(0) if shared_gate is not None else 0, _stream()), "moe_combine")
 
 
 # -------------------------------------------------------------------- sampling

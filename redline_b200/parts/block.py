@@ -1,7 +1,8 @@
 """Pre-norm residual block: h += mixer(norm(h)); h += ffn(norm(h)), the residual
 stream h in float32 (reference: src/cuda/model/llama.cpp:116-139).  A layer without a
 feed-forward stops after the first half.  Beside it the arrangements that norm a
-sublayer's output: on both sides ("sandwich") or on the output only ("outnorm")."""
+sublayer's output: on both sides ("sandwich") or on the output only ("outnorm"); and the one that norms the
+stream after every sum ("postnorm")."""
 
 from __future__ import annotations
 
@@ -135,6 +136,7 @@ class OutNormBlock(Block):
     nothing pending."""
 
     reads_stream = True
+    closing_op = "post_norm+add"
     mixer_post_norm = None
     ffn_post_norm = None
     AS_IS = "the stream as it is"          # marks ctx.block_normed: the buffer holds the stream, not a norm of it
@@ -153,16 +155,30 @@ class OutNormBlock(Block):
             from ..ops import kernels
             kernels.sandwich_norm(residual, pending, None, None, x if copy else None, 0.0, kernels.NORM_RMS, rows=T)
             op_mark(ctx, "stream_copy", nbytes=PreNormBlock._norm_bytes(residual, pending, x))
-        a = self.mixer.forward(x, ctx, cache, state)
+        ctx.block_stream = residual              # (a mixer may read the float32 rows that x was rounded from)
+        try:
+            a = self.mixer.forward(x, ctx, cache, state)
+        finally:
+            ctx.block_stream = None
         last = self.ffn is None
         nxt = copy and (not last or isinstance(ctx.block_next, OutNormBlock))
         self.mixer_post_norm.add_post_cast(residual, a, x if nxt else None, rows=T)
-        op_mark(ctx, "post_norm+add", nbytes=PreNormBlock._norm_bytes(residual, a, x))
+        op_mark(ctx, self.closing_op, nbytes=PreNormBlock._norm_bytes(residual, a, x))
         if not last:
             f = self.ffn.forward(x, ctx)
             nxt = copy and isinstance(ctx.block_next, OutNormBlock)
             self.ffn_post_norm.add_post_cast(residual, f, x if nxt else None, rows=T)
-            op_mark(ctx, "post_norm+add", nbytes=PreNormBlock._norm_bytes(residual, f, x))
+            op_mark(ctx, self.closing_op, nbytes=PreNormBlock._norm_bytes(residual, f, x))
         if nxt:
             ctx.block_normed = (self.AS_IS, x)
         return None
+
+
+@register("block", "postnorm")
+class PostNormBlock(OutNormBlock):
+    """h = norm_1(alpha h + s_1 * mixer(h)); h = norm_2(alpha h + s_2 * ffn(h)): the sublayers read the stream
+    itself and the stream is normed after every sum.  The norms (``rmsnorm_sum``) hold alpha and the vectors s;
+    everything else is as in "outnorm": one row-wise kernel per sublayer, which also writes the rounded copy for
+    the sublayer after it."""
+
+    closing_op = "sum+norm"

@@ -2,7 +2,7 @@
 ("routed_experts", whose experts may also be gated, W_down (f(W_gate h) * (W_up h)), and whose router may
 have a bias): a router scores the experts per token in float32 (sigmoid or softmax), experts lie in
 equal groups of neighbours of which only the best ``group_keep`` (by the sum of their ``group_top`` best
-scores) can be chosen, the ``top`` best experts of those run for the token, weighted by their scores
+choice scores) can be chosen, the ``top`` best experts of those run for the token, weighted by their scores
 (as they are, or divided by their sum), and a shared expert of the same form may run for every token.
 The experts' products are grouped matrix products over (token, expert) pairs listed expert by expert on
 the device (csrc/moe.cu); nothing of the routing is read by the host.
@@ -12,7 +12,8 @@ weight * h and runs no product); ``choice_bias``: a number per router output tha
 the choice alone (the weights are the scores without it); ``renorm_floor`` joins the sum the chosen scores are
 divided by, ``weight_scale`` multiplies the weights; gated experts may use ``clamped_swish`` (gate and up
 clamped by ``limit``, g * sigmoid(slope * g) * (up + 1)); the shared expert of gated experts is gated too, with
-``shared_limit`` as its clamp.
+``shared_limit`` as its clamp; ``shared_gate`` multiplies the shared expert by sigmoid(w_sg . h), one number per
+token, whose product is one more row of the router's.
 """
 
 from __future__ import annotations
@@ -91,6 +92,7 @@ class RoutedExpertsParams:
     limit: float = 0.0                   # clamped_swish: the clamp of gate and up
     slope: float = 1.0                   # clamped_swish: g * sigmoid(slope * g)
     shared_limit: float = 0.0            # the shared expert's clamp (0: ``limit``)
+    shared_gate: bool = False            # the shared expert counts sigmoid(w_sg . h) times
 
 
 @register("ffn", "routed_experts")
@@ -111,6 +113,8 @@ class RoutedExperts(FeedForward):
             raise ValueError("routed_experts: clamped_swish goes with gated experts and a positive limit")
         self.act = kernels.ACT_CLAMPED_SWISH if self.clamped else kernels.ACTIVATIONS[p.activation]
         self.shared = None
+        if p.shared_gate and p.shared_intermediate_size <= 0:
+            raise ValueError("routed_experts: a gate of the shared expert needs a shared expert")
         if p.shared_intermediate_size > 0 and p.gated:
             from .mlp import GatedMLPParams, SwiGLUMLP
             from .spec import PartSpec
@@ -137,16 +141,20 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             if p.gated:
                 t["shared_gate"] = TensorSpec((p.shared_intermediate_size, p.hidden_size))
+            if p.shared_gate:
+                t["shared_sg"] = TensorSpec((1, p.hidden_size))
             t["shared_up"] = TensorSpec((p.shared_intermediate_size, p.hidden_size))
             t["shared_down"] = TensorSpec((p.hidden_size, p.shared_intermediate_size))
         return t
 
     def fused(self) -> Dict[str, list]:
         n = self.params.num_experts
-        if self.params.gated:      # every expert's gate rows, then its up rows
-            return {"up_all": [f"{m}{e}" for e in range(n) for m in ("gate", "up")],
-                    "down_all": [f"down{e}" for e in range(n)]}
-        return {"up_all": [f"up{e}" for e in range(n)], "down_all": [f"down{e}" for e in range(n)]}
+        # (gated: every expert's gate rows, then its up rows)
+        stems = ("gate", "up") if self.params.gated else ("up",)
+        out = {"up_all": [f"{m}{e}" for e in range(n) for m in stems], "down_all": [f"down{e}" for e in range(n)]}
+        if self.params.shared_gate:
+            out["router_all"] = ["router", "shared_sg"]
+        return out
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         p = self.params
@@ -163,7 +171,10 @@ class RoutedExperts(FeedForward):
         self.b_router = tensors["router_bias"].float().contiguous() if p.router_bias else None
         self.b_choice = tensors["choice_bias"].float().contiguous() if p.choice_bias else None
         self.w_down = stacked("down_all", "down")      # [experts * hidden, ff]
-        self.w_router = tensors["router"]
+        self.w_router = tensors.get("router")
+        if p.shared_gate:
+            self.w_router = tensors["router_all"] if "router_all" in tensors else torch.cat(
+                [tensors["router"], tensors["shared_sg"].to(tensors["router"].dtype)], dim=0).contiguous()
         if self.shared is not None and p.gated:
             self.shared.load({"gate": tensors["shared_gate"], "up": tensors["shared_up"], "down": tensors["shared_down"]})
         elif self.shared is not None:
@@ -189,8 +200,10 @@ class RoutedExperts(FeedForward):
         tile_rows = ws.get("moe.tile_rows", (cap_tiles,), torch.int32)
         meta = ws.get("moe.meta", (4,), torch.int32)
         # the router's logits as a matrix product with float32 sums and a float32 result, then the choice
-        logits = ws.get("moe.logits", (rt.max_tokens, self.outputs), torch.float32)[:T]
-        linear(x, self.w_router, logits)
+        # (behind the router's outputs, the shared expert's gate if it has one)
+        scored = ws.get("moe.logits", (rt.max_tokens, self.w_router.shape[0]), torch.float32)[:T]
+        linear(x, self.w_router, scored)
+        logits = scored[:, :self.outputs]
         kernels.moe_route(logits, None, choice, weight, T, p.groups, p.group_keep, p.group_top, p.top,
                           softmax=p.score == "softmax", renorm=p.renormalize, bias=self.b_router,
                           choice_bias=self.b_choice, weight_scale=p.weight_scale, renorm_floor=p.renorm_floor)
@@ -218,9 +231,11 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             shared = self.shared.run(x, ctx, "moe.shared")
         out = ws.get("ffn.out", (rt.max_tokens, p.hidden_size), rt.dtype)[:T]
+        gate = scored[:, self.outputs] if p.shared_gate else None
         if p.identity > 0:
-            kernels.moe_combine(y, weight, shared, out, T, p.top, choice=choice, real_experts=p.num_experts, x=x)
+            kernels.moe_combine(y, weight, shared, out, T, p.top, choice=choice, real_experts=p.num_experts, x=x,
+                                shared_gate=gate)
         else:
-            kernels.moe_combine(y, weight, shared, out, T, p.top)
+            kernels.moe_combine(y, weight, shared, out, T, p.top, shared_gate=gate)
         op_mark(ctx, "combine", nbytes=float((pairs + 2 * T) * p.hidden_size * elem))
         return out

@@ -1,6 +1,9 @@
 """RMSNorm fused with the residual add: y = x * rsqrt(mean(x^2) + eps) * w with the
-weight multiplying directly (no 1 + w), sums in float32
-(reference: src/cuda/kernels/elementwise.cu:29-64)."""
+weight multiplying directly, sums in float32
+(reference: src/cuda/kernels/elementwise.cu:29-64); designs that store the weight around
+zero (``zero_centred``) multiply by 1 + w, formed in float32 when the weights are loaded.
+``rmsnorm_sum`` norms the weighted sum of the stream and a sublayer's output, for blocks
+that norm after the sum."""
 
 from __future__ import annotations
 
@@ -18,6 +21,7 @@ from .spec import TensorSpec
 class RMSNormParams:
     size: int
     eps: float
+    zero_centred: bool = False
 
 
 @register("norm", "rmsnorm")
@@ -27,6 +31,8 @@ class RMSNorm(Norm):
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         self.weight = tensors["weight"]
+        if self.params.zero_centred:
+            self.weight = (1.0 + self.weight.float()).contiguous()
 
     def nbytes(self) -> int:
         return self.weight.numel() * self.weight.element_size()
@@ -36,3 +42,39 @@ class RMSNorm(Norm):
 
     def rms_params(self):
         return self.weight, self.params.eps
+
+
+@dataclass(frozen=True)
+class RMSNormSumParams:
+    size: int
+    eps: float
+    alpha: float = 1.0             # factor on the stream
+    zero_centred: bool = False
+    scaled: bool = False           # the sublayer's output is multiplied by a vector first
+
+
+@register("norm", "rmsnorm_sum")
+class RMSNormSum(Norm):
+    """stream = rmsnorm(alpha * stream + scale * delta) * weight: the norm after the sum ("postnorm" blocks)."""
+
+    def tensors(self) -> Dict[str, TensorSpec]:
+        t = {"weight": TensorSpec((self.params.size,))}
+        if self.params.scaled:
+            t["scale"] = TensorSpec((self.params.size,))
+        return t
+
+    def load(self, tensors: Dict[str, torch.Tensor]) -> None:
+        self.weight = tensors["weight"].float()
+        if self.params.zero_centred:
+            self.weight = 1.0 + self.weight
+        self.weight = self.weight.contiguous()
+        self.scale = tensors["scale"].float().contiguous() if self.params.scaled else None
+
+    def nbytes(self) -> int:
+        return self.weight.numel() * 4 * (2 if self.params.scaled else 1)
+
+    def add_post_cast(self, residual: torch.Tensor, delta: torch.Tensor, out: Optional[torch.Tensor],
+                      rows: Optional[int] = None) -> None:
+        """The norm of the sum in place on the stream; with ``out`` also out = the new stream rows in out's type."""
+        p = self.params
+        kernels.sum_norm(residual, delta, self.weight, self.scale, p.alpha, p.eps, out, rows=rows)

@@ -81,58 +81,24 @@ class NoPosition(PositionEncoding):
 
 @dataclass(frozen=True)
 class RotaryPairsParams:
-    dims: int              # how many entries of a head are rotated: the first ``dims`` (an even number)
-    base: float
-    max_positions: int
+    """Rotation of the first ``dims`` entries of a head, with optional YaRN scaling of the frequencies
+    (``factor`` 0 or 1: none)."""
 
-
-_pair_tables = {}          # tables shared by the parts that ask for the same ones
-
-
-@register("position", "rope_pairs")
-class RotaryPairs(PositionEncoding):
-    """Rotation of neighbouring pairs: entries (2i, 2i+1), i < dims / 2, of a head turn by the angle
-    pos * base^(-2i / dims); the entries from ``dims`` on stay as they are.  The tables hold the cosines and
-    sines [positions, dims / 2] in float32 of angles formed in double precision; the mixer applies them."""
-
-    pairing = "neighbours"
-
-    def __init__(self, spec, rt):
-        super().__init__(spec, rt)
-        p = self.params
-        if p.dims <= 0 or p.dims % 2 != 0:
-            raise ValueError(f"rope_pairs rotates an even number of entries, got {p.dims}")
-        n = max(min(p.max_positions, rt.max_seq_len) if rt.max_seq_len > 0 else p.max_positions, 1)
-        key = (p.dims, float(p.base), n, str(rt.device))
-        if key not in _pair_tables:
-            freq = np.asarray([float(p.base) ** (-2.0 * i / p.dims) for i in range(p.dims // 2)], dtype=np.float64)
-            angle = np.arange(n, dtype=np.float64)[:, None] * freq[None, :]
-            _pair_tables[key] = (torch.from_numpy(np.cos(angle).astype(np.float32)).to(rt.device),
-                                 torch.from_numpy(np.sin(angle).astype(np.float32)).to(rt.device))
-        self.cos, self.sin = _pair_tables[key]
-
-    def rotary_tables(self):
-        return self.cos, self.sin
-
-    def nbytes(self) -> int:
-        return 2 * self.cos.numel() * 4
-
-
-@dataclass(frozen=True)
-class RotaryHalvesParams:
-    """Rotation of the first ``dims`` entries of a head, entry i paired with entry i + dims / 2, with optional
-    YaRN scaling of the frequencies (``factor`` 0 or 1: none)."""
-
-    dims: int
+    dims: int                  # an even number
     base: float
     max_positions: int
     factor: float = 0.0        # YaRN: how far the context is stretched
-    original: int = 0          # the context length the frequencies were made for
+    original: float = 0        # the context length the frequencies were made for
     fast: float = 32.0         # pairs that turn at least so often within ``original`` keep their frequency
     slow: float = 1.0          # pairs that turn at most so often are divided by ``factor``
 
 
-def yarn_frequencies(p: RotaryHalvesParams) -> Tuple[List[float], float]:
+@dataclass(frozen=True)
+class RotaryHalvesParams(RotaryPairsParams):
+    """The same with entry i paired with entry i + dims / 2."""
+
+
+def yarn_frequencies(p: RotaryPairsParams) -> Tuple[List[float], float]:
     """(frequency of every pair, factor on cos and sin).  With f_i = base^(-2i/dims) and
     index(turns) = dims ln(original / (2 pi turns)) / (2 ln base): lo = max(floor(index(fast)), 0),
     hi = min(ceil(index(slow)), dims - 1), ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1); pair i turns at
@@ -154,34 +120,47 @@ def yarn_frequencies(p: RotaryHalvesParams) -> Tuple[List[float], float]:
     return out, 0.1 * math.log(p.factor) + 1.0
 
 
-_half_tables = {}
+_tables = {}          # tables shared by the parts that ask for the same ones
 
 
-@register("position", "rope_halves")
-class RotaryHalves(PositionEncoding):
+class PairTables(PositionEncoding):
     """Tables [positions, dims / 2] of cos and sin (float32 of angles formed in double precision, the YaRN
-    factor multiplied in); the mixer's kernel pairs entry i with entry i + dims / 2."""
+    factor multiplied in) for a rotation of pairs; the mixer's kernels apply them."""
 
-    pairing = "halves"
+    pairing = ""
 
     def __init__(self, spec, rt):
         super().__init__(spec, rt)
         p = self.params
         if p.dims <= 0 or p.dims % 2 != 0:
-            raise ValueError(f"rope_halves rotates an even number of entries, got {p.dims}")
+            raise ValueError(f"{spec.kind} rotates an even number of entries, got {p.dims}")
         if p.factor and p.factor != 1.0 and (p.factor < 0 or p.original <= 0 or p.fast <= 0 or p.slow <= 0 or p.base <= 1):
-            raise ValueError("rope_halves: a scaling needs positive factor, original, fast and slow and a base above 1")
+            raise ValueError(f"{spec.kind}: a scaling needs positive factor, original, fast and slow and a base above 1")
         n = max(min(p.max_positions, rt.max_seq_len) if rt.max_seq_len > 0 else p.max_positions, 1)
-        key = (p, n, str(rt.device))
-        if key not in _half_tables:
+        key = (p.dims, p.base, p.factor, p.original, p.fast, p.slow, n, str(rt.device))
+        if key not in _tables:
             freq, mag = yarn_frequencies(p)
             angle = np.arange(n, dtype=np.float64)[:, None] * np.asarray(freq, dtype=np.float64)[None, :]
-            _half_tables[key] = (torch.from_numpy((np.cos(angle) * mag).astype(np.float32)).to(rt.device),
-                                 torch.from_numpy((np.sin(angle) * mag).astype(np.float32)).to(rt.device))
-        self.cos, self.sin = _half_tables[key]
+            _tables[key] = (torch.from_numpy((np.cos(angle) * mag).astype(np.float32)).to(rt.device),
+                            torch.from_numpy((np.sin(angle) * mag).astype(np.float32)).to(rt.device))
+        self.cos, self.sin = _tables[key]
 
     def rotary_tables(self):
         return self.cos, self.sin
 
     def nbytes(self) -> int:
         return 2 * self.cos.numel() * 4
+
+
+@register("position", "rope_pairs")
+class RotaryPairs(PairTables):
+    """Entries (2i, 2i + 1), i < dims / 2, of a head turn together; the entries from ``dims`` on stay."""
+
+    pairing = "neighbours"
+
+
+@register("position", "rope_halves")
+class RotaryHalves(PairTables):
+    """Entry i < dims / 2 of a head turns with entry i + dims / 2; the entries from ``dims`` on stay."""
+
+    pairing = "halves"

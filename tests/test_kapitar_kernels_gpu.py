@@ -122,8 +122,9 @@ def test_linear_attention_from_a_state_serial_and_in_chunks(dtype, H, D, DV):
         out = torch.zeros(T, H * DV, device=DEV)
         chunk, max_chunks = (64, (max(lens) + 63) // 64) if chunked else (0, 1)
         scratch = torch.full((3 * max_chunks * H * D * DV,), float("nan"), device=DEV) if chunked else None
-        kernels.linear_attention(proj.to(DEV), 0, H * D, 2 * H * D, seq_of, slot_t, dec, state, out, T, 3, H, D, DV,
-                                 scratch, chunk, max_chunks)
+        dev = proj.to(DEV)
+        kernels.linear_attention(dev[:, :H * D], dev[:, H * D:2 * H * D], dev[:, 2 * H * D:2 * H * D + H * DV], seq_of, slot_t,
+                                 dec, state, out, T, 3, H, D, DV, scratch, chunk, max_chunks)
         assert rel(out, want_o) < (2e-5 if dtype == torch.float32 else 2e-5), chunked
         for s in range(6):
             if s in want_S:

@@ -69,8 +69,10 @@ def test_latent_between_projection_and_cache(dtype, tol, H, dn, dr, rank, rot):
     cache = torch.full((5, 1, ps, key), float("nan"), dtype=dtype, device=DEV)
     qa = torch.full((T, H * key), float("nan"), dtype=dtype, device=DEV)
     status = torch.zeros(1, dtype=torch.int32, device=DEV)
-    kernels.latent_prep(proj.to(DEV), pos.to(DEV), T, H, dn, dr, rank, rot, nw.to(DEV), eps, cos, sin, qa, slots.to(DEV), cache,
-                        ps, status)
+    dev = proj.to(DEV)
+    q_dev, lat_dev = dev[:, :H * (dn + dr)], dev[:, H * (dn + dr):]
+    kernels.latent_prep(q_dev, lat_dev, pos.to(DEV), T, H, dn, dr, rank, rot, nw.to(DEV), eps, cos, sin, qa, slots.to(DEV),
+                        cache, ps, status)
     assert int(status.item()) == 0
     p64 = proj.double()
     craw = p64[:, H * (dn + dr):]
@@ -89,7 +91,7 @@ def test_latent_between_projection_and_cache(dtype, tol, H, dn, dr, rank, rot):
     written[slots[slots >= 0].long()] = True
     assert torch.isnan(flat[~written]).all()
     if dr > 0:
-        kernels.latent_prep(proj.to(DEV), torch.full((T,), 500, dtype=torch.int32, device=DEV), T, H, dn, dr, rank, rot,
+        kernels.latent_prep(q_dev, lat_dev, torch.full((T,), 500, dtype=torch.int32, device=DEV), T, H, dn, dr, rank, rot,
                             nw.to(DEV), eps, cos, sin, qa, None, cache, ps, status)
         assert int(status.item()) == 2
 
