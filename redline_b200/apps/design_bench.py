@@ -1,5 +1,5 @@
 """Prefill and decode throughput of one architecture beside another at equal layer sizes, with the
-per-op roofline fractions of both (``bench.py --compare-design kapitar``, ``pufevik`` or ``vizotar``).
+per-op roofline fractions of both (``bench.py --compare-design kapitar``, ``pufevik``, ``vizotar``, ``venezen`` or ``lakatar``).
 
 Every size is a handful of layers whose matrices have the shapes of a real model's (random weights):
 the Kapitar model has one layer of every kind (attention + dense, lightning + routed, attention + routed,
@@ -29,6 +29,13 @@ it stands Kapitar, the closest architecture the package has (layer norms, attent
 over the same window with two score maps of half the key size, routed experts with a shared one; linear
 attention where Venezen attends over latents), at the same width, heads, kv heads, window and expert count;
 Venezen's gated feed-forwards have three matrices for Kapitar's two and are two thirds as wide.
+
+The Lakatar model has four layers, all with routed experts and a shared one: time mixing, attention over a cached
+latent, retention, attention over the other layer's latent.  Beside it stand Venezen, the closest architecture the
+package has (the same attention over latents of the same sizes, the same experts without groups; half of its
+feed-forwards are dense and as wide as Lakatar's chosen and shared experts together), and Vizotar for its
+recurrence (the delta rule with a decay per key channel, as many state entries per head as Lakatar's time mixing
+has in two heads), both at the same width.
 """
 
 from __future__ import annotations
@@ -66,6 +73,15 @@ VENEZEN_SIZES: Dict[str, Dict[str, int]] = {
               gated_shared_ff=768, identity=2),
     "m": dict(SIZES["m"], lat_dim=64, rot_dim=32, lat_vdim=64, kv_rank=192, gated_ff=5632, gated_expert_ff=704,
               gated_shared_ff=1408, identity=4),
+}
+LAKATAR_SIZES: Dict[str, Dict[str, int]] = {
+    # VENEZEN_SIZES' keys that the latent attention and the experts share, the time mixing's and the retention's heads
+    "s": dict(width=1024, heads=8, lat_dim=64, rot_dim=32, lat_vdim=64, kv_rank=192, q_rank=384, wkv_heads=16, wkv_dim=64,
+              decay_rank=64, ret_heads=4, ret_dim=128, ret_vdim=256, experts=16, top=4, expert_ff=384, shared_ff=768, groups=4,
+              keep=2, vocab=32000),
+    "m": dict(width=2048, heads=16, lat_dim=64, rot_dim=32, lat_vdim=64, kv_rank=192, q_rank=768, wkv_heads=32, wkv_dim=64,
+              decay_rank=64, ret_heads=8, ret_dim=128, ret_vdim=256, experts=32, top=4, expert_ff=704, shared_ff=1408, groups=4,
+              keep=2, vocab=32000),
 }
 WINDOW, KEEP_FIRST = 1024, 4
 PROMPT = 2048
@@ -141,11 +157,30 @@ def venezen_config(s: Dict[str, int]) -> Dict[str, Any]:
                        {"type": "latent_attention", "mixer": latent, "mlp": moe}, {"type": "attention", "mixer": windowed, "mlp": dense}]}
 
 
-# design -> (its sizes, its configuration, the architecture beside it, that one's configuration at the same sizes)
-DESIGNS = {"kapitar": (SIZES, kapitar_config, "llama", llama_config),
-           "pufevik": (PUFEVIK_SIZES, pufevik_config, "llama", llama_beside_pufevik),
-           "vizotar": (VIZOTAR_SIZES, vizotar_config, "pufevik", pufevik_config),
-           "venezen": (VENEZEN_SIZES, venezen_config, "kapitar", kapitar_config)}
+def lakatar_config(s: Dict[str, int]) -> Dict[str, Any]:
+    latent = {"heads": s["heads"], "dim": s["lat_dim"], "rot_dim": s["rot_dim"], "vdim": s["lat_vdim"], "kv_rank": s["kv_rank"],
+              "q_rank": s["q_rank"], "scale": (s["lat_dim"] + s["rot_dim"]) ** -0.5,
+              "rot": {"base": 500000.0, "dims": s["rot_dim"],
+                      "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    n = s["ret_heads"]
+    ret = {"heads": n, "dim": s["ret_dim"], "vdim": s["ret_vdim"], "rot": {"base": 10000.0, "dims": s["ret_dim"]},
+           "decay": [1.0 - 2.0 ** -(5 + 4 * h / max(n - 1, 1)) for h in range(n)]}
+    wkv = {"heads": s["wkv_heads"], "dim": s["wkv_dim"], "decay_rank": s["decay_rank"]}
+    moe = {"kind": "moe", "expert": {"ff": s["expert_ff"]}, "shared": {"ff": s["shared_ff"]},
+           "router": {"experts": s["experts"], "top": s["top"], "scale": 2.5, "groups": {"count": s["groups"], "keep": s["keep"]}}}
+    return {"architecture": "Lakatar", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "postln_alpha": 1.7,
+            "layers": [{"type": "wkv", "mixer": wkv, "mlp": moe}, {"type": "latent_attention", "mixer": latent, "mlp": moe},
+                       {"type": "retention", "mixer": ret, "mlp": moe},
+                       {"type": "latent_attention", "mixer": dict(latent, kv_from=1), "mlp": moe}]}
+
+
+# design -> (its sizes, its configuration, [(architecture beside it, that one's sizes, its configuration at them)])
+DESIGNS = {"kapitar": (SIZES, kapitar_config, [("llama", SIZES, llama_config)]),
+           "pufevik": (PUFEVIK_SIZES, pufevik_config, [("llama", PUFEVIK_SIZES, llama_beside_pufevik)]),
+           "vizotar": (VIZOTAR_SIZES, vizotar_config, [("pufevik", VIZOTAR_SIZES, pufevik_config)]),
+           "venezen": (VENEZEN_SIZES, venezen_config, [("kapitar", VENEZEN_SIZES, kapitar_config)]),
+           "lakatar": (LAKATAR_SIZES, lakatar_config, [("venezen", VENEZEN_SIZES, venezen_config),
+                                                       ("vizotar", VIZOTAR_SIZES, vizotar_config)])}
 
 
 def _prefill(model: str, tokens: int, reps: int, warmup: int) -> float:
@@ -244,8 +279,8 @@ def compare(design: str, sizes: List[str], steps: int, warmup: int, batch: int, 
     from ..weights import write_random_model
     if design not in DESIGNS:
         raise ValueError(f"no comparison is defined for '{design}' ({', '.join(DESIGNS)})")
-    table, design_config, beside, beside_config = DESIGNS[design]
-    out: Dict[str, Any] = {"design": design, "beside": beside, "prompt_tokens": PROMPT, "decode_batch": batch,
+    table, design_config, beside = DESIGNS[design]
+    out: Dict[str, Any] = {"design": design, "beside": beside[0][0] if len(beside) == 1 else [b[0] for b in beside], "prompt_tokens": PROMPT, "decode_batch": batch,
                            "decode_prompt": DECODE_PROMPT, "dtype": "bf16", "data": "synthetic (random weights and tokens)",
                            "sizes": {}}
     with tempfile.TemporaryDirectory() as tmp:
@@ -254,7 +289,7 @@ def compare(design: str, sizes: List[str], steps: int, warmup: int, batch: int, 
             entry: Dict[str, Any] = {"shape": dict(s, layers=4, window=WINDOW)}
             if design == "kapitar":
                 entry["shape"]["keep_first"] = KEEP_FIRST
-            for arch, cfg in ((design, design_config(s)), (beside, beside_config(s))):
+            for arch, cfg in [(design, design_config(s))] + [(b, conf(sizes_of[name])) for b, sizes_of, conf in beside]:
                 d = os.path.join(tmp, f"{arch}_{name}")
                 t0 = time.time()
                 write_random_model(d, config_from_dict(cfg), seed=0)

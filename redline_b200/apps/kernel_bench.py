@@ -8,6 +8,7 @@ package, if present).
     python -m redline_b200.apps.kernel_bench gemm_tc --rows 2048 --n 8192 --k 2048 --epilogue swiglu [--library]
     python -m redline_b200.apps.kernel_bench head_linear --tokens 2048 --heads 16 --n 192 --k 64 [--impl 1]
     python -m redline_b200.apps.kernel_bench latent_attn --tokens 2048 --heads 16 --rank 192 --rot 32 [--impl 1]
+    python -m redline_b200.apps.kernel_bench recurrence --tokens 2048 --heads 32 --head-dim 64 --vdim 64 [--channel] [--seqs 1]
 
 Each kernel runs over several distinct copies of its large operands (more than the
 L2 holds), captured in a CUDA graph so that launch overhead of the host is not
@@ -277,10 +278,57 @@ def bench_latent_attn(args) -> None:
                       "frac_of_measured_bf16": round(flops / us / 1e6 / pk["bf16_tflops"], 4)}))
 
 
+def bench_recurrence(args) -> None:
+    """Linear attention's recurrence over sequences of equal length, cut as the engine cuts them: one decay per head
+    with rotated queries and keys (float32 sums out), or (--channel) a decay per token and channel with a bonus and
+    the heads finished by the kernel."""
+    dev = "cuda"
+    T, H, D, DV, S = args.tokens, args.heads, args.head_dim, args.vdim, args.seqs
+    per = T // S
+    T = per * S
+    copies = max(2, min(args.copies, int(2e9 // (T * H * (2 * D + 3 * DV) * 4))))
+    bf = torch.bfloat16
+    q, k = ([torch.randn(T, H * D, device=dev).to(bf) for _ in range(copies)] for _ in range(2))
+    v, g = ([torch.randn(T, H * DV, device=dev).to(bf) for _ in range(copies)] for _ in range(2))
+    seq = (torch.arange(T, dtype=torch.int32) // per).to(dev)
+    slot = torch.arange(S, dtype=torch.int32, device=dev)
+    state = torch.zeros(S, H * D * DV, device=dev)
+    o = torch.empty(T, H * DV, device=dev)
+    y = torch.empty(T, H * DV, device=dev, dtype=bf)
+    chunk, chunks = kernels.linear_attention_chunks(per, blocks=args.impl == 0 and D % 16 == 0 and DV % 16 == 0)
+    if args.chunk:
+        chunk, chunks = args.chunk, (per + args.chunk - 1) // args.chunk
+    kw = dict(chunk=chunk, max_chunks=chunks, longest=0 if args.impl == 1 else per, status=torch.zeros(1, dtype=torch.int32, device=dev))
+    if chunks > 1:
+        kw.update(chunk_state=torch.empty(S * chunks * H * D * DV, device=dev), chunk_decay=torch.empty(S * chunks * H * D, device=dev))
+    if args.channel:
+        z = [torch.randn(T, H * D, device=dev) - 3.0 for _ in range(copies)]
+        kw.update(decay_bias=torch.zeros(H * D, device=dev), bonus=torch.randn(H * D, device=dev))
+    else:
+        z = [torch.full((H,), 0.98, device=dev)] * copies
+        ang = torch.arange(per + 1, device=dev)[:, None] * 0.01 * torch.arange(D // 2, device=dev)[None, :]
+        kw.update(cos=torch.cos(ang).contiguous(), sin=torch.sin(ang).contiguous(),
+                  positions=(torch.arange(T, dtype=torch.int32, device=dev) % per).contiguous())
+
+    def fn(i):
+        i %= copies
+        done = {} if args.sums else dict(y=y, gate=g[i], gate_mode=kernels.GATE_SILU, eps=1e-6)
+        kernels.linear_attention(q[i], k[i], v[i], seq, slot, z[i], state, o, T, S, H, D, DV, **done, **kw)
+
+    us = graph_time_us(fn, copies, use_graph=not args.no_graph)
+    nbytes = T * H * (2 * D + 3 * DV) * 2.0 + (T * H * D * 4.0 if args.channel else 0.0) + 2.0 * state.numel() * 4
+    flops = (6.0 if args.channel else 4.0) * T * H * D * DV
+    pk = peaks()
+    print(json.dumps({"kernel": "recurrence", "channel": bool(args.channel), "tokens": T, "seqs": S, "heads": H, "dim": D,
+                      "vdim": DV, "chunk": chunk, "us": round(us, 2), "GB/s": round(nbytes / us / 1e3, 1),
+                      "TFLOP/s": round(flops / us / 1e6, 2), "frac_of_measured_hbm": round(nbytes / us / 1e3 / pk["hbm_gbs"], 3),
+                      "copies": copies}))
+
+
 def main() -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     sub = ap.add_subparsers(dest="kernel", required=True)
-    for name in ("attn_decode", "attn_prefill", "skinny", "gemm_tc", "gemm_mid", "head_linear", "latent_attn"):
+    for name in ("attn_decode", "attn_prefill", "skinny", "gemm_tc", "gemm_mid", "head_linear", "latent_attn", "recurrence"):
         p = sub.add_parser(name)
         p.add_argument("--heads", type=int, default=32)
         p.add_argument("--kv-heads", type=int, default=8)
@@ -300,6 +348,14 @@ def main() -> int:
             p.add_argument("--k", type=int, default=64, help="head_linear: inputs of a head")
             p.add_argument("--rank", type=int, default=192, help="latent_attn: size of the cached latent")
             p.add_argument("--rot", type=int, default=32, help="latent_attn: size of the rotated key part")
+        if name == "recurrence":
+            p.add_argument("--tokens", type=int, default=2048)
+            p.add_argument("--vdim", type=int, default=64)
+            p.add_argument("--seqs", type=int, default=1, help="sequences of equal length (tokens in all)")
+            p.add_argument("--impl", type=int, default=0, help="0 auto, 1 CUDA cores, token by token")
+            p.add_argument("--chunk", type=int, default=0, help="tokens of a chunk (default: as the engine cuts)")
+            p.add_argument("--sums", action="store_true", help="float32 sums instead of finished heads")
+            p.add_argument("--channel", action="store_true", help="a decay per token and key channel, with a bonus")
         if name == "attn_prefill":
             p.add_argument("--tokens", type=int, default=2048)
             p.add_argument("--impl", type=int, default=0, help="0 auto, 1 CUDA cores, 2 mma.sync kernel, 3 tcgen05 kernel")
@@ -334,7 +390,7 @@ def main() -> int:
         return 1
     {"attn_decode": bench_attn_decode, "attn_prefill": bench_attn_prefill, "skinny": bench_skinny,
      "gemm_tc": bench_gemm_tc, "gemm_mid": bench_gemm_mid, "head_linear": bench_head_linear,
-     "latent_attn": bench_latent_attn}[args.kernel](args)
+     "latent_attn": bench_latent_attn, "recurrence": bench_recurrence}[args.kernel](args)
     return 0
 
 

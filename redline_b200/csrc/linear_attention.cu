@@ -7,15 +7,18 @@
 //
 // (the second form's read-out sees the token's own write through the bonus u only).  One kernel serves prompt
 // portions and single tokens: a CTA takes one sequence of the step, one head and a block of value columns.
-// Columns of S never mix.  A thread keeps two neighbouring columns of a group of rows (up to 32) in
-// registers; the G = 2, 4 or 8 groups of a column lie in one warp and their partial read-outs meet by
-// shuffles.  The state is read from the request's slot at the start and written back at the end.
+// Columns of S never mix.  A thread keeps four neighbouring columns of a group of eight rows in registers, as
+// pairs of rows (fma.rn.f32x2: two rows per instruction, each rounded as a single fma); the G = 1 to 32 groups
+// of a column lie in one warp and their partial read-outs meet by shuffles that leave each lane with a column
+// of its own.  The state is read from the request's slot at the start and written back at the end.
 //
-// q, k and v are read in the activation type and staged a few tokens at a time in shared memory as float32,
-// where they may be
+// q, k, v, the gate (in the activation type), the decays' projections and the rotation's table rows of eight
+// tokens at a time are copied to shared memory asynchronously, into one of two buffers while the tokens of the
+// other are worked on; there q, k and v become float32 (every v twice in a row: an operand for two rows), and q
+// and k may be
 //   rotated   entry i of the first 2 * rot_pairs with entry i + rot_pairs, cosines and sines from tables,
 //   scaled    k by a constant,
-// and the decays are formed from their projections.  The state, the decays, the sums are float32.
+// and the decays are formed.  The state, the decays, the sums are float32.
 //
 // Output: float32 o; or, where one CTA covers all columns of a head, the finished heads right away:
 // y = o / sqrt(mean over the head (o^2) + eps) (* weight) (* act(gate)) in the activation type
@@ -36,15 +39,15 @@ namespace rl {
 
 constexpr int kD = RL_LIN_DIM;
 static_assert(kD >= 1 && kD <= 256, "key size out of range");
-constexpr int kGroups = kD <= 64 ? 2 : (kD <= 128 ? 4 : 8);            // row groups of a column
-constexpr int kRows = ((kD + kGroups - 1) / kGroups + 3) / 4 * 4;      // rows of a group (float4 loads)
+constexpr int kRows = 8;                                               // rows of a group
+constexpr int kGroups = kD <= 8 ? 1 : (kD <= 16 ? 2 : (kD <= 32 ? 4 : (kD <= 64 ? 8 : (kD <= 128 ? 16 : 32))));
 constexpr int kStride = kRows + 4;                                     // floats between groups in shared memory (spreads the banks)
 constexpr int kSm = kGroups * kStride;                                 // floats of one staged vector
-constexpr int kCols = 2;                                               // columns of a thread
-constexpr int kSlots = 32 / kGroups;                                   // column pairs of a warp
-constexpr int kTok = kD <= 64 ? 16 : 8;                                // tokens staged at a time
-constexpr int kMaxThreads = kGroups <= 2 ? 128 : 256;
-constexpr int kMaxCols = kMaxThreads / kGroups * kCols;
+constexpr int kCols = 4;                                               // columns of a thread
+constexpr int kSlots = 32 / kGroups;                                   // column quadruples of a warp
+constexpr int kTok = 8;                                                // tokens staged at a time
+constexpr int kMaxThreads = 256;
+constexpr int kTcMinTokens = 16, kTcMaxCols = 128;                     // blocks of tokens on the tensor cores: from so many on
 
 enum { GATE_NONE = 0, GATE_SIGMOID = 1, GATE_SILU = 2 };
 
@@ -63,7 +66,7 @@ struct LinArgs {
   const float* bonus;            // per channel: u [heads * D]
   float* state;                  // [slots] x [heads, D, DV]
   long long slot_stride;         // floats from one slot to the next
-  float* out;                    // [tokens, heads * DV], or null with y
+  float* out;                    // [tokens, heads * DV] float32 (with y: scratch)
   T* y;                          // the finished heads (one CTA per head's columns), or null
   int y_ld;
   const T* gate;
@@ -74,7 +77,8 @@ struct LinArgs {
   float* chunk_decay;            // per channel: [sequences, chunks, heads, D]
   int* status;
   int tokens, heads, dv, chunk, max_chunks;
-  int pairs_ok;                  // column pairs of the state start on 8-byte boundaries
+  int quads_ok;                  // column quadruples of the state start on 16-byte boundaries
+  int qk_ok, v_ok, g_ok, z_ok, rot_ok; // rows of q and k / values / gates / decays / tables are made of 16-byte pieces
 };
 
 // First token index t in [0, n] with seq_of_token[t] >= s (sequences lie in order in a step): all 32 lanes of
@@ -96,9 +100,67 @@ __device__ __forceinline__ int first_token_of(const int32_t* __restrict__ seq_of
 }
 
 __device__ __forceinline__ float gate_value(float g, int mode) {
-  const float s = 1.f / (1.f + expf(-g));
+  const float s = __fdividef(1.f, 1.f + __expf(-g));           // (0 where exp(-g) is infinite)
   return mode == GATE_SILU ? g * s : s;
 }
+// (the inner exponential's relative error is that of the distance of the decay from 1)
+__device__ __forceinline__ float channel_decay(float z) { return expf(-__expf(z)); }
+
+__device__ __forceinline__ void async_copy16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<unsigned>(__cvta_generic_to_shared(dst))), "l"(src));
+}
+__device__ __forceinline__ void async_copies_done() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
+// Two floats as one operand.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ void unpack2(f32x2 v, float& lo, float& hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
+// What one buffer of staged tokens holds, in bytes; every token's part starts on a 16-byte boundary.
+struct RawLayout {
+  int q, k, v, g, z, cs, sn, bytes;      // offsets of the parts within a buffer; a buffer's size
+  int qk_row, v_row, z_row, rot_row;     // bytes of a token in its part (values and gate: v_row)
+  int pairs, sums;                       // behind the two buffers: the values as operands, the read-outs; bytes of each
+};
+__host__ __device__ inline RawLayout raw_layout(int elem, int cols, int rot_pairs, bool channel, bool with_q, bool gated,
+                                                int finished_cols) {
+  RawLayout r;
+  r.qk_row = (kD * elem + 15) / 16 * 16;
+  r.v_row = (cols * elem + 15) / 16 * 16;
+  r.z_row = channel ? (kD * 4 + 15) / 16 * 16 : 0;
+  r.rot_row = (rot_pairs * 4 + 15) / 16 * 16;
+  r.q = 0;
+  r.k = with_q ? kTok * r.qk_row : 0;
+  r.v = r.k + kTok * r.qk_row;
+  r.g = r.v + kTok * r.v_row;
+  r.z = r.g + (gated ? kTok * r.v_row : 0);
+  r.cs = r.z + kTok * r.z_row;
+  r.sn = r.cs + kTok * r.rot_row;
+  r.bytes = r.sn + kTok * r.rot_row;
+  r.pairs = kTok * cols * 8;
+  r.sums = kTok * finished_cols * 4;
+  return r;
+}
+
+// A pair of neighbouring elements (the address is a multiple of the pair's size).
+__device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+__device__ __forceinline__ float2 load2(const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
 
 // mode 0: the whole sequence serially from the slot's state (state written back)
 // mode 1: chunk c from zero, no outputs; the chunk's state goes to chunk_state[seq][c]
@@ -106,16 +168,16 @@ __device__ __forceinline__ float gate_value(float g, int mode) {
 //         c - 1; for c = 0 the slot's state, which pass 2 has copied to the entry of the last chunk, since
 //         the last chunk's CTA overwrites the slot), outputs written; the last chunk writes the slot
 template <typename T, int MODE, bool CHANNEL>
-__global__ void __launch_bounds__(kMaxThreads, MODE == 0 ? 1 : 512 / kMaxThreads)
+__global__ void __launch_bounds__(kMaxThreads, 2)
 linear_attention_kernel(const LinArgs<T> a) {
   pdl_launch();
   pdl_wait();
   __shared__ __align__(16) float qs[MODE == 1 ? 1 : kTok][kSm];
   __shared__ __align__(16) float ks[kTok][kSm];
   __shared__ __align__(16) float as[CHANNEL ? kTok : 1][kSm];
-  __shared__ __align__(8) float vs[kTok][kMaxCols];
+  __shared__ __align__(8) float us[CHANNEL && MODE != 1 ? kD : 1], db[CHANNEL ? kD : 1];      // per channel: the head's bonus and decay bias
   __shared__ float bs[kTok];                       // per channel: sum_i q_i u_i k_i of every staged token
-  extern __shared__ float os[];                    // [kTok][DV] read-outs, where the heads are finished here
+  extern __shared__ __align__(16) unsigned char raw[];     // two buffers, the values, the read-outs (RawLayout)
   const int seq = blockIdx.z, head = blockIdx.y % a.heads, c = blockIdx.y / a.heads;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
   const int group = lane / kSlots;
@@ -123,7 +185,10 @@ linear_attention_kernel(const LinArgs<T> a) {
   const int col0 = blockIdx.x * block_cols;                               // the CTA's first column
   const int local = (warp * kSlots + lane % kSlots) * kCols;
   const int col = col0 + local;
-  const bool in0 = col < a.dv, in1 = col + 1 < a.dv;
+  const bool finish = MODE != 1 && a.y != nullptr, gated = finish && a.gate_mode != GATE_NONE;
+  const RawLayout lay = raw_layout(sizeof(T), block_cols, a.rot_pairs, CHANNEL, MODE != 1, gated, finish ? a.dv : 0);
+  float* vs = reinterpret_cast<float*>(raw + 2 * lay.bytes);              // [kTok][block_cols] values, each twice
+  float* os = vs + lay.pairs / 4;                                         // [kTok][DV] read-outs
   const int seq_begin = first_token_of(a.seq_of_token, a.tokens, seq);
   const int seq_end = first_token_of(a.seq_of_token, a.tokens, seq + 1);
   if (seq_begin >= seq_end) return;
@@ -135,15 +200,56 @@ linear_attention_kernel(const LinArgs<T> a) {
   }
   const bool last_chunk = t1 == seq_end;
   if (MODE == 1 && last_chunk) return;             // nobody starts from the state after the last chunk
+  int pos0 = 0;                                    // the position of token t0 (a sequence's positions are consecutive)
+  if (a.rot_pairs > 0) {
+    pos0 = a.positions[t0];
+    if (pos0 < 0 || pos0 + (t1 - t0) > a.max_pos) {
+      if (threadIdx.x == 0) atomicOr(a.status, 2);
+      pos0 = -1;                                   // every token then takes the tables' first row
+    }
+  }
+
+  // tokens tb .. tb + nt - 1 on their way into buffer b: a warp takes one token at a time, its lanes the pieces of
+  // the token's parts, one part after another
+  auto stage = [&](int b, int tb, int nt) {
+    constexpr int E = sizeof(T);
+    for (int tt = warp; tt < nt; tt += nwarps) {
+      unsigned char* buf = raw + b * lay.bytes;
+      const size_t t = tb + tt;
+      auto part = [&](unsigned char* to, const void* from, int bytes, bool pieces, int elem) {
+        if (pieces) {
+          for (int e = lane; e < bytes / 16; e += 32) async_copy16(to + e * 16, static_cast<const unsigned char*>(from) + e * 16);
+        } else if (elem == 4) {
+          for (int e = lane; e < bytes / 4; e += 32) reinterpret_cast<float*>(to)[e] = static_cast<const float*>(from)[e];
+        } else {
+          for (int e = lane; e < bytes / 2; e += 32) reinterpret_cast<bf16*>(to)[e] = static_cast<const bf16*>(from)[e];
+        }
+      };
+      if (MODE != 1) part(buf + lay.q + tt * lay.qk_row, a.q + t * a.q_ld + head * kD, kD * E, a.qk_ok, E);
+      part(buf + lay.k + tt * lay.qk_row, a.k + t * a.k_ld + head * kD, kD * E, a.qk_ok, E);
+      const int cols = min(block_cols, a.dv - col0);
+      part(buf + lay.v + tt * lay.v_row, a.v + t * a.v_ld + head * a.dv + col0, cols * E, a.v_ok, E);
+      if (gated) part(buf + lay.g + tt * lay.v_row, a.gate + t * a.gate_ld + head * a.dv, a.dv * E, a.g_ok, E);
+      if (CHANNEL) part(buf + lay.z + tt * lay.z_row, a.decay + (t * a.heads + head) * kD, kD * 4, a.z_ok, 4);
+      if (a.rot_pairs > 0) {
+        const size_t at = pos0 < 0 ? 0 : static_cast<size_t>(pos0 + tb + tt - t0) * a.rot_pairs;
+        part(buf + lay.cs + tt * lay.rot_row, a.cos_t + at, a.rot_pairs * 4, a.rot_ok, 4);
+        part(buf + lay.sn + tt * lay.rot_row, a.sin_t + at, a.rot_pairs * 4, a.rot_ok, 4);
+      }
+    }
+  };
+  stage(0, t0, min(kTok, t1 - t0));
+
   const size_t plane = static_cast<size_t>(kD) * a.dv;
   float* slot_state = a.state + static_cast<size_t>(a.state_slot[seq]) * a.slot_stride + head * plane;
   float* chunk_state = MODE == 0 ? nullptr
       : a.chunk_state + ((static_cast<size_t>(seq) * a.max_chunks + c) * a.heads + head) * plane;
-
-  float S[kRows][kCols];
+  f32x2 S[kRows / 2][kCols];                       // rows 2i and 2i + 1 of the group
   if (MODE == 1) {
 #pragma unroll
-    for (int i = 0; i < kRows; ++i) S[i][0] = S[i][1] = 0.f;
+    for (int i = 0; i < kRows / 2; ++i)
+#pragma unroll
+      for (int j = 0; j < kCols; ++j) S[i][j] = 0;
   } else {
     const float* from = slot_state;
     if (MODE == 3 && c > 0) from = chunk_state - static_cast<size_t>(a.heads) * plane;
@@ -152,17 +258,23 @@ linear_attention_kernel(const LinArgs<T> a) {
       from = chunk_state + static_cast<size_t>(chunks - 1) * a.heads * plane;
     }
 #pragma unroll
-    for (int i = 0; i < kRows; ++i) {
-      const int row = group * kRows + i;
-      const float* p = from + static_cast<size_t>(row) * a.dv + col;
-      if (a.pairs_ok) {
-        const float2 s = (in0 && row < kD) ? *reinterpret_cast<const float2*>(p) : make_float2(0.f, 0.f);
-        S[i][0] = s.x;
-        S[i][1] = s.y;
-      } else {
-        S[i][0] = (in0 && row < kD) ? p[0] : 0.f;
-        S[i][1] = (in1 && row < kD) ? p[1] : 0.f;
+    for (int i = 0; i < kRows / 2; ++i) {
+      float v[2][kCols];
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int row = group * kRows + 2 * i + h;
+        const float* p = from + static_cast<size_t>(row) * a.dv + col;
+        const bool in = row < kD && col < a.dv;
+        if (a.quads_ok) {
+          const float4 s = in ? *reinterpret_cast<const float4*>(p) : make_float4(0.f, 0.f, 0.f, 0.f);
+          v[h][0] = s.x; v[h][1] = s.y; v[h][2] = s.z; v[h][3] = s.w;
+        } else {
+#pragma unroll
+          for (int j = 0; j < kCols; ++j) v[h][j] = (in && col + j < a.dv) ? p[j] : 0.f;
+        }
       }
+#pragma unroll
+      for (int j = 0; j < kCols; ++j) S[i][j] = pack2(v[0][j], v[1][j]);
     }
   }
   if (kGroups * kRows > kD) {                      // rows beyond D: zero keys and queries, never written again
@@ -173,146 +285,195 @@ linear_attention_kernel(const LinArgs<T> a) {
     }
   }
   const float decay = CHANNEL ? 0.f : a.decay[head];
-  float prod[(kD + 31) / 32];                      // MODE 1, per channel: thread d of warp 0 .. its channels' products
+  const f32x2 decay2 = pack2(decay, decay);
+  constexpr int kPer = (kD + 31) / 32;             // channels of a lane
+  float prod[CHANNEL && MODE == 1 ? kPer : 1];     // per channel, mode 1, warp 0: the products of its channels' decays
+  if (CHANNEL) {
+    for (int d = threadIdx.x; d < kD; d += blockDim.x) {
+      db[d] = a.decay_bias[head * kD + d];
+      if (MODE != 1) us[d] = a.bonus[head * kD + d];
+    }
+    if (MODE == 1) {
 #pragma unroll
-  for (int i = 0; i < (kD + 31) / 32; ++i) prod[i] = 1.f;
+      for (int j = 0; j < kPer; ++j) prod[j] = 1.f;
+    }
+  }
 
-  for (int tb = t0; tb < t1; tb += kTok) {
+  int b = 0;
+  for (int tb = t0; tb < t1; tb += kTok, b ^= 1) {
     const int nt = min(kTok, t1 - tb);
-    __syncthreads();
-    // ---- a warp stages one token at a time, its lanes over the channels
+    async_copies_done();
+    __syncthreads();               // this batch has arrived, and the one before has been worked on
+    if (tb + kTok < t1) stage(b ^ 1, tb + kTok, min(kTok, t1 - tb - kTok));
+    const unsigned char* buf = raw + b * lay.bytes;
+    // ---- a warp readies one token at a time, its lanes over the channels (two neighbours each where sizes are even)
     for (int tt = warp; tt < nt; tt += nwarps) {
-      const size_t t = tb + tt;
-      const T* qr = a.q + t * a.q_ld + head * kD;
-      const T* kr = a.k + t * a.k_ld + head * kD;
-      const float *cs = nullptr, *sn = nullptr;
-      if (a.rot_pairs > 0) {
-        int pos = a.positions[t];
-        if (pos < 0 || pos >= a.max_pos) {
-          if (lane == 0) atomicOr(a.status, 2);
-          pos = 0;
-        }
-        cs = a.cos_t + static_cast<size_t>(pos) * a.rot_pairs;
-        sn = a.sin_t + static_cast<size_t>(pos) * a.rot_pairs;
-      }
+      const T* qr = reinterpret_cast<const T*>(buf + lay.q + tt * lay.qk_row);
+      const T* kr = reinterpret_cast<const T*>(buf + lay.k + tt * lay.qk_row);
+      const float* zr = reinterpret_cast<const float*>(buf + lay.z + tt * lay.z_row);
+      const float* cs = reinterpret_cast<const float*>(buf + lay.cs + tt * lay.rot_row);
+      const float* sn = reinterpret_cast<const float*>(buf + lay.sn + tt * lay.rot_row);
       float bonus = 0.f;
+      if (kD % 2 == 0 && a.rot_pairs % 2 == 0) {
 #pragma unroll
-      for (int j = 0; j < (kD + 31) / 32; ++j) {
-        const int d = j * 32 + lane;
-        if (d >= kD) continue;
-        const int sm = (d / kRows) * kStride + d % kRows;
-        float qv = MODE == 1 ? 0.f : to_float(qr[d]), kv = to_float(kr[d]);
-        if (d < 2 * a.rot_pairs) {
-          const bool first = d < a.rot_pairs;
-          const int pair = first ? d : d - a.rot_pairs, other = first ? d + a.rot_pairs : pair;
-          const float cv = cs[pair], sv = first ? -sn[pair] : sn[pair];
-          kv = kv * cv + to_float(kr[other]) * sv;
-          if (MODE != 1) qv = qv * cv + to_float(qr[other]) * sv;
+        for (int j = 0; j < (kD + 63) / 64; ++j) {
+          const int d = j * 64 + 2 * lane;
+          if (d >= kD) continue;
+          const int sm = (d / kRows) * kStride + d % kRows;
+          float2 kv = load2(kr + d), qv = make_float2(0.f, 0.f);
+          if (MODE != 1) qv = load2(qr + d);
+          if (d < 2 * a.rot_pairs) {
+            const bool first = d < a.rot_pairs;
+            const int pair = first ? d : d - a.rot_pairs, other = first ? d + a.rot_pairs : pair;
+            const float2 cv = load2(cs + pair);
+            float2 sv = load2(sn + pair);
+            if (first) sv = make_float2(-sv.x, -sv.y);
+            const float2 ko = load2(kr + other);
+            kv = make_float2(kv.x * cv.x + ko.x * sv.x, kv.y * cv.y + ko.y * sv.y);
+            if (MODE != 1) {
+              const float2 qo = load2(qr + other);
+              qv = make_float2(qv.x * cv.x + qo.x * sv.x, qv.y * cv.y + qo.y * sv.y);
+            }
+          }
+          kv = make_float2(kv.x * a.k_scale, kv.y * a.k_scale);
+          *reinterpret_cast<float2*>(&ks[tt][sm]) = kv;
+          if (MODE != 1) *reinterpret_cast<float2*>(&qs[tt][sm]) = qv;
+          if (CHANNEL) {
+            const float2 z = load2(zr + d), bias = load2(db + d);
+            *reinterpret_cast<float2*>(&as[tt][sm]) = make_float2(channel_decay(z.x + bias.x), channel_decay(z.y + bias.y));
+            if (MODE != 1) {
+              const float2 u = load2(us + d);
+              bonus = fmaf(qv.x * u.x, kv.x, fmaf(qv.y * u.y, kv.y, bonus));
+            }
+          }
         }
-        kv *= a.k_scale;
-        ks[tt][sm] = kv;
-        if (MODE != 1) qs[tt][sm] = qv;
-        if (CHANNEL) {
-          const int ch = head * kD + d;
-          as[tt][sm] = expf(-expf(a.decay[t * (a.heads * kD) + ch] + a.decay_bias[ch]));
-          if (MODE != 1) bonus = fmaf(qv * a.bonus[ch], kv, bonus);
+      } else {
+        for (int d = lane; d < kD; d += 32) {
+          const int sm = (d / kRows) * kStride + d % kRows;
+          float qv = MODE == 1 ? 0.f : to_float(qr[d]), kv = to_float(kr[d]);
+          if (d < 2 * a.rot_pairs) {
+            const bool first = d < a.rot_pairs;
+            const int pair = first ? d : d - a.rot_pairs, other = first ? d + a.rot_pairs : pair;
+            const float cv = cs[pair], sv = first ? -sn[pair] : sn[pair];
+            kv = kv * cv + to_float(kr[other]) * sv;
+            if (MODE != 1) qv = qv * cv + to_float(qr[other]) * sv;
+          }
+          kv *= a.k_scale;
+          ks[tt][sm] = kv;
+          if (MODE != 1) qs[tt][sm] = qv;
+          if (CHANNEL) {
+            as[tt][sm] = channel_decay(zr[d] + db[d]);
+            if (MODE != 1) bonus = fmaf(qv * us[d], kv, bonus);
+          }
         }
       }
       if (CHANNEL && MODE != 1) {
         bonus = warp_sum(bonus);
         if (lane == 0) bs[tt] = bonus;
       }
-      const T* vr = a.v + t * a.v_ld + head * a.dv + col0;
-      for (int i = lane; i < block_cols; i += 32) vs[tt][i] = col0 + i < a.dv ? to_float(vr[i]) : 0.f;
+      const T* vr = reinterpret_cast<const T*>(buf + lay.v + tt * lay.v_row);
+      for (int i = 2 * lane; i < block_cols; i += 64) {
+        const float2 v = load2(vr + i);
+        *reinterpret_cast<float4*>(vs + (tt * block_cols + i) * 2) = make_float4(v.x, v.x, v.y, v.y);
+      }
     }
     __syncthreads();
     if (CHANNEL && MODE == 1 && blockIdx.x == 0 && warp == 0) {
       for (int tt = 0; tt < nt; ++tt)
 #pragma unroll
-        for (int j = 0; j < (kD + 31) / 32; ++j) {
+        for (int j = 0; j < kPer; ++j) {
           const int d = j * 32 + lane;
           if (d < kD) prod[j] *= as[tt][(d / kRows) * kStride + d % kRows];
         }
     }
     auto token = [&](int tt) {
-      const float4* k4 = reinterpret_cast<const float4*>(&ks[tt][group * kStride]);
-      const float4* q4 = reinterpret_cast<const float4*>(&qs[MODE == 1 ? 0 : tt][group * kStride]);
-      const float4* a4 = reinterpret_cast<const float4*>(&as[CHANNEL ? tt : 0][group * kStride]);
-      const float2 v = *reinterpret_cast<const float2*>(&vs[tt][local]);
-      float o00 = 0.f, o01 = 0.f, o10 = 0.f, o11 = 0.f;       // two chains per column
+      const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(&ks[tt][group * kStride]);
+      const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(&qs[MODE == 1 ? 0 : tt][group * kStride]);
+      const ulonglong2* a4 = reinterpret_cast<const ulonglong2*>(&as[CHANNEL ? tt : 0][group * kStride]);
+      const ulonglong2* v4 = reinterpret_cast<const ulonglong2*>(vs + (tt * block_cols + local) * 2);
+      const ulonglong2 va = v4[0], vb = v4[1];
+      const f32x2 v2[kCols] = {va.x, va.y, vb.x, vb.y};
+      f32x2 o2[kCols];
+      // (the bonus counts once: in the first half of the first group's pairs)
+      const f32x2 bonus = pack2((CHANNEL && MODE != 1 && group == 0) ? bs[tt] : 0.f, 0.f);
 #pragma unroll
-      for (int i = 0; i < kRows; i += 4) {
-        const float4 kv = k4[i >> 2];
-        const float kk[4] = {kv.x, kv.y, kv.z, kv.w};
-        float qq[4] = {0.f, 0.f, 0.f, 0.f}, aa[4];
-        if (MODE != 1) {
-          const float4 qv = q4[i >> 2];
-          qq[0] = qv.x; qq[1] = qv.y; qq[2] = qv.z; qq[3] = qv.w;
-        }
-        if (CHANNEL) {
-          const float4 av = a4[i >> 2];
-          aa[0] = av.x; aa[1] = av.y; aa[2] = av.z; aa[3] = av.w;
-        }
+      for (int j = 0; j < kCols; ++j) o2[j] = CHANNEL && MODE != 1 ? mul2(bonus, v2[j]) : 0;
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          float &s0 = S[i + j][0], &s1 = S[i + j][1];
-          if (CHANNEL) {
-            if (MODE != 1) {
-              if (j & 1) { o01 = fmaf(s0, qq[j], o01); o11 = fmaf(s1, qq[j], o11); }
-              else       { o00 = fmaf(s0, qq[j], o00); o10 = fmaf(s1, qq[j], o10); }
-            }
-            s0 = fmaf(aa[j], s0, kk[j] * v.x);
-            s1 = fmaf(aa[j], s1, kk[j] * v.y);
-          } else {
-            s0 = fmaf(decay, s0, kk[j] * v.x);
-            s1 = fmaf(decay, s1, kk[j] * v.y);
-            if (MODE != 1) {
-              if (j & 1) { o01 = fmaf(s0, qq[j], o01); o11 = fmaf(s1, qq[j], o11); }
-              else       { o00 = fmaf(s0, qq[j], o00); o10 = fmaf(s1, qq[j], o10); }
-            }
+      for (int i = 0; i < kRows / 4; ++i) {
+        const ulonglong2 kv = k4[i];
+        ulonglong2 qv = make_ulonglong2(0, 0), av = make_ulonglong2(decay2, decay2);
+        if (MODE != 1) qv = q4[i];
+        if (CHANNEL) av = a4[i];
+#pragma unroll
+        for (int j = 0; j < kCols; ++j) {
+          f32x2 &s0 = S[2 * i][j], &s1 = S[2 * i + 1][j];
+          if (CHANNEL && MODE != 1) {
+            o2[j] = fma2(s0, qv.x, o2[j]);
+            o2[j] = fma2(s1, qv.y, o2[j]);
+          }
+          s0 = fma2(av.x, s0, mul2(kv.x, v2[j]));
+          s1 = fma2(av.y, s1, mul2(kv.y, v2[j]));
+          if (!CHANNEL && MODE != 1) {
+            o2[j] = fma2(s0, qv.x, o2[j]);
+            o2[j] = fma2(s1, qv.y, o2[j]);
           }
         }
       }
-      if (MODE != 1) {
-        float o0 = o00 + o01, o1 = o10 + o11;
+      if (MODE == 1) return;
+      float o[kCols];
 #pragma unroll
-        for (int off = kSlots; off < 32; off <<= 1) {
-          o0 += __shfl_xor_sync(0xffffffffu, o0, off);
-          o1 += __shfl_xor_sync(0xffffffffu, o1, off);
-        }
-        if (CHANNEL) {
-          o0 = fmaf(bs[tt], v.x, o0);
-          o1 = fmaf(bs[tt], v.y, o1);
-        }
-        if (group == 0) {
-          float* dst = a.y != nullptr ? os + tt * a.dv + col
-                                      : a.out + static_cast<size_t>(tb + tt) * (a.heads * a.dv) + head * a.dv + col;
-          if (in0) dst[0] = o0;
-          if (in1) dst[1] = o1;
-        }
+      for (int j = 0; j < kCols; ++j) {
+        float lo, hi;
+        unpack2(o2[j], lo, hi);
+        o[j] = lo + hi;
+      }
+      // the groups' partial sums: lanes of two groups exchange the columns the other one keeps
+      int keep = 0;
+      constexpr int n = kGroups >= 4 ? 1 : (kGroups == 2 ? 2 : kCols);      // columns a lane is left with
+      if (kGroups >= 2) {
+        const bool up = lane & 16;
+        const float r0 = __shfl_xor_sync(0xffffffffu, up ? o[0] : o[2], 16);
+        const float r1 = __shfl_xor_sync(0xffffffffu, up ? o[1] : o[3], 16);
+        o[0] = (up ? o[2] : o[0]) + r0;
+        o[1] = (up ? o[3] : o[1]) + r1;
+        keep = up ? 2 : 0;
+      }
+      if (kGroups >= 4) {
+        const bool up = lane & 8;
+        const float r0 = __shfl_xor_sync(0xffffffffu, up ? o[0] : o[1], 8);
+        o[0] = (up ? o[1] : o[0]) + r0;
+        keep += up ? 1 : 0;
+      }
+      if (kSlots <= 4) o[0] += __shfl_xor_sync(0xffffffffu, o[0], 4);
+      if (kSlots <= 2) o[0] += __shfl_xor_sync(0xffffffffu, o[0], 2);
+      if (kSlots <= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], 1);
+      if (kSlots <= 4 && (lane & (8 - kSlots))) return;            // (one lane of those with equal sums writes)
+#pragma unroll
+      for (int j = 0; j < n; ++j) {
+        if (col + keep + j >= a.dv) continue;
+        if (finish) os[tt * a.dv + col + keep + j] = o[j];
+        else a.out[static_cast<size_t>(tb + tt) * (a.heads * a.dv) + head * a.dv + col + keep + j] = o[j];
       }
     };
-    if (nt == kTok) {
-#pragma unroll 2
-      for (int tt = 0; tt < kTok; ++tt) token(tt);
-    } else {
-      for (int tt = 0; tt < nt; ++tt) token(tt);
-    }
-    if (MODE != 1 && a.y != nullptr) {
+#pragma unroll 1
+    for (int tt = 0; tt < nt; ++tt) token(tt);
+    if (finish) {
       // ---- the staged tokens' heads are complete: unit norm, weight, gate
       __syncthreads();
       for (int tt = warp; tt < nt; tt += nwarps) {
         const float* o = os + tt * a.dv;
+        const T* gr = reinterpret_cast<const T*>(buf + lay.g + tt * lay.v_row);
+        const size_t t = tb + tt;
         float ss = 0.f;
         for (int d = lane; d < a.dv; d += 32) ss = fmaf(o[d], o[d], ss);
         const float r = rsqrtf(warp_sum(ss) / static_cast<float>(a.dv) + a.eps);
-        const size_t t = tb + tt;
+        T* yr = a.y + t * a.y_ld + head * a.dv;
+        const float* w = a.norm_w != nullptr ? a.norm_w + head * a.dv : nullptr;
         for (int d = lane; d < a.dv; d += 32) {
-          const int e = head * a.dv + d;
           float y = o[d] * r;
-          if (a.norm_w != nullptr) y *= a.norm_w[e];
-          if (a.gate_mode != GATE_NONE) y *= gate_value(to_float(a.gate[t * a.gate_ld + e]), a.gate_mode);
-          a.y[t * a.y_ld + e] = from_float<T>(y);
+          if (w != nullptr) y *= w[d];
+          if (gated) y *= gate_value(to_float(gr[d]), a.gate_mode);
+          yr[d] = from_float<T>(y);
         }
       }
     }
@@ -320,25 +481,40 @@ linear_attention_kernel(const LinArgs<T> a) {
   if (CHANNEL && MODE == 1 && blockIdx.x == 0 && warp == 0) {
     float* cd = a.chunk_decay + ((static_cast<size_t>(seq) * a.max_chunks + c) * a.heads + head) * kD;
 #pragma unroll
-    for (int j = 0; j < (kD + 31) / 32; ++j)
+    for (int j = 0; j < kPer; ++j)
       if (j * 32 + lane < kD) cd[j * 32 + lane] = prod[j];
   }
   float* to = MODE == 1 ? chunk_state : ((MODE == 0 || last_chunk) ? slot_state : nullptr);
   if (to != nullptr) {
 #pragma unroll
-    for (int i = 0; i < kRows; ++i) {
-      const int row = group * kRows + i;
-      if (row >= kD) continue;
-      float* p = to + static_cast<size_t>(row) * a.dv + col;
-      if (a.pairs_ok) {
-        if (in0) *reinterpret_cast<float2*>(p) = make_float2(S[i][0], S[i][1]);
-      } else {
-        if (in0) p[0] = S[i][0];
-        if (in1) p[1] = S[i][1];
+    for (int i = 0; i < kRows / 2; ++i) {
+      float v[2][kCols];
+#pragma unroll
+      for (int j = 0; j < kCols; ++j) unpack2(S[i][j], v[0][j], v[1][j]);
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int row = group * kRows + 2 * i + h;
+        if (row >= kD || col >= a.dv) continue;
+        float* p = to + static_cast<size_t>(row) * a.dv + col;
+        if (a.quads_ok) {
+          *reinterpret_cast<float4*>(p) = make_float4(v[h][0], v[h][1], v[h][2], v[h][3]);
+        } else {
+#pragma unroll
+          for (int j = 0; j < kCols; ++j)
+            if (col + j < a.dv) p[j] = v[h][j];
+        }
       }
     }
   }
 }
+
+}  // namespace rl
+
+#if RL_LIN_DIM % 16 == 0
+#include "linear_attention_tc.cuh"
+#endif
+
+namespace rl {
 
 // Pass 2: chunk_state[seq][c] <- A_c * (state after chunk c - 1) + chunk_state[seq][c], in order of c; A_c is the
 // product of chunk c's decays (every chunk before the last is full).  One thread per element of a head's state.
@@ -412,32 +588,97 @@ __global__ void linear_output_kernel(const float* __restrict__ o, const T* __res
   }
 }
 
+inline bool on16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
 // Threads of a CTA for a head of dv columns.
 inline int lin_threads(int dv) {
   const int need = (dv + kCols - 1) / kCols * kGroups;
   return need >= kMaxThreads ? kMaxThreads : (need + 31) / 32 * 32;
 }
 
-template <typename T, bool CHANNEL>
-int launch_linear_attention(const LinArgs<T>& a, int sequences, cudaStream_t stream) {
+template <typename T, int MODE, bool CHANNEL>
+cudaError_t launch_pass(const LinArgs<T>& a, dim3 grid, int th, cudaStream_t stream) {
+  const int cols = th / 32 * kSlots * kCols;
+  const bool finish = MODE != 1 && a.y != nullptr;
+  const RawLayout lay = raw_layout(sizeof(T), cols, a.rot_pairs, CHANNEL, MODE != 1, finish && a.gate_mode != GATE_NONE,
+                                   finish ? a.dv : 0);
+  const size_t smem = 2 * static_cast<size_t>(lay.bytes) + lay.pairs + lay.sums;
+  static size_t set_for = 0;
+  if (smem > set_for) {                  // (the kernel also has static shared memory: beyond 48 KB in all the limit must be raised)
+    const cudaError_t e = cudaFuncSetAttribute(linear_attention_kernel<T, MODE, CHANNEL>,
+                                               cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return e;
+    set_for = smem;
+  }
+  return launch_kernel(linear_attention_kernel<T, MODE, CHANNEL>, grid, dim3(th), smem, stream, a);
+}
+
+#if RL_LIN_DIM % 16 == 0
+inline int tc_warps(int dv) { return min(kTcMaxWarps, dv / 16); }
+
+template <typename T, int MODE, bool CHANNEL>
+cudaError_t launch_tc_pass(const LinArgs<bf16>& a, dim3 grid, int warps, cudaStream_t stream) {
+  const bool finish = MODE != 1 && a.y != nullptr;
+  const TcLayout lay = tc_layout(warps * 16, a.rot_pairs, CHANNEL, MODE != 1, finish && a.gate_mode != GATE_NONE, finish);
+  static int set_for = 0;
+  if (lay.bytes > set_for) {
+    const cudaError_t e = cudaFuncSetAttribute(linear_attention_tc_kernel<MODE, CHANNEL>,
+                                               cudaFuncAttributeMaxDynamicSharedMemorySize, lay.bytes);
+    if (e != cudaSuccess) return e;
+    set_for = lay.bytes;
+  }
+  return launch_kernel(linear_attention_tc_kernel<MODE, CHANNEL>, grid, dim3(warps * 32), lay.bytes, stream, a);
+}
+#endif
+
+// One pass of the recurrence in the form that fits: blocks of tokens on the tensor cores, or token by token.
+template <typename T, int MODE, bool CHANNEL>
+cudaError_t launch_either(const LinArgs<T>& a, int rows, int sequences, bool tc, cudaStream_t stream) {
+#if RL_LIN_DIM % 16 == 0
+  if constexpr (sizeof(T) == 2) {
+    if (tc) {
+      const int warps = tc_warps(a.dv);
+      return launch_tc_pass<T, MODE, CHANNEL>(a, dim3((a.dv + warps * 16 - 1) / (warps * 16), rows, sequences), warps, stream);
+    }
+  }
+#endif
   const int th = lin_threads(a.dv);
-  const int cols = th / kGroups * kCols, blocks = (a.dv + cols - 1) / cols;
-  const size_t smem = a.y != nullptr ? static_cast<size_t>(kTok) * a.dv * sizeof(float) : 0;
-  if (a.y != nullptr && blocks != 1) return static_cast<int>(cudaErrorInvalidValue);
-  if (a.chunk_state == nullptr || a.max_chunks <= 1)
-    return static_cast<int>(launch_kernel(linear_attention_kernel<T, 0, CHANNEL>, dim3(blocks, a.heads, sequences),
-                                          dim3(th), smem, stream, a));
-  cudaError_t e = launch_kernel(linear_attention_kernel<T, 1, CHANNEL>, dim3(blocks, a.heads * a.max_chunks, sequences),
-                                dim3(th), 0, stream, a);
-  if (e != cudaSuccess) return static_cast<int>(e);
-  const int plane = kD * a.dv;
-  e = launch_kernel(linear_attention_chain_kernel, dim3((plane + 255) / 256, a.heads, sequences), dim3(256), 0, stream,
-                    a.seq_of_token, a.state_slot, a.decay, static_cast<const float*>(CHANNEL ? a.chunk_decay : nullptr),
-                    static_cast<const float*>(a.state), a.slot_stride, a.chunk_state, a.tokens, a.heads, a.dv, a.chunk,
-                    a.max_chunks);
-  if (e != cudaSuccess) return static_cast<int>(e);
-  return static_cast<int>(launch_kernel(linear_attention_kernel<T, 3, CHANNEL>,
-                                        dim3(blocks, a.heads * a.max_chunks, sequences), dim3(th), smem, stream, a));
+  const int cols = th / 32 * kSlots * kCols;
+  return launch_pass<T, MODE, CHANNEL>(a, dim3((a.dv + cols - 1) / cols, rows, sequences), th, stream);
+}
+
+template <typename T>
+cudaError_t launch_output(const LinArgs<T>& a, cudaStream_t stream) {
+  const int items = a.tokens * a.heads, warps = 8;
+  return launch_kernel(linear_output_kernel<T>, dim3((items + warps - 1) / warps), dim3(warps * 32), 0, stream,
+                       static_cast<const float*>(a.out), a.gate, a.gate_ld, a.gate_mode, a.norm_w, a.y, a.y_ld, items,
+                       a.heads, a.dv, a.eps);
+}
+
+template <typename T, bool CHANNEL>
+int launch_linear_attention(const LinArgs<T>& a0, int sequences, bool tc, cudaStream_t stream) {
+  // finished heads: by the recurrence itself where one CTA has all columns of a head, else by a kernel behind it
+  LinArgs<T> a = a0;
+  const int th = lin_threads(a.dv);
+  const bool one_block = a.dv <= (tc ? kTcMaxCols : th / 32 * kSlots * kCols);
+  const bool behind = a.y != nullptr && !one_block;
+  if (behind) a.y = nullptr;
+  cudaError_t e;
+  if (a.chunk_state == nullptr || a.max_chunks <= 1) {
+    e = launch_either<T, 0, CHANNEL>(a, a.heads, sequences, tc, stream);
+  } else {
+    e = launch_either<T, 1, CHANNEL>(a, a.heads * a.max_chunks, sequences, tc, stream);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    const int plane = kD * a.dv;
+    e = launch_kernel(linear_attention_chain_kernel, dim3((plane + 255) / 256, a.heads, sequences), dim3(256), 0, stream,
+                      a.seq_of_token, a.state_slot, a.decay, static_cast<const float*>(CHANNEL ? a.chunk_decay : nullptr),
+                      static_cast<const float*>(a.state), a.slot_stride, a.chunk_state, a.tokens, a.heads, a.dv, a.chunk,
+                      a.max_chunks);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    e = launch_either<T, 3, CHANNEL>(a, a.heads * a.max_chunks, sequences, tc, stream);
+  }
+  if (e == cudaSuccess && behind) e = launch_output(a0, stream);
+  return static_cast<int>(e);
 }
 
 }  // namespace rl
@@ -446,12 +687,9 @@ using namespace rl;
 
 extern "C" {
 
-// Whether one CTA covers all columns of a head (the finished heads can then be asked for).
-int rl_linear_one_block(int dv) {
-  const int th = lin_threads(dv);
-  return dv <= th / kGroups * kCols ? 1 : 0;
-}
-
+// With y the finished heads are asked for, and out [tokens, heads * DV] is scratch that may be used on the way.
+// longest: the most tokens any sequence of the step brings (from kTcMinTokens on, and where sizes allow, bfloat16
+// steps run in blocks on the tensor cores; 0: never).
 // chunk_state null or max_chunks <= 1: every sequence is one serial chain.  Otherwise sequences are cut
 // into chunks of `chunk` tokens (max_chunks = the most chunks any sequence of the step has) and
 // chunk_state holds [sequences, max_chunks, heads, D, DV] floats, chunk_decay (a decay per channel only)
@@ -462,10 +700,10 @@ int rl_linear_attention(int dtype, const void* q, int q_ld, const void* k, int k
                         const float* decay_bias, const float* bonus, float* state, long long slot_stride, float* out,
                         void* y, int y_ld, const void* gate, int gate_ld, int gate_mode, const float* norm_w, float eps,
                         float* chunk_state, float* chunk_decay, int* status, int tokens, int sequences, int heads,
-                        int dv, int chunk, int max_chunks, cudaStream_t stream) {
+                        int dv, int chunk, int max_chunks, int longest, cudaStream_t stream) {
   if (tokens <= 0 || sequences <= 0) return 0;
   const bool channel = bonus != nullptr;
-  if (channel && (decay_bias == nullptr || (max_chunks > 1 && chunk_state != nullptr && chunk_decay == nullptr)))
+  if (out == nullptr || (channel && (decay_bias == nullptr || (max_chunks > 1 && chunk_state != nullptr && chunk_decay == nullptr))))
     return static_cast<int>(cudaErrorInvalidValue);
 #define RL_CASE(T)                                                                                                \
   do {                                                                                                            \
@@ -478,28 +716,22 @@ int rl_linear_attention(int dtype, const void* q, int q_ld, const void* k, int k
     a.gate = static_cast<const T*>(gate); a.gate_ld = gate_ld; a.gate_mode = gate_mode; a.norm_w = norm_w;        \
     a.eps = eps; a.chunk_state = chunk_state; a.chunk_decay = chunk_decay; a.status = status; a.tokens = tokens;  \
     a.heads = heads; a.dv = dv; a.chunk = chunk; a.max_chunks = max_chunks;                                       \
-    a.pairs_ok = dv % 2 == 0 && slot_stride % 2 == 0 && reinterpret_cast<uintptr_t>(state) % 8 == 0 &&            \
-                 reinterpret_cast<uintptr_t>(chunk_state) % 8 == 0;                                               \
-    if (channel) return launch_linear_attention<T, true>(a, sequences, stream);                                   \
-    return launch_linear_attention<T, false>(a, sequences, stream);                                               \
+    a.quads_ok = dv % 4 == 0 && slot_stride % 4 == 0 && on16(state) && on16(chunk_state);                         \
+    constexpr int E = 16 / sizeof(T);      /* elements of a 16-byte piece */                                      \
+    a.qk_ok = kD % E == 0 && q_ld % E == 0 && k_ld % E == 0 && on16(q) && on16(k);                                \
+    a.v_ok = dv % E == 0 && v_ld % E == 0 && on16(v);                                                             \
+    a.g_ok = dv % E == 0 && gate_ld % E == 0 && on16(gate);                                                       \
+    a.z_ok = kD % 4 == 0 && on16(decay);                                                                          \
+    a.rot_ok = rot_pairs % 4 == 0 && on16(cos_t) && on16(sin_t);                                                  \
+    const bool tc = longest >= kTcMinTokens && sizeof(T) == 2 && kD % 16 == 0 && dv % 16 == 0 && a.qk_ok &&       \
+                    a.v_ok && (a.g_ok || gate_mode == GATE_NONE || y == nullptr) && (a.z_ok || !channel) &&       \
+                    (a.rot_ok || rot_pairs == 0);                                                                 \
+    if (channel) return launch_linear_attention<T, true>(a, sequences, tc, stream);                               \
+    return launch_linear_attention<T, false>(a, sequences, tc, stream);                                           \
   } while (0)
   if (dtype == 0) RL_CASE(float);
   else RL_CASE(bf16);
 #undef RL_CASE
-}
-
-int rl_linear_output(int dtype, const float* o, const void* gate, int gate_ld, int gate_mode, const float* w, void* y,
-                     int y_ld, int tokens, int heads, int dv, float eps, cudaStream_t stream) {
-  const int items = tokens * heads, warps = 8;
-  if (items <= 0) return 0;
-  const dim3 grid((items + warps - 1) / warps);
-  if (dtype == 0)
-    launch_kernel(linear_output_kernel<float>, grid, dim3(warps * 32), 0, stream, o, static_cast<const float*>(gate),
-                  gate_ld, gate_mode, w, static_cast<float*>(y), y_ld, items, heads, dv, eps);
-  else
-    launch_kernel(linear_output_kernel<bf16>, grid, dim3(warps * 32), 0, stream, o, static_cast<const bf16*>(gate),
-                  gate_ld, gate_mode, w, static_cast<bf16*>(y), y_ld, items, heads, dv, eps);
-  RL_LAUNCH_END();
 }
 
 }  // extern "C"

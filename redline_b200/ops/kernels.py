@@ -927,12 +927,16 @@ LINEAR_ATTN_CHUNK_FROM = 256       # sequences that bring at least so many token
 LINEAR_ATTN_MAX_CHUNKS = 64
 
 
-def linear_attention_chunks(longest: int) -> Tuple[int, int]:
+def linear_attention_chunks(longest: int, blocks: bool = False) -> Tuple[int, int]:
     """(chunk length, most chunks) for a step whose longest sequence brings ``longest`` tokens; (0, 1) when
-    every sequence is run as one chain."""
+    every sequence is run as one chain.  ``blocks``: for the form that runs blocks of tokens on the tensor cores,
+    whose state costs more to hand from chunk to chunk than to carry on."""
     if longest < LINEAR_ATTN_CHUNK_FROM:
         return 0, 1
-    chunk = max(64, (longest + LINEAR_ATTN_MAX_CHUNKS - 1) // LINEAR_ATTN_MAX_CHUNKS)
+    most = 16 if blocks else LINEAR_ATTN_MAX_CHUNKS
+    chunk = max(64, (longest + most - 1) // most)
+    if blocks:
+        chunk = (chunk + 63) // 64 * 64
     return chunk, (longest + chunk - 1) // chunk
 
 
@@ -945,13 +949,8 @@ def _lin(dim: int) -> ctypes.CDLL:
     return _lib(f"linear_attention_d{dim}", "linear_attention.cu", {"RL_LIN_DIM": dim})
 
 
-def linear_attention_finishes(dim: int, vdim: int) -> bool:
-    """Whether the recurrence's kernel can also norm, weigh and gate the heads (``y`` of ``linear_attention``)."""
-    return bool(_fn(_lin(dim), "rl_linear_one_block", [c_int])(vdim))
-
-
 def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, seq_of_token: torch.Tensor,
-                     state_slot: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: Optional[torch.Tensor],
+                     state_slot: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
                      tokens: int, sequences: int, heads: int, dim: int, vdim: int,
                      chunk_state: Optional[torch.Tensor] = None, chunk: int = 0, max_chunks: int = 1,
                      k_scale: float = 1.0, cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None,
@@ -959,7 +958,7 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, seq_of_t
                      bonus: Optional[torch.Tensor] = None, chunk_decay: Optional[torch.Tensor] = None,
                      y: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_mode: int = GATE_NONE,
                      norm_w: Optional[torch.Tensor] = None, eps: float = 0.0,
-                     status: Optional[torch.Tensor] = None) -> None:
+                     status: Optional[torch.Tensor] = None, longest: int = 0) -> None:
     """A recurrence per head over every sequence of the step, from and into the sequences' state slots
     (csrc/linear_attention.cu).  q, k [tokens, heads * dim] and v [tokens, heads * vdim] are row-strided views of
     one type; state float32 [slots, heads * dim * vdim] (or [slots, heads, dim, vdim]).
@@ -970,11 +969,12 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, seq_of_t
     float32 [heads * dim].  q and k are rotated first (``cos``, ``sin`` [positions, pairs]: entry i with entry
     i + pairs), k multiplied by ``k_scale``.
 
-    ``out`` receives o (float32 [tokens, heads * vdim]); or ``y`` (where ``linear_attention_finishes``) the
-    finished heads, o / sqrt(mean over the head (o^2) + eps) * norm_w * act(gate), in the activation type.
+    ``out`` (float32 [tokens, heads * vdim]) receives o; with ``y`` the finished heads go there, o / sqrt(mean over
+    the head (o^2) + eps) * norm_w * act(gate), in the activation type, and ``out`` is scratch.
     With ``chunk_state`` (float32, sequences * max_chunks * heads * dim * vdim; per channel also ``chunk_decay``,
     sequences * max_chunks * heads * dim) sequences are cut into chunks of ``chunk`` tokens that run side by
-    side."""
+    side.  ``longest``: the most tokens any sequence of the step brings; bfloat16 steps with longer sequences run in
+    blocks of 16 tokens on the tensor cores where sizes allow (0: never)."""
     _need_cuda(q, k, v, state, out, y, gate, decay, decay_bias, bonus, chunk_state, chunk_decay, norm_w)
     channel = bonus is not None
     for t in (decay, decay_bias, bonus, out, norm_w, chunk_state, chunk_decay):
@@ -991,9 +991,8 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, seq_of_t
         raise KernelError("linear_attention: decays per channel come with a bias and a bonus of [heads * dim]")
     if not channel and decay.numel() != heads:
         raise KernelError("linear_attention: one decay per head")
-    if (out is None) == (y is None) or (y is not None and (y.dtype != q.dtype or y.stride(1) != 1
-                                                           or not linear_attention_finishes(dim, vdim))):
-        raise KernelError("linear_attention: either float32 sums or (where one CTA has a head) the finished heads")
+    if out.shape[1] != heads * vdim or (y is not None and (y.dtype != q.dtype or y.stride(1) != 1 or y.shape[1] != heads * vdim)):
+        raise KernelError("linear_attention: float32 sums [tokens, heads * vdim], finished heads of q's type")
     if gate is not None and (gate.dtype != q.dtype or gate.stride(1) != 1 or gate.shape[1] != heads * vdim):
         raise KernelError("linear_attention: the gate has one entry per output and the activation type")
     pairs = 0
@@ -1009,7 +1008,7 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, seq_of_t
     f = _fn(_lin(dim), "rl_linear_attention",
             [c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int,
              c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_void_p,
-             c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+             c_int, c_int, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
              c_void_p])
     _check(f(_code(q.dtype), _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), float(k_scale), _ptr(cos),
              _ptr(sin), _ptr(positions), pairs, cos.shape[0] if cos is not None else 0, _ptr(seq_of_token),
@@ -1017,23 +1016,7 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, seq_of_t
              y.stride(0) if y is not None else 0, _ptr(gate), gate.stride(0) if gate is not None else 0,
              gate_mode if gate is not None else GATE_NONE, _ptr(norm_w), float(eps),
              _ptr(chunk_state) if chunked else None, _ptr(chunk_decay) if chunked and channel else None, _ptr(status), tokens,
-             sequences, heads, vdim, chunk, max_chunks if chunked else 1, _stream()), "linear_attention", 3 if chunked else 1)
-
-
-def linear_output(o: torch.Tensor, gate: Optional[torch.Tensor], gate_mode: int, norm_w: Optional[torch.Tensor],
-                  y: torch.Tensor, tokens: int, heads: int, dim: int, vdim: int, eps: float) -> None:
-    """y = o / sqrt(mean over the head (o^2) + eps) (* norm_w) (* act(gate)): o float32 [tokens, heads * vdim],
-    gate and y row-strided views of the activation type, norm_w float32 [heads * vdim]."""
-    _need_cuda(o, gate, norm_w, y)
-    if o.dtype != torch.float32 or not o.is_contiguous() or y.stride(1) != 1 \
-            or (gate is not None and (gate.dtype != y.dtype or gate.stride(1) != 1)) \
-            or (norm_w is not None and (norm_w.dtype != torch.float32 or norm_w.numel() != heads * vdim)):
-        raise KernelError("linear_output: bad shapes")
-    f = _fn(_lin(dim), "rl_linear_output", [c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int,
-                                            c_int, c_int, c_float, c_void_p])
-    _check(f(_code(y.dtype), _ptr(o), _ptr(gate), gate.stride(0) if gate is not None else 0,
-             gate_mode if gate is not None else GATE_NONE, _ptr(norm_w), _ptr(y), y.stride(0), tokens, heads, vdim,
-             float(eps), _stream()), "linear_output")
+             sequences, heads, vdim, chunk, max_chunks if chunked else 1, longest, _stream()), "linear_attention", 3 if chunked else 1)
 
 
 # ------------------------------------------------------- matrix memory with exponential gates

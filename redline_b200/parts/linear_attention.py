@@ -42,25 +42,23 @@ class LinearAttentionParams:
 def run_recurrence(part, ctx, q, k, v, decay, state, y, heads: int, dim: int, vdim: int, gate, gate_mode: int,
                    norm_w=None, eps: float = 0.0, finish: bool = True, **kw) -> Optional[torch.Tensor]:
     """The recurrence of csrc/linear_attention.cu over the step, cut into chunks where sequences are long.  With
-    ``finish`` the heads are normed (per head), weighed and gated into ``y``, in the recurrence's kernel where
-    that can; without, the float32 sums are returned."""
+    ``finish`` the heads are normed (per head), weighed and gated into ``y``; without, the float32 sums are
+    returned."""
     rt, T = part.rt, ctx.T
     ws = rt.workspace
     # (how a step is cut depends on its shape alone: single-token steps and full portions replay as graphs)
-    chunk, max_chunks = kernels.linear_attention_chunks(1 if ctx.num_tiles == 0 else max(ctx.host.q_len))
+    longest = 1 if ctx.num_tiles == 0 else max(ctx.host.q_len)
+    chunk, max_chunks = kernels.linear_attention_chunks(longest, blocks=rt.dtype == torch.bfloat16 and dim % 16 == 0 and vdim % 16 == 0)
     if max_chunks > 1:
         kw["chunk_state"] = ws.get("lin.chunks", (ctx.S * max_chunks * heads * dim * vdim,), torch.float32)
         if kw.get("bonus") is not None:
             kw["chunk_decay"] = ws.get("lin.chunk_decay", (ctx.S * max_chunks * heads * dim,), torch.float32)
-    kw.update(chunk=chunk, max_chunks=max_chunks, status=ctx.status)
-    in_kernel = finish and kernels.linear_attention_finishes(dim, vdim)
-    o = None if in_kernel else ws.get("lin.o", (rt.max_tokens, heads * vdim), torch.float32)[:T]
-    if in_kernel:
+    kw.update(chunk=chunk, max_chunks=max_chunks, status=ctx.status, longest=longest)
+    o = ws.get("lin.o", (rt.max_tokens, heads * vdim), torch.float32)[:T]
+    if finish:
         kw.update(y=y, gate=gate, gate_mode=gate_mode, norm_w=norm_w, eps=eps)
     kernels.linear_attention(q, k, v, ctx.seq_of_token, ctx.state_slot, decay, state, o, T, ctx.S, heads, dim, vdim, **kw)
-    if finish and not in_kernel:
-        kernels.linear_output(o, gate, gate_mode, norm_w, y, T, heads, dim, vdim, eps)
-    return o
+    return None if finish else o
 
 
 @register("mixer", "linear_attention")
