@@ -59,6 +59,9 @@ struct SkinnyArgs {
   const float* ss_in;
   int ss_n;
   int gate_act;           // kSwiglu: what is applied to the gate, 0 SiLU, 1 the tanh form of GELU
+  // GROUPED (unstaged bfloat16 x of up to 8 rows): features f * x_group .. (f + 1) * x_group - 1 multiply the
+  // activations at x + f * x_stride (several products with inputs of their own as one; x_group a multiple of 16)
+  int x_group, x_stride;
 };
 
 
@@ -136,7 +139,7 @@ __device__ __noinline__ void hand_over_epilogue(const float* red, const float* e
 // 16-row weight stream; EPI: epilogue; NORM: fused norm.  The CTA's WARPS / KW groups of warps
 // take different streams at the same time: 16-row tiles next to each other and, for the gated
 // product, the gate rows and the up rows of a tile.
-template <int MT, int WARPS, int KW, int EPI, bool NORM>
+template <int MT, int WARPS, int KW, int EPI, bool NORM, bool GROUPED>
 __global__ void __launch_bounds__(WARPS * 32, WARPS <= 8 ? 2 : 1)     // (at most 128 registers: two CTAs of 8 warps per SM)
 gemm_skinny_kernel(const SkinnyArgs a, int kc, int extra_off) {
   constexpr bool GATED = (EPI == kSwiglu);
@@ -177,7 +180,9 @@ gemm_skinny_kernel(const SkinnyArgs a, int kc, int extra_off) {
   // the wait for the kernels before this one, the norm and the staging.
   WFrag fa, fb;
   const bf16 *w_lo, *w_hi;
+  int x_off = 0;                             // GROUPED: where the load cursor's tile finds its activations
   auto set_rows = [&](int n0) {
+    if (GROUPED) x_off = min(n0, a.N - 1) / a.x_group * a.x_stride;
     const int r_lo = min(n0 + g, a.N - 1), r_hi = min(n0 + g + 8, a.N - 1);   // clamped; stores are predicated
     w_lo = a.w + static_cast<size_t>(stream * a.N + r_lo) * K;
     w_hi = a.w + static_cast<size_t>(stream * a.N + r_hi) * K;
@@ -196,7 +201,7 @@ gemm_skinny_kernel(const SkinnyArgs a, int kc, int extra_off) {
   auto load_x = [&](uint4& xv, int q) {          // (after the wait on the kernels before: they wrote x)
     const int k = l_sb * kSB + q * 32 + t * 8;
     const bool ok = l_ok && k < K && g < M;
-    xv = ok ? *reinterpret_cast<const uint4*>(a.x + static_cast<size_t>(g) * a.ldx + k) : make_uint4(0, 0, 0, 0);
+    xv = ok ? *reinterpret_cast<const uint4*>(a.x + (GROUPED ? x_off : 0) + static_cast<size_t>(g) * a.ldx + k) : make_uint4(0, 0, 0, 0);
   };
   auto load_advance = [&]() {
     l_sb += KW;
@@ -208,12 +213,12 @@ gemm_skinny_kernel(const SkinnyArgs a, int kc, int extra_off) {
     }
   };
   pdl_launch();
-  const int sb0 = l_sb;
+  const int sb0 = l_sb, xo0 = x_off;
   const bool ok0 = l_ok;
 #pragma unroll
   for (int q = 0; q < 4; ++q) load_piece(fa.lo[q], fa.hi[q], q);
   load_advance();
-  const int sb1 = l_sb;
+  const int sb1 = l_sb, xo1 = x_off;
   const bool ok1 = l_ok;
 #pragma unroll
   for (int q = 0; q < 4; ++q) load_piece(fb.lo[q], fb.hi[q], q);
@@ -235,18 +240,21 @@ gemm_skinny_kernel(const SkinnyArgs a, int kc, int extra_off) {
     }
   }
   if (XG) {     // the activations of the first two steps (the load cursor is already two steps on)
-    const int sb2 = l_sb;
+    const int sb2 = l_sb, xo2 = x_off;
     const bool ok2 = l_ok;
     l_sb = sb0;
     l_ok = ok0;
+    x_off = xo0;
 #pragma unroll
     for (int q = 0; q < 4; ++q) load_x(fa.x[q], q);
     l_sb = sb1;
     l_ok = ok1;
+    x_off = xo1;
 #pragma unroll
     for (int q = 0; q < 4; ++q) load_x(fb.x[q], q);
     l_sb = sb2;
     l_ok = ok2;
+    x_off = xo2;
   }
 
   // a norm handed over by the product before: row m's partial sums are added up by warp m after the k loop
@@ -410,7 +418,7 @@ gemm_skinny_kernel(const SkinnyArgs a, int kc, int extra_off) {
   }
 }
 
-template <int MT, int WARPS, int KW, int EPI, bool NORM>
+template <int MT, int WARPS, int KW, int EPI, bool NORM, bool GROUPED>
 int launch_one(const SkinnyArgs& a0, int sm_count, cudaStream_t stream) {
   constexpr int STREAMS = (EPI == kSwiglu) ? 2 : 1;
   constexpr int TPC = WARPS / KW / STREAMS;
@@ -445,12 +453,12 @@ int launch_one(const SkinnyArgs& a0, int sm_count, cudaStream_t stream) {
   if (smem > 200 * 1024) return static_cast<int>(cudaErrorInvalidValue);
   static size_t set_for = 0;
   if (smem > set_for) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_skinny_kernel<MT, WARPS, KW, EPI, NORM>,
+    cudaError_t e = cudaFuncSetAttribute(gemm_skinny_kernel<MT, WARPS, KW, EPI, NORM, GROUPED>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     set_for = smem;
   }
-  launch_kernel(gemm_skinny_kernel<MT, WARPS, KW, EPI, NORM>, dim3(ctas), dim3(WARPS * 32), smem, stream, a, kc,
+  launch_kernel(gemm_skinny_kernel<MT, WARPS, KW, EPI, NORM, GROUPED>, dim3(ctas), dim3(WARPS * 32), smem, stream, a, kc,
                 static_cast<int>(extra_off));
   return static_cast<int>(cudaGetLastError());
 }
@@ -467,19 +475,19 @@ inline int choose_kw(int N, int K, int streams, int sm_count) {
   return kw;
 }
 
-template <int MT, int EPI, bool NORM>
+template <int MT, int EPI, bool NORM, bool GROUPED = false>
 int launch_kw(const SkinnyArgs& a, int sm_count, cudaStream_t stream) {
   constexpr int STREAMS = (EPI == kSwiglu) ? 2 : 1;
   int kw = choose_kw(a.N, a.K, STREAMS, sm_count);
   if (STREAMS == 2 && kw > 4) kw = 4;      // 8 warps hold both streams of a tile
   switch (kw) {
-    case 1: return launch_one<MT, 8, 1, EPI, NORM>(a, sm_count, stream);
-    case 2: return launch_one<MT, 8, 2, EPI, NORM>(a, sm_count, stream);
-    case 4: return launch_one<MT, 8, 4, EPI, NORM>(a, sm_count, stream);
+    case 1: return launch_one<MT, 8, 1, EPI, NORM, GROUPED>(a, sm_count, stream);
+    case 2: return launch_one<MT, 8, 2, EPI, NORM, GROUPED>(a, sm_count, stream);
+    case 4: return launch_one<MT, 8, 4, EPI, NORM, GROUPED>(a, sm_count, stream);
     case 8:
-      if constexpr (STREAMS == 1) return launch_one<MT, 8, 8, EPI, NORM>(a, sm_count, stream);
+      if constexpr (STREAMS == 1) return launch_one<MT, 8, 8, EPI, NORM, GROUPED>(a, sm_count, stream);
     default:
-      if constexpr (STREAMS == 1) return launch_one<MT, 16, 16, EPI, NORM>(a, sm_count, stream);
+      if constexpr (STREAMS == 1) return launch_one<MT, 16, 16, EPI, NORM, GROUPED>(a, sm_count, stream);
   }
   return static_cast<int>(cudaErrorInvalidValue);
 }
@@ -518,8 +526,7 @@ int rl_gemm_skinny_handover(const void* w, const void* x, int ldx, const float* 
     return static_cast<int>(cudaErrorInvalidValue);
   if (ss_in != nullptr && (norm || M > 8 || ss_n <= 0 || epilogue == kAddResidual))
     return static_cast<int>(cudaErrorInvalidValue);
-  SkinnyArgs a;
-  a.gate_act = 0;
+  SkinnyArgs a = {};
   if (epilogue == 4) {            // the gated product with the tanh form of GELU on the gate
     epilogue = kSwiglu;
     a.gate_act = 1;
@@ -560,6 +567,27 @@ int rl_gemm_skinny_handover(const void* w, const void* x, int ldx, const float* 
     }
   }
   return static_cast<int>(cudaErrorInvalidValue);
+}
+
+// Several products of up to 8 rows as one: feature n multiplies the activations at x + n / x_group * x_stride.
+int rl_gemm_skinny_grouped(const void* w, const void* x, int ldx, int x_group, int x_stride, void* y, int ldy, int M, int N,
+                           int K, int sm_count, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (M > 8 || K % 8 != 0 || ldx % 8 != 0 || x_group <= 0 || x_group % 16 != 0 || x_stride % 8 != 0)
+    return static_cast<int>(cudaErrorInvalidValue);
+  SkinnyArgs a = {};
+  a.w = static_cast<const bf16*>(w);
+  a.x = static_cast<const bf16*>(x);
+  a.y = y;
+  a.M = M;
+  a.N = N;
+  a.K = K;
+  a.ldx = ldx;
+  a.ldy = ldy;
+  a.row_tiles = 1;
+  a.x_group = x_group;
+  a.x_stride = x_stride;
+  return launch_kw<8, kStoreBf16, false, true>(a, sm_count, stream);
 }
 
 int rl_gemm_skinny(const void* w, const void* x, int ldx, const float* residual, const void* norm_w,

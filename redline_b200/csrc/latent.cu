@@ -16,7 +16,8 @@
 //                 neighbours, cos and sin from tables), [c | k_r] into the paged cache, q_r into the
 //                 attention's query rows; the norm of the queries' latent
 //   head_linear   y[t, h, :] = W_h x[t, h, :] for every head h, W [heads, n, k], float32 sums in ascending k
-//                 (a row's result does not depend on what else is in the launch); FFMA for float32, and
+//                 (a row's result does not depend on what else is in the launch); the heads' rotated query
+//                 parts may go along; FFMA for float32, and
 //                 mma.sync.m16n8k16 for bfloat16 operands whose sizes allow it
 #include "common.cuh"
 
@@ -115,16 +116,45 @@ latent_prep_kernel(const TA* __restrict__ q, const TA* __restrict__ craw, const 
 
 // ------------------------------------------------------------------ per-head products
 // y[t, y_col + h * y_head + j] = sum_k W[h, j, k] x[t, x_col + h * x_head + k]
+// and, with turn.dims > 0, the rotated part of every head's row goes along: y[t, y_col + h * y_head + turn.y + d] =
+// entry d of the part at x[t, x_col + h * x_head + turn.x], turned by the token's position (see `rotated`).
+struct Turn {
+  int dims, rot_dims, pairs, x, y, max_pos;      // dims: entries of the part, of which the first rot_dims turn
+  const float *cos_t, *sin_t;                    // [max_pos, rot_dims / 2]
+  const int32_t* positions;
+  int* status;
+};
 struct HeadLinearArgs {
   int tokens, heads, n, k;
   int x_ld, x_col, x_head;
   int y_ld, y_col, y_head;
+  Turn turn;
 };
+
+// The rotated parts of tokens t0 .. t0 + rows - 1 of head h, by all threads of a CTA.
+template <typename TA>
+__device__ __forceinline__ void turn_parts(const TA* __restrict__ x, TA* __restrict__ y, const HeadLinearArgs& a, int t0,
+                                           int rows, int h) {
+  const Turn& r = a.turn;
+  for (int i = threadIdx.x; i < rows * r.dims; i += blockDim.x) {
+    const int t = t0 + i / r.dims, d = i % r.dims;
+    if (t >= a.tokens) return;
+    int pos = r.positions[t];
+    if (pos < 0 || pos >= r.max_pos) {
+      atomicOr(r.status, 2);
+      pos = 0;
+    }
+    const size_t at = static_cast<size_t>(pos) * (r.rot_dims / 2);
+    y[static_cast<size_t>(t) * a.y_ld + a.y_col + h * a.y_head + r.y + d] = from_float<TA>(
+        rotated(x + static_cast<size_t>(t) * a.x_ld + a.x_col + h * a.x_head + r.x, d, r.rot_dims, r.pairs, r.cos_t + at,
+                r.sin_t + at));
+  }
+}
 
 constexpr int kHlRows = 16, kHlCols = 128, kHlK = 32;
 
 // CUDA cores: a CTA takes 16 tokens x 128 outputs of one head; thread j owns output column j for all 16 tokens.
-template <typename TA, typename TW>
+template <typename TA, typename TW, bool TURN>
 __global__ void __launch_bounds__(kHlCols)
 head_linear_kernel(const TA* __restrict__ x, const TW* __restrict__ w, TA* __restrict__ y, const HeadLinearArgs a) {
   pdl_launch();
@@ -132,6 +162,10 @@ head_linear_kernel(const TA* __restrict__ x, const TW* __restrict__ w, TA* __res
   __shared__ float xs[kHlRows][kHlK];
   __shared__ float wsm[kHlK][kHlCols + 1];
   const int t0 = blockIdx.x * kHlRows, j0 = blockIdx.y * kHlCols, h = blockIdx.z;
+  if (TURN && blockIdx.y == gridDim.y - 1) {          // the last row of CTAs turns the rotated parts
+    turn_parts(x, y, a, t0, kHlRows, h);
+    return;
+  }
   const int j = j0 + threadIdx.x;
   const TW* wh = w + static_cast<size_t>(h) * a.n * a.k;
   float acc[kHlRows];
@@ -177,6 +211,7 @@ __device__ __forceinline__ void hl_mma(float* d, const uint32_t* a, uint32_t b0,
 
 constexpr int kHmRows = 64, kHmCols = 64;
 
+template <bool TURN>
 __global__ void __launch_bounds__(128)
 head_linear_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16* __restrict__ y,
                        const HeadLinearArgs a) {
@@ -184,6 +219,10 @@ head_linear_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, b
   pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
   const int t0 = blockIdx.x * kHmRows + warp * 16, j0 = blockIdx.y * kHmCols, h = blockIdx.z;
+  if (TURN && blockIdx.y == gridDim.y - 1) {
+    turn_parts(x, y, a, blockIdx.x * kHmRows, kHmRows, h);
+    return;
+  }
   if (t0 >= a.tokens) return;
   const int r0 = t0 + gid, r1 = r0 + 8;
   const bool ok0 = r0 < a.tokens, ok1 = r1 < a.tokens;
@@ -220,6 +259,69 @@ head_linear_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, b
       *reinterpret_cast<__nv_bfloat162*>(y + static_cast<size_t>(r1) * a.y_ld + a.y_col + h * a.y_head + j) =
           __floats2bfloat162_rn(acc[nt][2], acc[nt][3]);
   }
+}
+
+// A few tokens (single-token steps): the product is bound by the stream of the heads' matrices, and CTAs of the
+// kernel above would be few and each walk all of k.  A warp takes four output features of one head and streams
+// their rows in 16-byte pieces, lanes side by side, up to eight tokens at a time; the lanes' sums meet by
+// shuffles.  Needs k % 8 == 0 and rows on 16-byte boundaries.
+constexpr int kHfTokens = 8, kHfCols = 4;
+template <bool TURN>
+__global__ void __launch_bounds__(128)
+head_linear_few_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16* __restrict__ y, const HeadLinearArgs a) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h = blockIdx.y, t0 = blockIdx.z * kHfTokens;
+  pdl_launch();
+  if (TURN && blockIdx.x == gridDim.x - 1) {
+    pdl_wait();
+    turn_parts(x, y, a, t0, kHfTokens, h);
+    return;
+  }
+  const int j0 = (blockIdx.x * 4 + warp) * kHfCols;
+  if (j0 >= a.n) return;
+  const bf16* wr[kHfCols];
+#pragma unroll
+  for (int f = 0; f < kHfCols; ++f) wr[f] = w + (static_cast<size_t>(h) * a.n + min(j0 + f, a.n - 1)) * a.k;
+  float acc[kHfCols][kHfTokens];
+#pragma unroll
+  for (int f = 0; f < kHfCols; ++f)
+#pragma unroll
+    for (int t = 0; t < kHfTokens; ++t) acc[f][t] = 0.f;
+  const int nt = min(kHfTokens, a.tokens - t0);
+  const bf16* xr = x + static_cast<size_t>(t0) * a.x_ld + a.x_col + h * a.x_head;
+  for (int c0 = 0; c0 < a.k; c0 += 256) {
+    const int c = c0 + lane * 8;
+    const bool in = c < a.k;
+    float wv[kHfCols][8];
+#pragma unroll
+    for (int f = 0; f < kHfCols; ++f) {
+      if (in) load16(wr[f] + c, wv[f]);
+      else {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) wv[f][i] = 0.f;
+      }
+    }
+    if (c0 == 0) pdl_wait();                   // (the matrices come from no earlier kernel of the step)
+#pragma unroll
+    for (int t = 0; t < kHfTokens; ++t) {
+      if (t < nt && in) {
+        float xv[8];
+        load16(xr + static_cast<size_t>(t) * a.x_ld + c, xv);
+#pragma unroll
+        for (int f = 0; f < kHfCols; ++f)
+#pragma unroll
+          for (int i = 0; i < 8; ++i) acc[f][t] = fmaf(wv[f][i], xv[i], acc[f][t]);
+      }
+    }
+  }
+#pragma unroll
+  for (int f = 0; f < kHfCols; ++f)
+#pragma unroll
+    for (int t = 0; t < kHfTokens; ++t) {
+      const float v = warp_sum(acc[f][t]);
+      if (lane == 0 && t < nt && j0 + f < a.n)
+        y[static_cast<size_t>(t0 + t) * a.y_ld + a.y_col + h * a.y_head + j0 + f] = __float2bfloat16_rn(v);
+    }
 }
 
 }  // namespace rl
@@ -263,9 +365,11 @@ int rl_latent_prep(int act_dtype, int w_dtype, const void* q, int q_src_ld, cons
   RL_LAUNCH_END();
 }
 
-// impl 0: the tensor cores where they apply; 1: CUDA cores.
+// impl 0: the form that fits (few tokens, tensor cores, CUDA cores); 1: CUDA cores; 2: tensor cores where they apply.
 int rl_head_linear(int act_dtype, int w_dtype, const void* x, int x_ld, int x_col, int x_head, const void* w, int heads,
-                   int n, int k, void* y, int y_ld, int y_col, int y_head, int tokens, int impl, cudaStream_t stream) {
+                   int n, int k, void* y, int y_ld, int y_col, int y_head, int tokens, int impl, int turn_dims,
+                   int rot_dims, int pairs, int turn_x, int turn_y, const float* cos_t, const float* sin_t, int max_pos,
+                   const int32_t* positions, int* status, cudaStream_t stream) {
   if (tokens <= 0 || heads <= 0 || n <= 0) return 0;
   HeadLinearArgs a;
   a.tokens = tokens;
@@ -278,18 +382,35 @@ int rl_head_linear(int act_dtype, int w_dtype, const void* x, int x_ld, int x_co
   a.y_ld = y_ld;
   a.y_col = y_col;
   a.y_head = y_head;
+  a.turn = Turn{turn_dims, rot_dims, pairs, turn_x, turn_y, max_pos, cos_t, sin_t, positions, status};
   const bool even = ((x_ld | x_col | x_head | y_ld | y_col | y_head) & 1) == 0 &&
                     reinterpret_cast<uintptr_t>(x) % 4 == 0 && reinterpret_cast<uintptr_t>(y) % 4 == 0 &&
                     reinterpret_cast<uintptr_t>(w) % 4 == 0;
-  if (act_dtype == 1 && w_dtype == 1 && impl == 0 && k % 16 == 0 && n % 8 == 0 && even) {
-    launch_kernel(head_linear_mma_kernel, dim3((tokens + kHmRows - 1) / kHmRows, (n + kHmCols - 1) / kHmCols, heads),
-                  dim3(128), 0, stream, static_cast<const bf16*>(x), static_cast<const bf16*>(w), static_cast<bf16*>(y), a);
+  const int turning = turn_dims > 0 ? 1 : 0;
+  const bool pieces = act_dtype == 1 && w_dtype == 1 && k % 8 == 0 && x_ld % 8 == 0 && x_col % 8 == 0 && x_head % 8 == 0 &&
+                      reinterpret_cast<uintptr_t>(x) % 16 == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0;
+  if (impl == 0 && pieces && tokens <= 2 * kHfTokens) {
+    const dim3 grid((n + 4 * kHfCols - 1) / (4 * kHfCols) + turning, heads, (tokens + kHfTokens - 1) / kHfTokens);
+    if (turning) launch_kernel(head_linear_few_kernel<true>, grid, dim3(128), 0, stream, static_cast<const bf16*>(x), static_cast<const bf16*>(w), static_cast<bf16*>(y), a);
+    else launch_kernel(head_linear_few_kernel<false>, grid, dim3(128), 0, stream, static_cast<const bf16*>(x), static_cast<const bf16*>(w), static_cast<bf16*>(y), a);
     RL_LAUNCH_END();
   }
-  dim3 grid((tokens + kHlRows - 1) / kHlRows, (n + kHlCols - 1) / kHlCols, heads);
-#define RL_CASE(TA, TW)                                                                                       \
-  launch_kernel(head_linear_kernel<TA, TW>, grid, dim3(kHlCols), 0, stream, static_cast<const TA*>(x),        \
-                static_cast<const TW*>(w), static_cast<TA*>(y), a)
+  if (act_dtype == 1 && w_dtype == 1 && impl != 1 && k % 16 == 0 && n % 8 == 0 && even) {
+    const dim3 grid((tokens + kHmRows - 1) / kHmRows, (n + kHmCols - 1) / kHmCols + turning, heads);
+    if (turning) launch_kernel(head_linear_mma_kernel<true>, grid, dim3(128), 0, stream, static_cast<const bf16*>(x), static_cast<const bf16*>(w), static_cast<bf16*>(y), a);
+    else launch_kernel(head_linear_mma_kernel<false>, grid, dim3(128), 0, stream, static_cast<const bf16*>(x), static_cast<const bf16*>(w), static_cast<bf16*>(y), a);
+    RL_LAUNCH_END();
+  }
+  dim3 grid((tokens + kHlRows - 1) / kHlRows, (n + kHlCols - 1) / kHlCols + turning, heads);
+#define RL_CASE(TA, TW)                                                                                          \
+  do {                                                                                                           \
+    if (turning)                                                                                                 \
+      launch_kernel(head_linear_kernel<TA, TW, true>, grid, dim3(kHlCols), 0, stream, static_cast<const TA*>(x), \
+                    static_cast<const TW*>(w), static_cast<TA*>(y), a);                                          \
+    else                                                                                                         \
+      launch_kernel(head_linear_kernel<TA, TW, false>, grid, dim3(kHlCols), 0, stream,                           \
+                    static_cast<const TA*>(x), static_cast<const TW*>(w), static_cast<TA*>(y), a);               \
+  } while (0)
   if (act_dtype == 0) RL_CASE(float, float);
   else if (w_dtype == 0) RL_CASE(bf16, float);
   else RL_CASE(bf16, bf16);

@@ -419,40 +419,41 @@ linear_attention_kernel(const LinArgs<T> a) {
           }
         }
       }
-      if (MODE == 1) return;
-      float o[kCols];
+      if constexpr (MODE != 1) {
+        float o[kCols];
 #pragma unroll
-      for (int j = 0; j < kCols; ++j) {
-        float lo, hi;
-        unpack2(o2[j], lo, hi);
-        o[j] = lo + hi;
-      }
-      // the groups' partial sums: lanes of two groups exchange the columns the other one keeps
-      int keep = 0;
-      constexpr int n = kGroups >= 4 ? 1 : (kGroups == 2 ? 2 : kCols);      // columns a lane is left with
-      if (kGroups >= 2) {
-        const bool up = lane & 16;
-        const float r0 = __shfl_xor_sync(0xffffffffu, up ? o[0] : o[2], 16);
-        const float r1 = __shfl_xor_sync(0xffffffffu, up ? o[1] : o[3], 16);
-        o[0] = (up ? o[2] : o[0]) + r0;
-        o[1] = (up ? o[3] : o[1]) + r1;
-        keep = up ? 2 : 0;
-      }
-      if (kGroups >= 4) {
-        const bool up = lane & 8;
-        const float r0 = __shfl_xor_sync(0xffffffffu, up ? o[0] : o[1], 8);
-        o[0] = (up ? o[1] : o[0]) + r0;
-        keep += up ? 1 : 0;
-      }
-      if (kSlots <= 4) o[0] += __shfl_xor_sync(0xffffffffu, o[0], 4);
-      if (kSlots <= 2) o[0] += __shfl_xor_sync(0xffffffffu, o[0], 2);
-      if (kSlots <= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], 1);
-      if (kSlots <= 4 && (lane & (8 - kSlots))) return;            // (one lane of those with equal sums writes)
+        for (int j = 0; j < kCols; ++j) {
+          float lo, hi;
+          unpack2(o2[j], lo, hi);
+          o[j] = lo + hi;
+        }
+        // the groups' partial sums: lanes of two groups exchange the columns the other one keeps
+        int keep = 0;
+        constexpr int n = kGroups >= 4 ? 1 : (kGroups == 2 ? 2 : kCols);      // columns a lane is left with
+        if (kGroups >= 2) {
+          const bool up = lane & 16;
+          const float r0 = __shfl_xor_sync(0xffffffffu, up ? o[0] : o[2], 16);
+          const float r1 = __shfl_xor_sync(0xffffffffu, up ? o[1] : o[3], 16);
+          o[0] = (up ? o[2] : o[0]) + r0;
+          o[1] = (up ? o[3] : o[1]) + r1;
+          keep = up ? 2 : 0;
+        }
+        if (kGroups >= 4) {
+          const bool up = lane & 8;
+          const float r0 = __shfl_xor_sync(0xffffffffu, up ? o[0] : o[1], 8);
+          o[0] = (up ? o[1] : o[0]) + r0;
+          keep += up ? 1 : 0;
+        }
+        if (kSlots <= 4) o[0] += __shfl_xor_sync(0xffffffffu, o[0], 4);
+        if (kSlots <= 2) o[0] += __shfl_xor_sync(0xffffffffu, o[0], 2);
+        if (kSlots <= 1) o[0] += __shfl_xor_sync(0xffffffffu, o[0], 1);
+        if (kSlots <= 4 && (lane & (8 - kSlots))) return;            // (one lane of those with equal sums writes)
 #pragma unroll
-      for (int j = 0; j < n; ++j) {
-        if (col + keep + j >= a.dv) continue;
-        if (finish) os[tt * a.dv + col + keep + j] = o[j];
-        else a.out[static_cast<size_t>(tb + tt) * (a.heads * a.dv) + head * a.dv + col + keep + j] = o[j];
+        for (int j = 0; j < n; ++j) {
+          if (col + keep + j >= a.dv) continue;
+          if (finish) os[tt * a.dv + col + keep + j] = o[j];
+          else a.out[static_cast<size_t>(tb + tt) * (a.heads * a.dv) + head * a.dv + col + keep + j] = o[j];
+        }
       }
     };
 #pragma unroll 1

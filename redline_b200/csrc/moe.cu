@@ -24,7 +24,7 @@
 
 namespace rl {
 
-enum { ACT_NONE = 0, ACT_RELU_SQ = 1, ACT_GELU_ERF = 2, ACT_SILU = 3, ACT_GELU_TANH = 4 };
+enum { ACT_NONE = 0, ACT_RELU_SQ = 1, ACT_GELU_ERF = 2, ACT_SILU = 3, ACT_GELU_TANH = 4, ACT_CLAMPED_SWISH = 6 };
 
 __device__ __forceinline__ float moe_activate(float z, int mode) {
   switch (mode) {
@@ -56,23 +56,23 @@ __device__ __forceinline__ ArgMax warp_argmax(ArgMax a) {
   return a;
 }
 
+struct RouteArgs {
+  int ld, tokens, width, experts, groups, keep, group_top, top, softmax, renorm;
+  const float* bias;
+  const float* choice_bias;
+  float weight_scale, renorm_floor;
+};
+
+// One token's choice by one warp; `score` points to 2 * experts + 2 * groups floats of the warp's own.
 template <typename TA, typename TW>
-__global__ void moe_route_kernel(const TA* __restrict__ x, int ld, const TW* __restrict__ router, int tokens,
-                                 int width, int experts, int groups, int keep, int group_top, int top, int softmax,
-                                 int renorm, const float* __restrict__ bias, const float* __restrict__ choice_bias,
-                                 float weight_scale, float renorm_floor, int32_t* __restrict__ choice,
-                                 float* __restrict__ weight) {
-  pdl_launch();
-  pdl_wait();
-  extern __shared__ float sm[];
-  const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t = blockIdx.x * warps + warp;
-  if (t >= tokens) return;
-  float* score = sm + warp * (2 * experts + 2 * groups);   // [experts] scores, [experts] working copy, 2 x [groups]
-  float* work = score + experts;
+__device__ __forceinline__ void route_token(const RouteArgs& a, const TA* __restrict__ xr, const TW* __restrict__ router,
+                                            int t, float* score, int32_t* choice, float* weight) {
+  const int lane = threadIdx.x & 31;
+  const int width = a.width, experts = a.experts, groups = a.groups, keep = a.keep, group_top = a.group_top, top = a.top;
+  const float *bias = a.bias, *choice_bias = a.choice_bias;
+  float* work = score + experts;           // [experts] scores, [experts] working copy, 2 x [groups]
   float* gscore = work + experts;
   float* gsel = gscore + groups;
-  const TA* xr = x + static_cast<size_t>(t) * ld;
   if (router == nullptr) {
     // x holds the logits themselves [tokens, experts] (a matrix product before this kernel made them)
     for (int e = lane; e < experts; e += 32) score[e] = to_float(xr[e]);
@@ -90,7 +90,7 @@ __global__ void moe_route_kernel(const TA* __restrict__ x, int ld, const TW* __r
     for (int e = lane; e < experts; e += 32) score[e] += bias[e];
     __syncwarp();
   }
-  if (softmax) {
+  if (a.softmax) {
     float mx = -INFINITY;
     for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, score[e]);
     mx = warp_max(mx);
@@ -172,63 +172,158 @@ __global__ void moe_route_kernel(const TA* __restrict__ x, int ld, const TW* __r
     if (found) total += score[a.i];
     __syncwarp();
   }
-  if (lane == 0 && (renorm || weight_scale != 1.f)) {
+  if (lane == 0 && (a.renorm || a.weight_scale != 1.f)) {
     for (int k = 0; k < top; ++k) {
       float wk = weight[static_cast<size_t>(t) * top + k];
-      if (renorm) wk /= total + renorm_floor;
-      weight[static_cast<size_t>(t) * top + k] = wk * weight_scale;
+      if (a.renorm) wk /= total + a.renorm_floor;
+      weight[static_cast<size_t>(t) * top + k] = wk * a.weight_scale;
     }
   }
 }
 
-// ------------------------------------------------------------------ pairs grouped by expert
-// One CTA.  counts -> offsets -> order; then the tiles.  meta: [0] number of tiles.
-constexpr int kTileRows = 64;
-
-__global__ void moe_group_kernel(const int32_t* __restrict__ choice, int pairs, int experts, int tiled,
-                                 int32_t* __restrict__ order, int32_t* __restrict__ tile_expert,
-                                 int32_t* __restrict__ tile_begin, int32_t* __restrict__ tile_rows,
-                                 int32_t* __restrict__ meta) {
+template <typename TA, typename TW>
+__global__ void moe_route_kernel(const TA* __restrict__ x, const TW* __restrict__ router, const RouteArgs a,
+                                 int32_t* __restrict__ choice, float* __restrict__ weight) {
   pdl_launch();
   pdl_wait();
-  extern __shared__ int32_t cnt[];          // [experts] counts, then [experts + 1] offsets
-  int32_t* off = cnt + experts;
-  for (int e = threadIdx.x; e < experts; e += blockDim.x) cnt[e] = 0;
-  __syncthreads();
-  for (int p = threadIdx.x; p < pairs; p += blockDim.x) atomicAdd(&cnt[choice[p]], 1);
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    int at = 0, tiles = 0;
-    for (int e = 0; e < experts; ++e) {
-      off[e] = at;
-      for (int r = 0; r < cnt[e] && e < tiled; r += kTileRows) {      // (experts from `tiled` on have no matrices)
-        tile_expert[tiles] = e;
-        tile_begin[tiles] = at + r;
-        tile_rows[tiles] = min(kTileRows, cnt[e] - r);
-        ++tiles;
+  extern __shared__ float sm[];
+  const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5;
+  const int t = blockIdx.x * warps + warp;
+  if (t >= a.tokens) return;
+  route_token(a, x + static_cast<size_t>(t) * a.ld, router, t, sm + warp * (2 * a.experts + 2 * a.groups), choice, weight);
+}
+
+// ------------------------------------------------------------------ pairs grouped by expert
+// One CTA.  counts -> offsets -> order (an expert's pairs in ascending order); then the tiles.  meta: [0] number of
+// tiles.
+constexpr int kTileRows = 64;
+constexpr int kGroupThreads = 1024;
+
+// Offsets of the experts' lists and their tiles from the counts; by one warp (running sums, 32 experts at a time;
+// experts from `tiled` on have no matrices and get no tiles).
+__device__ __forceinline__ void group_offsets(const int32_t* cnt, int experts, int tiled, int32_t* off, int32_t* first,
+                                              int32_t* __restrict__ meta) {
+  const int lane = threadIdx.x & 31;
+  int at = 0, tiles = 0;
+  for (int e0 = 0; e0 < experts; e0 += 32) {
+    const int e = e0 + lane, n = e < experts ? cnt[e] : 0;
+    const int nt = e < tiled ? (n + kTileRows - 1) / kTileRows : 0;
+    int s = n, st = nt;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int u = __shfl_up_sync(0xffffffffu, s, o), v = __shfl_up_sync(0xffffffffu, st, o);
+      if (lane >= o) {
+        s += u;
+        st += v;
       }
-      at += cnt[e];
     }
-    off[experts] = at;
-    meta[0] = tiles;
+    if (e < experts) {
+      off[e] = at + s - n;
+      first[e] = tiles + st - nt;
+    }
+    at += __shfl_sync(0xffffffffu, s, 31);
+    tiles += __shfl_sync(0xffffffffu, st, 31);
+  }
+  if (lane == 0) meta[0] = tiles;
+}
+__device__ __forceinline__ void group_tiles(const int32_t* cnt, const int32_t* off, const int32_t* first, int experts,
+                                            int tiled, int32_t* __restrict__ tile_expert, int32_t* __restrict__ tile_begin,
+                                            int32_t* __restrict__ tile_rows) {
+  for (int e = threadIdx.x; e < experts && e < tiled; e += blockDim.x)
+    for (int r = 0, i = first[e]; r < cnt[e]; r += kTileRows, ++i) {
+      tile_expert[i] = e;
+      tile_begin[i] = off[e] + r;
+      tile_rows[i] = min(kTileRows, cnt[e] - r);
+    }
+}
+
+// Every warp counts the experts of a run of pairs of its own (`rows` warps share the work: as many as their
+// counters fit in shared memory); the runs' counts are summed in order, and a pair's place is its expert's offset,
+// the counts of the runs before, and its rank within the run (pairs of one expert among 32 find each other by a
+// warp-wide match).
+__global__ void __launch_bounds__(kGroupThreads)
+moe_group_kernel(const int32_t* __restrict__ choice, int pairs, int experts, int tiled, int rows,
+                 int32_t* __restrict__ order, int32_t* __restrict__ tile_expert,
+                 int32_t* __restrict__ tile_begin, int32_t* __restrict__ tile_rows, int32_t* __restrict__ meta) {
+  pdl_launch();
+  pdl_wait();
+  extern __shared__ int32_t cnt[];          // [experts] counts, offsets, first tiles; [rows][experts] the runs' counts
+  int32_t *off = cnt + experts, *first = off + experts, *hist = first + experts;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int i = threadIdx.x; i < rows * experts; i += blockDim.x) hist[i] = 0;
+  __syncthreads();
+  const int run = ((pairs + rows - 1) / rows + 31) / 32 * 32;
+  int32_t* mine = hist + warp * experts;
+  const int begin = warp * run, end = min(pairs, begin + run);
+  if (warp < rows)
+    for (int p0 = begin; p0 < end; p0 += 32) {
+      const int p = p0 + lane;
+      const int e = p < end ? choice[p] : -1;
+      const unsigned same = __match_any_sync(0xffffffffu, e);
+      if (e >= 0 && lane == __ffs(same) - 1) mine[e] += __popc(same);
+      __syncwarp();
+    }
+  __syncthreads();
+  for (int e = threadIdx.x; e < experts; e += blockDim.x) {
+    int sum = 0;
+    for (int w = 0; w < rows; ++w) {
+      const int n = hist[w * experts + e];
+      hist[w * experts + e] = sum;
+      sum += n;
+    }
+    cnt[e] = sum;
   }
   __syncthreads();
-  // a pair's place within its expert's list: the pairs of an expert in ascending order (a fixed order,
-  // though no result depends on it)
-  for (int e = threadIdx.x; e < experts; e += blockDim.x) cnt[e] = 0;
+  if (warp == 0) group_offsets(cnt, experts, tiled, off, first, meta);
   __syncthreads();
-  if (pairs <= 4096) {
-    for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
-      const int e = choice[p];
-      int before = 0;
-      for (int q = 0; q < p; ++q) before += choice[q] == e;
-      order[off[e] + before] = p;
+  group_tiles(cnt, off, first, experts, tiled, tile_expert, tile_begin, tile_rows);
+  if (warp < rows)
+    for (int p0 = begin; p0 < end; p0 += 32) {
+      const int p = p0 + lane;
+      const int e = p < end ? choice[p] : -1;
+      const unsigned same = __match_any_sync(0xffffffffu, e);
+      if (e >= 0) order[off[e] + mine[e] + __popc(same & ((1u << lane) - 1))] = p;
+      __syncwarp();
+      if (e >= 0 && lane == __ffs(same) - 1) mine[e] += __popc(same);
+      __syncwarp();
     }
-  } else {
-    for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
-      const int e = choice[p];
-      order[off[e] + atomicAdd(&cnt[e], 1)] = p;
-    }
+}
+
+// Router and grouping of a step of few tokens in one CTA, a warp per token (float32 logits; every pair gets its
+// place as in moe_group_kernel).
+__global__ void __launch_bounds__(512)
+moe_route_group_kernel(const float* __restrict__ x, const RouteArgs a, int tiled, int32_t* choice, float* weight,
+                       int32_t* __restrict__ order, int32_t* __restrict__ tile_expert, int32_t* __restrict__ tile_begin,
+                       int32_t* __restrict__ tile_rows, int32_t* __restrict__ meta) {
+  pdl_launch();
+  pdl_wait();
+  extern __shared__ float sm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
+  const int per = 2 * a.experts + 2 * a.groups, pairs = a.tokens * a.top;
+  int32_t* chosen = reinterpret_cast<int32_t*>(sm + nwarps * per);      // [pairs], then [experts] counts, offsets, first tiles
+  int32_t* cnt = chosen + pairs;
+  int32_t* off = cnt + a.experts;
+  int32_t* first = off + a.experts;
+  for (int t = warp; t < a.tokens; t += nwarps) {
+    route_token<float, float>(a, x + static_cast<size_t>(t) * a.ld, nullptr, t, sm + warp * per, choice, weight);
+    __syncwarp();
+    for (int k = lane; k < a.top; k += 32) chosen[t * a.top + k] = choice[static_cast<size_t>(t) * a.top + k];
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < a.experts; e += blockDim.x) {
+    int n = 0;
+    for (int p = 0; p < pairs; ++p) n += chosen[p] == e;
+    cnt[e] = n;
+  }
+  __syncthreads();
+  if (warp == 0) group_offsets(cnt, a.experts, tiled, off, first, meta);
+  __syncthreads();
+  group_tiles(cnt, off, first, a.experts, tiled, tile_expert, tile_begin, tile_rows);
+  for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
+    const int e = chosen[p];
+    int before = 0;
+    for (int q = 0; q < p; ++q) before += chosen[q] == e;
+    order[off[e] + before] = p;
   }
 }
 
@@ -301,27 +396,36 @@ moe_gemm_simt_kernel(const TA* __restrict__ src, int ld_src, int src_div, const 
 }
 
 // The tile on the tensor cores for bfloat16: 64 pairs x 128 output features per CTA, eight warps in a
-// 2 x 4 grid (32 rows x 32 features each: 2 x 4 MMAs per 16 of k).  A (the pairs' rows) and W tiles of
-// 32 k go through shared memory as bfloat16; the next k block's 16-byte pieces are asked for before the
-// MMAs of the running one and stored after them.  mma.sync.m16n8k16, float32 accumulators, k ascending.
+// 2 x 4 grid (32 rows x 32 features each: 2 x 4 MMAs per 16 of k).  A (the pairs' rows) and W blocks of 64 k
+// come by asynchronous copies into a ring of three stages, two of which are on their way while the MMAs of the
+// third run; fragments by ldmatrix.  mma.sync.m16n8k16, float32 accumulators, k ascending.
 __device__ __forceinline__ void mma_bf16_16816(float* d, const uint32_t* a, const uint32_t* b) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
+__device__ __forceinline__ void ldmatrix4(uint32_t* r, unsigned addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+// 16 bytes on their way, or zeros
+__device__ __forceinline__ void async_piece(unsigned dst, const void* src, bool in) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(in ? 16 : 0));
+}
 
-constexpr int kMmaCols = 128;
+constexpr int kMmaCols = 128, kMmaK = 64, kMmaStages = 3, kMmaLd = kMmaK + 8;      // 144-byte rows: ldmatrix hits distinct banks
+constexpr int kMmaStage = (kTileRows + kMmaCols) * kMmaLd;                         // elements of a stage: A rows, then W rows
+constexpr int kMmaSmem = kMmaStages * kMmaStage * 2;
 
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 2)
 moe_gemm_mma_kernel(const bf16* __restrict__ src, int ld_src, int src_div, const bf16* __restrict__ w, int n, int k,
                     bf16* __restrict__ dst, int ld_dst, const int32_t* __restrict__ order,
                     const int32_t* __restrict__ tile_expert, const int32_t* __restrict__ tile_begin,
                     const int32_t* __restrict__ tile_rows, const int32_t* __restrict__ meta, int act) {
   pdl_launch();
   pdl_wait();
-  constexpr int BM = kTileRows, BN = kMmaCols, BK = 32, LD = BK + 8;      // 80-byte rows: fragment reads hit distinct banks
-  __shared__ __align__(16) bf16 As[BM][LD];
-  __shared__ __align__(16) bf16 Ws[BN][LD];
+  constexpr int BM = kTileRows, BN = kMmaCols, BK = kMmaK, LD = kMmaLd;
+  extern __shared__ __align__(16) bf16 ring[];
   __shared__ int32_t pair_of[BM];
   const int tile = blockIdx.x;
   if (tile >= meta[0]) return;
@@ -340,53 +444,65 @@ moe_gemm_mma_kernel(const bf16* __restrict__ src, int ld_src, int src_div, const
     for (int j = 0; j < 4; ++j)
 #pragma unroll
       for (int f = 0; f < 4; ++f) acc[i][j][f] = 0.f;
-  // this thread's pieces of a k block: one of A (64 rows x 4 pieces), two of W (128 rows x 4 pieces)
-  const int ar = threadIdx.x >> 2, ac = (threadIdx.x & 3) * 8;
-  const int ap = pair_of[ar];
-  const bf16* a_src = ap >= 0 ? src + static_cast<size_t>(ap / src_div) * ld_src + ac : nullptr;
-  const bf16* w_src[2];
+  // this thread's pieces of a k block: rows (tid / 8) + 32 i of A (i < 2) and of W (i < 4), piece tid % 8
+  const int pr = threadIdx.x >> 3, pc = (threadIdx.x & 7) * 8;
+  const bf16* a_src[2];
+  const bf16* w_src[4];
 #pragma unroll
-  for (int h = 0; h < 2; ++h) {
-    const int r = ar + h * 64;
-    w_src[h] = n0 + r < n ? we + static_cast<size_t>(n0 + r) * k + ac : nullptr;
+  for (int i = 0; i < 2; ++i) {
+    const int p = pair_of[pr + 32 * i];
+    a_src[i] = p >= 0 ? src + static_cast<size_t>(p / src_div) * ld_src + pc : nullptr;
   }
-  const uint4 zero = make_uint4(0, 0, 0, 0);
-  uint4 pa = zero, pw[2] = {zero, zero};
-  auto fetch = [&](int k0) {
-    const bool in = k0 + ac < k;
-    pa = (a_src != nullptr && in) ? *reinterpret_cast<const uint4*>(a_src + k0) : zero;
 #pragma unroll
-    for (int h = 0; h < 2; ++h) pw[h] = (w_src[h] != nullptr && in) ? *reinterpret_cast<const uint4*>(w_src[h] + k0) : zero;
+  for (int i = 0; i < 4; ++i) {
+    const int r = n0 + pr + 32 * i;
+    w_src[i] = r < n ? we + static_cast<size_t>(r) * k + pc : nullptr;
+  }
+  const unsigned base = static_cast<unsigned>(__cvta_generic_to_shared(ring));
+  auto fetch = [&](int stage, int k0) {
+    const unsigned at = base + static_cast<unsigned>(stage * kMmaStage + pr * LD + pc) * 2;
+    const bool in = k0 + pc < k;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const bool ok = in && a_src[i] != nullptr;
+      async_piece(at + 32 * i * LD * 2, ok ? a_src[i] + k0 : src, ok);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const bool ok = in && w_src[i] != nullptr;
+      async_piece(at + (BM + 32 * i) * LD * 2, ok ? w_src[i] + k0 : w, ok);
+    }
   };
-  fetch(0);
-  for (int k0 = 0; k0 < k; k0 += BK) {
-    __syncthreads();                                  // the block before has been read
-    *reinterpret_cast<uint4*>(&As[ar][ac]) = pa;
-    *reinterpret_cast<uint4*>(&Ws[ar][ac]) = pw[0];
-    *reinterpret_cast<uint4*>(&Ws[ar + 64][ac]) = pw[1];
-    __syncthreads();
-    if (k0 + BK < k) fetch(k0 + BK);                  // on its way while the MMAs run
+  const int blocks = (k + BK - 1) / BK;
+#pragma unroll
+  for (int s = 0; s < kMmaStages - 1; ++s) {
+    if (s < blocks) fetch(s, s * BK);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+  // where this lane's ldmatrix rows begin: A rows (16 x 16 tiles), W rows (two tiles of 8 features x 16 k)
+  const unsigned a_row = (wm * 32 + (lane & 15)) * LD + (lane >> 4) * 8;
+  const unsigned w_row = (BM + wn * 32 + (lane & 7) + (lane & 16 ? 8 : 0)) * LD + (lane & 8 ? 8 : 0);
+  int stage = 0;
+  for (int b = 0; b < blocks; ++b) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(kMmaStages - 2) : "memory");
+    __syncthreads();                                  // block b has arrived for all; block b - 1 has been read by all
+    const int ahead = b + kMmaStages - 1;
+    if (ahead < blocks) fetch(stage == 0 ? kMmaStages - 1 : stage - 1, ahead * BK);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    const unsigned at = base + static_cast<unsigned>(stage * kMmaStage) * 2;
 #pragma unroll
     for (int kk = 0; kk < BK; kk += 16) {
-      uint32_t b[4][2];
+      uint32_t fa[2][4], fb[2][4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const bf16* wr = &Ws[wn * 32 + j * 8 + gid][kk + tig * 2];
-        b[j][0] = *reinterpret_cast<const uint32_t*>(wr);
-        b[j][1] = *reinterpret_cast<const uint32_t*>(wr + 8);
-      }
+      for (int i = 0; i < 2; ++i) ldmatrix4(fa[i], at + (a_row + i * 16 * LD + kk) * 2);
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        uint32_t a[4];
-        const bf16* arow = &As[wm * 32 + i * 16 + gid][kk + tig * 2];
-        a[0] = *reinterpret_cast<const uint32_t*>(arow);
-        a[1] = *reinterpret_cast<const uint32_t*>(arow + 8 * LD);
-        a[2] = *reinterpret_cast<const uint32_t*>(arow + 8);
-        a[3] = *reinterpret_cast<const uint32_t*>(arow + 8 * LD + 8);
+      for (int j = 0; j < 2; ++j) ldmatrix4(fb[j], at + (w_row + j * 16 * LD + kk) * 2);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) mma_bf16_16816(acc[i][j], a, b[j]);
-      }
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) mma_bf16_16816(acc[i][j], fa[i], &fb[j >> 1][(j & 1) * 2]);
     }
+    stage = stage == kMmaStages - 1 ? 0 : stage + 1;
   }
 #pragma unroll
   for (int i = 0; i < 2; ++i)
@@ -409,25 +525,38 @@ moe_gemm_mma_kernel(const bf16* __restrict__ src, int ld_src, int src_div, const
     }
 }
 
+__device__ __forceinline__ uint4 stream16(const void* p) {
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  return v;
+}
+
 // For a handful of pairs (single-token steps) the products are bound by the stream of the chosen experts'
 // weights: one CTA per (tile, 16 output features), a warp takes four features at once and streams their
 // weight rows in 16-byte pieces, up to four of the tile's rows at a time (their input rows come from L1).
-template <typename T>
+// GATED: an expert has 2 n rows, gate rows and then up rows, and the result is act(gate) * up (two features and
+// their four rows at once; gate and up rounded to the activation type first, as when they are stored).
+template <typename T, bool GATED>
 __global__ void __launch_bounds__(128)
 moe_gemv_kernel(const T* __restrict__ src, int ld_src, int src_div, const T* __restrict__ w, int n, int k,
                 T* __restrict__ dst, int ld_dst, const int32_t* __restrict__ order,
                 const int32_t* __restrict__ tile_expert, const int32_t* __restrict__ tile_begin,
-                const int32_t* __restrict__ tile_rows, const int32_t* __restrict__ meta, int act) {
+                const int32_t* __restrict__ tile_rows, const int32_t* __restrict__ meta, int act, float limit,
+                float slope) {
   pdl_launch();
   pdl_wait();
-  constexpr int VEC = Vec16<T>::N, NF = 4, NR = 4;
+  constexpr int VEC = Vec16<T>::N, NF = 4, NR = 4, OF = GATED ? NF / 2 : NF;      // OF: output features of a warp
   const int tile = blockIdx.x;
   if (tile >= meta[0]) return;
   const int e = tile_expert[tile], begin = tile_begin[tile], rows = tile_rows[tile];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int f0 = blockIdx.y * 16 + warp * NF;
+  const int f0 = (blockIdx.y * 4 + warp) * OF;
   if (f0 >= n) return;
-  const T* we = w + static_cast<size_t>(e) * n * k;
+  const T* we = w + static_cast<size_t>(e) * (GATED ? 2 * n : n) * k;
+  const T* wr[NF];                               // (a feature beyond n: the last one's row, its result is not stored)
+#pragma unroll
+  for (int f = 0; f < NF; ++f)
+    wr[f] = we + (static_cast<size_t>(min(f0 + f % OF, n - 1)) + (f >= OF ? n : 0)) * k;
   const bool vec = (k % VEC == 0) && (ld_src % VEC == 0) && (reinterpret_cast<uintptr_t>(src) % 16 == 0) &&
                    (reinterpret_cast<uintptr_t>(w) % 16 == 0);
   for (int r0 = 0; r0 < rows; r0 += NR) {
@@ -445,16 +574,19 @@ moe_gemv_kernel(const T* __restrict__ src, int ld_src, int src_div, const T* __r
 #pragma unroll
       for (int r = 0; r < NR; ++r) acc[f][r] = 0.f;
     if (vec) {
-      for (int c = lane * VEC; c < k; c += 32 * VEC) {
+      // (the next pieces of the weight rows are asked for before the sums over the present ones)
+      uint4 cur[NF];
+      int c = lane * VEC;
+#pragma unroll
+      for (int f = 0; f < NF; ++f) cur[f] = c < k ? stream16(wr[f] + c) : make_uint4(0, 0, 0, 0);
+      for (; c < k; c += 32 * VEC) {
+        uint4 nxt[NF];
+        const int cn = c + 32 * VEC;
+#pragma unroll
+        for (int f = 0; f < NF; ++f) nxt[f] = cn < k ? stream16(wr[f] + cn) : make_uint4(0, 0, 0, 0);
         float wv[NF][VEC];
 #pragma unroll
-        for (int f = 0; f < NF; ++f) {
-          if (f0 + f < n) load16(we + static_cast<size_t>(f0 + f) * k + c, wv[f]);
-          else {
-#pragma unroll
-            for (int i = 0; i < VEC; ++i) wv[f][i] = 0.f;
-          }
-        }
+        for (int f = 0; f < NF; ++f) load16(reinterpret_cast<const T*>(&cur[f]), wv[f]);
 #pragma unroll
         for (int r = 0; r < NR; ++r) {
           if (r < nr) {
@@ -466,6 +598,8 @@ moe_gemv_kernel(const T* __restrict__ src, int ld_src, int src_div, const T* __r
               for (int i = 0; i < VEC; ++i) acc[f][r] = fmaf(wv[f][i], xv[i], acc[f][r]);
           }
         }
+#pragma unroll
+        for (int f = 0; f < NF; ++f) cur[f] = nxt[f];
       }
     } else {
       for (int c = lane; c < k; c += 32) {
@@ -474,17 +608,28 @@ moe_gemv_kernel(const T* __restrict__ src, int ld_src, int src_div, const T* __r
           const float xv = r < nr ? to_float(xr[r][c]) : 0.f;
 #pragma unroll
           for (int f = 0; f < NF; ++f)
-            if (f0 + f < n) acc[f][r] = fmaf(to_float(we[static_cast<size_t>(f0 + f) * k + c]), xv, acc[f][r]);
+            acc[f][r] = fmaf(to_float(wr[f][c]), xv, acc[f][r]);
         }
       }
     }
 #pragma unroll
-    for (int f = 0; f < NF; ++f)
+    for (int f = 0; f < OF; ++f)
 #pragma unroll
       for (int r = 0; r < NR; ++r) {
-        const float v = warp_sum(acc[f][r]);
-        if (lane == 0 && r < nr && f0 + f < n)
-          dst[static_cast<size_t>(pair[r]) * ld_dst + f0 + f] = from_float<T>(moe_activate(v, act));
+        float v = warp_sum(acc[f][r]);
+        if (GATED) {
+          const float up = to_float(from_float<T>(warp_sum(acc[f + NF - OF][r])));
+          v = to_float(from_float<T>(v));
+          if (act == ACT_CLAMPED_SWISH) {
+            const float g = fminf(v, limit);
+            v = g / (1.f + expf(-slope * g)) * (fminf(fmaxf(up, -limit), limit) + 1.f);
+          } else {
+            v = moe_activate(v, act) * up;
+          }
+        } else {
+          v = moe_activate(v, act);
+        }
+        if (lane == 0 && r < nr && f0 + f < n) dst[static_cast<size_t>(pair[r]) * ld_dst + f0 + f] = from_float<T>(v);
       }
   }
 }
@@ -529,10 +674,11 @@ int rl_moe_route(const void* x, int act_dtype, int ld, const void* router, int w
   const int warps = 4;
   const size_t smem = static_cast<size_t>(warps) * (2 * experts + 2 * groups) * sizeof(float);
   dim3 grid((tokens + warps - 1) / warps), block(warps * 32);
+  const RouteArgs a{ld, tokens, width, experts, groups, keep, group_top, top, softmax, renorm, bias, choice_bias,
+                    weight_scale, renorm_floor};
 #define RL_CASE(TA, TW)                                                                                            \
-  launch_kernel(moe_route_kernel<TA, TW>, grid, block, smem, stream, static_cast<const TA*>(x), ld,                \
-                static_cast<const TW*>(router), tokens, width, experts, groups, keep, group_top, top, softmax,     \
-                renorm, bias, choice_bias, weight_scale, renorm_floor, choice, weight)
+  launch_kernel(moe_route_kernel<TA, TW>, grid, block, smem, stream, static_cast<const TA*>(x),                    \
+                static_cast<const TW*>(router), a, choice, weight)
   if (act_dtype == 0) RL_CASE(float, float);
   else if (w_dtype == 0) RL_CASE(bf16, float);
   else RL_CASE(bf16, bf16);
@@ -540,31 +686,58 @@ int rl_moe_route(const void* x, int act_dtype, int ld, const void* router, int w
   RL_LAUNCH_END();
 }
 
+// Router (from float32 logits) and grouping in one launch; tokens * top at most 256.
+int rl_moe_route_group(const float* logits, int ld, int tokens, int experts, int groups, int keep, int group_top, int top,
+                       int softmax, int renorm, const float* bias, const float* choice_bias, float weight_scale,
+                       float renorm_floor, int tiled, int32_t* choice, float* weight, int32_t* order,
+                       int32_t* tile_expert, int32_t* tile_begin, int32_t* tile_rows, int32_t* meta,
+                       cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (tokens * top > 256) return static_cast<int>(cudaErrorInvalidValue);
+  const int warps = max(4, min(16, tokens));
+  const size_t smem = (static_cast<size_t>(warps) * (2 * experts + 2 * groups) + tokens * top + 3 * experts) * sizeof(float);
+  if (smem > 48 * 1024) return static_cast<int>(cudaErrorInvalidValue);
+  const RouteArgs a{ld, tokens, 0, experts, groups, keep, group_top, top, softmax, renorm, bias, choice_bias,
+                    weight_scale, renorm_floor};
+  launch_kernel(moe_route_group_kernel, dim3(1), dim3(warps * 32), smem, stream, logits, a, tiled, choice, weight, order,
+                tile_expert, tile_begin, tile_rows, meta);
+  RL_LAUNCH_END();
+}
+
 int rl_moe_group(const int32_t* choice, int pairs, int experts, int tiled, int32_t* order, int32_t* tile_expert,
                  int32_t* tile_begin, int32_t* tile_rows, int32_t* meta, cudaStream_t stream) {
   if (pairs <= 0) return 0;
-  launch_kernel(moe_group_kernel, dim3(1), dim3(256), (2 * experts + 1) * sizeof(int32_t), stream, choice, pairs,
-                experts, tiled, order, tile_expert, tile_begin, tile_rows, meta);
+  // as many runs as there are warps' worth of pairs and as fit 48 KB of counters
+  int rows = max(1, min(kGroupThreads / 32, (pairs + 31) / 32));
+  while (rows > 1 && (3 + rows) * experts * sizeof(int32_t) > 48 * 1024) rows /= 2;
+  const size_t smem = (3 + static_cast<size_t>(rows)) * experts * sizeof(int32_t);
+  if (smem > 48 * 1024) return static_cast<int>(cudaErrorInvalidValue);
+  launch_kernel(moe_group_kernel, dim3(1), dim3(min(kGroupThreads, max(128, rows * 32))), smem, stream, choice, pairs,
+                experts, tiled, rows, order, tile_expert, tile_begin, tile_rows, meta);
   RL_LAUNCH_END();
 }
 
 // max_tiles: the most tiles the grouping can have made (pairs / 64 + experts); CTAs beyond the real
-// number leave at once.  few_pairs: the weight-streaming kernel for a handful of pairs (single-token steps).
+// number leave at once.  few_pairs: the weight-streaming kernel for a handful of pairs (single-token steps), which
+// can also form act(gate) * up from an expert's 2 n rows (gated).
 int rl_moe_gemm(int act_dtype, const void* src, int ld_src, int src_div, const void* w, int n, int k, void* dst,
                 int ld_dst, const int32_t* order, const int32_t* tile_expert, const int32_t* tile_begin,
-                const int32_t* tile_rows, const int32_t* meta, int max_tiles, int few_pairs, int act,
-                cudaStream_t stream) {
+                const int32_t* tile_rows, const int32_t* meta, int max_tiles, int few_pairs, int act, int gated,
+                float limit, float slope, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
+  if (gated && !few_pairs) return static_cast<int>(cudaErrorInvalidValue);
   if (few_pairs) {
-    dim3 g(max_tiles, (n + 15) / 16);
-    if (act_dtype == 0)
-      launch_kernel(moe_gemv_kernel<float>, g, dim3(128), 0, stream, static_cast<const float*>(src), ld_src, src_div,
-                    static_cast<const float*>(w), n, k, static_cast<float*>(dst), ld_dst, order, tile_expert, tile_begin,
-                    tile_rows, meta, act);
-    else
-      launch_kernel(moe_gemv_kernel<bf16>, g, dim3(128), 0, stream, static_cast<const bf16*>(src), ld_src, src_div,
-                    static_cast<const bf16*>(w), n, k, static_cast<bf16*>(dst), ld_dst, order, tile_expert, tile_begin,
-                    tile_rows, meta, act);
+    dim3 g(max_tiles, (n + (gated ? 7 : 15)) / (gated ? 8 : 16));
+#define RL_CASE(T, G)                                                                                              \
+  launch_kernel(moe_gemv_kernel<T, G>, g, dim3(128), 0, stream, static_cast<const T*>(src), ld_src, src_div,      \
+                static_cast<const T*>(w), n, k, static_cast<T*>(dst), ld_dst, order, tile_expert, tile_begin,     \
+                tile_rows, meta, act, limit, slope)
+    if (act_dtype == 0) {
+      if (gated) RL_CASE(float, true); else RL_CASE(float, false);
+    } else {
+      if (gated) RL_CASE(bf16, true); else RL_CASE(bf16, false);
+    }
+#undef RL_CASE
     RL_LAUNCH_END();
   }
   dim3 grid(max_tiles, (n + 63) / 64);
@@ -574,7 +747,13 @@ int rl_moe_gemm(int act_dtype, const void* src, int ld_src, int src_div, const v
                   tile_expert, tile_begin, tile_rows, meta, act);
   } else if (k % 8 == 0 && ld_src % 8 == 0 && (reinterpret_cast<uintptr_t>(src) % 16 == 0) &&
              (reinterpret_cast<uintptr_t>(w) % 16 == 0)) {
-    launch_kernel(moe_gemm_mma_kernel, dim3(max_tiles, (n + kMmaCols - 1) / kMmaCols), dim3(256), 0, stream,
+    static bool raised = false;
+    if (!raised) {
+      const cudaError_t e = cudaFuncSetAttribute(moe_gemm_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kMmaSmem);
+      if (e != cudaSuccess) return static_cast<int>(e);
+      raised = true;
+    }
+    launch_kernel(moe_gemm_mma_kernel, dim3(max_tiles, (n + kMmaCols - 1) / kMmaCols), dim3(256), kMmaSmem, stream,
                   static_cast<const bf16*>(src), ld_src, src_div,
                   static_cast<const bf16*>(w), n, k, static_cast<bf16*>(dst), ld_dst, order, tile_expert, tile_begin,
                   tile_rows, meta, act);

@@ -186,14 +186,26 @@ __global__ void sandwich_norm_reg_kernel(float* __restrict__ residual, const TA*
 // normed, out is the stream row as it is.  w float32 [hidden]; scale float32 [hidden] or null (ones).
 // The row lives in registers, NV pieces of four neighbouring elements per thread (VEC: rows start on 16-byte
 // boundaries and hidden is a multiple of 4; else the elements are handled one by one).
+// The output may also come as its terms (mix.top > 0): delta then holds top rows per stream row, and
+//   delta_r = sum_k weight[r, k] * rows[r * top + k] (+ shared[r], times sigmoid(gate_r) where gate is given)
+// in float32, k in order.
+template <typename TA>
+struct RowMix {
+  int top;
+  const float* weight;       // [rows, top]
+  const TA* shared;          // [rows, hidden] or null
+  const float* gate;         // a column of a float32 buffer, or null
+  int ld_gate;
+};
+
 template <typename TA, int NV, bool VEC>
 __global__ void sum_norm_kernel(float* __restrict__ residual, const TA* __restrict__ delta, int ld_delta,
                                 const float* __restrict__ w, const float* __restrict__ scale, float alpha, float eps,
-                                TA* __restrict__ out, int ld_out, int hidden) {
+                                TA* __restrict__ out, int ld_out, int hidden, const RowMix<TA> mix) {
   __shared__ float scratch[32];
   const int r = blockIdx.x;
   float* res = residual + static_cast<size_t>(r) * hidden;
-  const TA* d = delta != nullptr ? delta + static_cast<size_t>(r) * ld_delta : nullptr;
+  const TA* d = delta != nullptr ? delta + static_cast<size_t>(r) * max(mix.top, 1) * ld_delta : nullptr;
   // (weights come from no earlier kernel of the step: asked for before the wait)
   float wv[NV][4], sv[NV][4], v[NV][4];
   auto piece = [&](int i) { return (threadIdx.x + i * blockDim.x) * 4; };
@@ -219,22 +231,41 @@ __global__ void sum_norm_kernel(float* __restrict__ residual, const TA* __restri
   }
   pdl_launch();
   pdl_wait();
+  const TA* sh = mix.top > 0 && mix.shared != nullptr ? mix.shared + static_cast<size_t>(r) * hidden : nullptr;
+  const float sg = sh != nullptr && mix.gate != nullptr ? 1.f / (1.f + expf(-mix.gate[static_cast<size_t>(r) * mix.ld_gate])) : 1.f;
   float q = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int c = piece(i);
     float dv[4] = {0.f, 0.f, 0.f, 0.f};
+    if (mix.top > 0) {
+      auto add = [&](const TA* row, float weight) {
+        float x[4] = {0.f, 0.f, 0.f, 0.f};
+        if (VEC) {
+          if (c < hidden) load4(row + c, x);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            if (c + j < hidden) x[j] = to_float(row[c + j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) dv[j] = fmaf(weight, x[j], dv[j]);
+      };
+#pragma unroll 4
+      for (int k = 0; k < mix.top; ++k) add(d + static_cast<size_t>(k) * ld_delta, mix.weight[static_cast<size_t>(r) * mix.top + k]);
+      if (sh != nullptr) add(sh, sg);
+    }
     if (VEC) {
       if (c < hidden) {
         load4(res + c, v[i]);
-        if (d != nullptr) load4(d + c, dv);
+        if (d != nullptr && mix.top == 0) load4(d + c, dv);
       }
     } else {
 #pragma unroll
       for (int j = 0; j < 4; ++j)
         if (c + j < hidden) {
           v[i][j] = res[c + j];
-          if (d != nullptr) dv[j] = to_float(d[c + j]);
+          if (d != nullptr && mix.top == 0) dv[j] = to_float(d[c + j]);
         }
     }
     if (d != nullptr) {
@@ -306,6 +337,55 @@ __global__ void act_cast_kernel(const float* __restrict__ x, TA* __restrict__ y,
   pdl_wait();
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i < n) y[i] = from_float<TA>(activate(x[i], mode));
+}
+
+// ------------------------------------------------ z[r, n] = sum_j w[n, j] * act(x[r, j]), few rows
+// The second of two products with a small size between them: x float32 [rows, rank], the activated entries
+// rounded to the activation type TA, float32 sums and result.  A thread per output feature, all rows at once.
+constexpr int kLowRows = 16, kLowThreads = 128;
+template <typename TA>
+__global__ void __launch_bounds__(kLowThreads)
+low_rank_kernel(const float* __restrict__ x, const TA* __restrict__ w, float* __restrict__ z, int rows, int n, int rank,
+                int mode) {
+  extern __shared__ float xs[];              // [rank][kLowRows]
+  pdl_launch();
+  pdl_wait();
+  for (int i = threadIdx.x; i < rank * kLowRows; i += kLowThreads) {
+    const int j = i / kLowRows, r = i % kLowRows;
+    xs[i] = r < rows ? to_float(from_float<TA>(activate(x[static_cast<size_t>(r) * rank + j], mode))) : 0.f;
+  }
+  __syncthreads();
+  const int f = blockIdx.x * kLowThreads + threadIdx.x;
+  if (f >= n) return;
+  float acc[kLowRows];
+#pragma unroll
+  for (int r = 0; r < kLowRows; ++r) acc[r] = 0.f;
+  const TA* row = w + static_cast<size_t>(f) * rank;
+  auto add = [&](int j, float wv) {
+    const float4* p = reinterpret_cast<const float4*>(xs + j * kLowRows);
+#pragma unroll
+    for (int q = 0; q < kLowRows / 4; ++q) {
+      const float4 v = p[q];
+      acc[4 * q] = fmaf(wv, v.x, acc[4 * q]);
+      acc[4 * q + 1] = fmaf(wv, v.y, acc[4 * q + 1]);
+      acc[4 * q + 2] = fmaf(wv, v.z, acc[4 * q + 2]);
+      acc[4 * q + 3] = fmaf(wv, v.w, acc[4 * q + 3]);
+    }
+  };
+  constexpr int VEC = Vec16<TA>::N;
+  if (rank % VEC == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0) {
+    for (int j = 0; j < rank; j += VEC) {
+      float v[VEC];
+      load16(row + j, v);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) add(j + i, v[i]);
+    }
+  } else {
+    for (int j = 0; j < rank; ++j) add(j, to_float(row[j]));
+  }
+#pragma unroll
+  for (int r = 0; r < kLowRows; ++r)
+    if (r < rows) z[static_cast<size_t>(r) * n + f] = acc[r];
 }
 
 // ------------------------------------------------ cache[page, head, offset, :] = src[t, col + head * dim : ...]
@@ -590,9 +670,10 @@ int rl_sandwich_norm(float* residual, const void* delta, int ld_delta, const voi
   RL_LAUNCH_END();
 }
 
-// Rows of up to 16 x 1,024 elements (cudaErrorInvalidValue beyond).
+// Rows of up to 16 x 1,024 elements (cudaErrorInvalidValue beyond).  top > 0: the output comes as its terms (RowMix).
 int rl_sum_norm(float* residual, const void* delta, int ld_delta, const float* w, const float* scale, float alpha,
-                float eps, void* out, int ld_out, int act_dtype, int rows, int hidden, cudaStream_t stream) {
+                float eps, void* out, int ld_out, int act_dtype, int rows, int hidden, int top, const float* mix_weight,
+                const void* shared, const float* gate, int ld_gate, cudaStream_t stream) {
   if (rows <= 0) return 0;
   const int pieces = (hidden + 3) / 4, nv = pieces <= 1024 ? 1 : (pieces <= 2048 ? 2 : 4);
   if (pieces > 4096) return static_cast<int>(cudaErrorInvalidValue);
@@ -600,15 +681,17 @@ int rl_sum_norm(float* residual, const void* delta, int ld_delta, const float* w
   const size_t act = act_dtype == RL_F32 ? 16 : 8;
   const bool vec = hidden % 4 == 0 && ld_delta % 4 == 0 && ld_out % 4 == 0 && reinterpret_cast<uintptr_t>(residual) % 16 == 0 &&
                    reinterpret_cast<uintptr_t>(w) % 16 == 0 && reinterpret_cast<uintptr_t>(scale) % 16 == 0 &&
-                   reinterpret_cast<uintptr_t>(delta) % act == 0 && reinterpret_cast<uintptr_t>(out) % act == 0;
+                   reinterpret_cast<uintptr_t>(delta) % act == 0 && reinterpret_cast<uintptr_t>(out) % act == 0 &&
+                   reinterpret_cast<uintptr_t>(shared) % act == 0;
 #define RL_CASE(TA, NV)                                                                                            \
   do {                                                                                                             \
+    const RowMix<TA> mix{top, mix_weight, static_cast<const TA*>(shared), gate, ld_gate};                          \
     if (vec) launch_kernel(sum_norm_kernel<TA, NV, true>, dim3(rows), dim3(th), 0, stream, residual,               \
                            static_cast<const TA*>(delta), ld_delta, w, scale, alpha, eps, static_cast<TA*>(out),   \
-                           ld_out, hidden);                                                                        \
+                           ld_out, hidden, mix);                                                                   \
     else launch_kernel(sum_norm_kernel<TA, NV, false>, dim3(rows), dim3(th), 0, stream, residual,                  \
                        static_cast<const TA*>(delta), ld_delta, w, scale, alpha, eps, static_cast<TA*>(out),       \
-                       ld_out, hidden);                                                                            \
+                       ld_out, hidden, mix);                                                                       \
   } while (0)
   if (act_dtype == RL_F32) {
     if (nv == 1) RL_CASE(float, 1); else if (nv == 2) RL_CASE(float, 2); else RL_CASE(float, 4);
@@ -638,6 +721,19 @@ int rl_act_cast(const float* x, void* y, int act_dtype, int n, int mode, cudaStr
   const dim3 grid((n + 255) / 256);
   if (act_dtype == RL_F32) launch_kernel(act_cast_kernel<float>, grid, dim3(256), 0, stream, x, static_cast<float*>(y), n, mode);
   else launch_kernel(act_cast_kernel<bf16>, grid, dim3(256), 0, stream, x, static_cast<bf16*>(y), n, mode);
+  RL_LAUNCH_END();
+}
+
+int rl_low_rank(const float* x, const void* w, int w_dtype, float* z, int rows, int n, int rank, int mode,
+                cudaStream_t stream) {
+  if (rows <= 0 || n <= 0) return 0;
+  const size_t smem = static_cast<size_t>(rank) * kLowRows * sizeof(float);
+  if (rows > kLowRows || smem > 48 * 1024) return static_cast<int>(cudaErrorInvalidValue);
+  const dim3 grid((n + kLowThreads - 1) / kLowThreads);
+  if (w_dtype == RL_F32)
+    launch_kernel(low_rank_kernel<float>, grid, dim3(kLowThreads), smem, stream, x, static_cast<const float*>(w), z, rows, n, rank, mode);
+  else
+    launch_kernel(low_rank_kernel<bf16>, grid, dim3(kLowThreads), smem, stream, x, static_cast<const bf16*>(w), z, rows, n, rank, mode);
   RL_LAUNCH_END();
 }
 

@@ -24,7 +24,9 @@ from typing import Dict, Iterable, List, Optional, Tuple
 
 CSRC = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "csrc")
 ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
-BASE_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--shared", "-Xcompiler", "-fPIC"]
+# (-fno-gnu-unique: one source becomes several modules, and a static of a template or inline function, a "limit
+# already raised" say, must be each module's own; GNU unique symbols would be one for all of them)
+BASE_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--shared", "-Xcompiler", "-fPIC", "-Xcompiler", "-fno-gnu-unique"]
 
 _lock = threading.Lock()
 _build_dir: Optional[str] = None

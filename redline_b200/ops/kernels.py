@@ -260,6 +260,28 @@ def gemm_skinny(w: torch.Tensor, y: torch.Tensor, epilogue: int, rows: int, x: O
            "gemm_skinny")
 
 
+def gemm_skinny_grouped_ok(rows: int, x: torch.Tensor, w: torch.Tensor, group: int) -> bool:
+    """Whether gemm_skinny_grouped takes these products: at most 8 rows, bfloat16, groups of a multiple of 16
+    features, K a multiple of 8, 16-byte aligned rows."""
+    return (rows <= SKINNY_UNSTAGED_ROWS and skinny_ok(rows, w, x.dtype) and group % 16 == 0 and x.stride(2) == 1
+            and x.stride(1) % 8 == 0 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
+            and x.stride(0) * x.shape[0] < 2 ** 31)
+
+
+def gemm_skinny_grouped(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, rows: int, group: int) -> None:
+    """Several products of at most 8 rows as one launch: y[r, n] = sum_k w[n, k] * x[n // group, r, k]; x bfloat16
+    [groups, *, K], w [N, K], y bfloat16 [*, N]."""
+    _need_cuda(x, w, y)
+    N, K = w.shape
+    if not gemm_skinny_grouped_ok(rows, x, w, group) or x.shape[2] != K or (N + group - 1) // group > x.shape[0] \
+            or y.dtype != torch.bfloat16 or y.shape[1] != N or y.stride(1) != 1:
+        raise KernelError(f"gemm_skinny_grouped: shapes x{tuple(x.shape)} w{tuple(w.shape)} y{tuple(y.shape)}")
+    f = _fn(_lib("gemm_skinny", "gemm_skinny.cu"), "rl_gemm_skinny_grouped",
+            [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(w), _ptr(x), x.stride(1), group, x.stride(0), _ptr(y), y.stride(0), rows, N, K, sm_count(w.device),
+             _stream()), "gemm_skinny_grouped")
+
+
 # ------------------------------------------------------------ tcgen05 gemm
 
 _tc_status: Dict[int, torch.Tensor] = {}
@@ -615,10 +637,18 @@ SUM_NORM_MAX_WIDTH = 16384
 
 def sum_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: Optional[torch.Tensor],
              scale: Optional[torch.Tensor], alpha: float, eps: float, out: Optional[torch.Tensor],
-             rows: Optional[int] = None) -> None:
+             rows: Optional[int] = None, top: int = 0, mix_weight: Optional[torch.Tensor] = None,
+             shared: Optional[torch.Tensor] = None, shared_gate: Optional[torch.Tensor] = None) -> None:
     """residual (float32 stream) = rmsnorm(alpha * residual + scale * delta) * weight, out = the new rows in out's
-    type (out given); without ``delta`` only the copy.  weight and scale float32 [width] (scale None: ones)."""
-    _need_cuda(residual, delta, weight, scale, out)
+    type (out given); without ``delta`` only the copy.  weight and scale float32 [width] (scale None: ones).
+    With ``top`` the sublayer's output comes as its terms: delta holds ``top`` rows per stream row, weighed by
+    ``mix_weight`` (float32 [rows * top]) and summed in float32, plus ``shared`` (times sigmoid(shared_gate)): what
+    ``moe_combine`` makes, without the rounding in between."""
+    _need_cuda(residual, delta, weight, scale, out, mix_weight, shared, shared_gate)
+    if top > 0 and (delta is None or mix_weight is None or mix_weight.dtype != torch.float32 or delta.shape[0] < (
+            rows if rows is not None else residual.shape[0]) * top or (shared is not None and (
+                shared.dtype != delta.dtype or not shared.is_contiguous()))):
+        raise KernelError("sum_norm: the terms come with float32 weights, top rows each, a contiguous shared output")
     n = rows if rows is not None else residual.shape[0]
     act = out if out is not None else delta
     if act is None:
@@ -634,10 +664,11 @@ def sum_norm(residual: torch.Tensor, delta: Optional[torch.Tensor], weight: Opti
             or (delta is not None and out is not None and delta.dtype != out.dtype):
         raise KernelError("sum_norm: delta (with a weight) and out have one type and contiguous rows")
     f = _fn(_rw(), "rl_sum_norm", [c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_void_p, c_int, c_int,
-                                   c_int, c_int, c_void_p])
+                                   c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
     _check(f(_ptr(residual), _ptr(delta), delta.stride(0) if delta is not None else 0, _ptr(weight), _ptr(scale),
              float(alpha), float(eps), _ptr(out), out.stride(0) if out is not None else 0, _code(act.dtype), n, width,
-             _stream()), "sum_norm")
+             top, _ptr(mix_weight) if top else None, _ptr(shared) if top else None, _ptr(shared_gate) if top else None,
+             shared_gate.stride(0) if shared_gate is not None else 0, _stream()), "sum_norm")
 
 
 def bias_act(x: torch.Tensor, bias: Optional[torch.Tensor], act: int, cols: Optional[int] = None,
@@ -660,6 +691,21 @@ def act_cast(x: torch.Tensor, y: torch.Tensor, act: int) -> None:
         raise KernelError("act_cast: a contiguous float32 tensor and a contiguous output of its size")
     f = _fn(_rw(), "rl_act_cast", [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
     _check(f(_ptr(x), _ptr(y), _code(y.dtype), x.numel(), act, _stream()), "act_cast")
+
+
+LOW_RANK_ROWS, LOW_RANK_MAX = 16, 512
+
+
+def low_rank(x: torch.Tensor, w: torch.Tensor, z: torch.Tensor, act: int) -> None:
+    """z[r, n] = sum_j w[n, j] * act(x[r, j]) for at most LOW_RANK_ROWS rows of a small size (LOW_RANK_MAX): x and z
+    float32, the activated entries rounded to w's type first."""
+    _need_cuda(x, w, z)
+    if x.dtype != torch.float32 or z.dtype != torch.float32 or not x.is_contiguous() or not z.is_contiguous() \
+            or not w.is_contiguous() or w.shape != (z.shape[1], x.shape[1]) or x.shape[0] > LOW_RANK_ROWS \
+            or x.shape[1] > LOW_RANK_MAX or z.shape[0] != x.shape[0]:
+        raise KernelError(f"low_rank: shapes x{tuple(x.shape)} w{tuple(w.shape)} z{tuple(z.shape)}")
+    f = _fn(_rw(), "rl_low_rank", [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(x), _ptr(w), _code(w.dtype), _ptr(z), x.shape[0], z.shape[1], x.shape[1], act, _stream()), "low_rank")
 
 
 def cache_store(src: torch.Tensor, col: int, heads: int, dim: int, slots: torch.Tensor, cache: torch.Tensor,
@@ -905,9 +951,13 @@ def latent_prep(q: Optional[torch.Tensor], latent: Optional[torch.Tensor], posit
 
 
 def head_linear(x: torch.Tensor, x_col: int, x_head: int, w: torch.Tensor, y: torch.Tensor, y_col: int, y_head: int,
-                tokens: Optional[int] = None, impl: int = 0) -> None:
+                tokens: Optional[int] = None, impl: int = 0, turn: Optional[Tuple] = None) -> None:
     """y[t, y_col + h * y_head + j] = sum_k w[h, j, k] * x[t, x_col + h * x_head + k] for every head h:
-    w [heads, n, k]; float32 sums in ascending k.  impl 1: CUDA cores also where the tensor cores apply."""
+    w [heads, n, k]; float32 sums.  impl 0: a kernel for at most 16 tokens, tensor cores or CUDA cores, whichever
+    fits; 1: CUDA cores; 2: tensor cores where they apply.
+    ``turn`` = (entries, first of them in x's head, in y's head, cos, sin, positions, pairs, status): that part of
+    every head's row of x goes to y's turned by the token's position, the first 2 * cos.shape[1] entries as in
+    ``latent_prep``."""
     _need_cuda(x, w, y)
     heads, n, k = w.shape
     if x.dtype != y.dtype or x.stride(1) != 1 or y.stride(1) != 1 or not w.is_contiguous() \
@@ -915,10 +965,21 @@ def head_linear(x: torch.Tensor, x_col: int, x_head: int, w: torch.Tensor, y: to
         raise KernelError("head_linear: x and y have one type and contiguous rows; w contiguous [heads, n, k]")
     if x_col + (heads - 1) * x_head + k > x.shape[1] or y_col + (heads - 1) * y_head + n > y.shape[1]:
         raise KernelError("head_linear: the heads do not fit the rows")
+    dims = rot = tx = ty = max_pos = pairs = 0
+    cos = sin = positions = status = None
+    if turn is not None:
+        dims, tx, ty, cos, sin, positions, pairs, status = turn
+        rot, max_pos = 2 * cos.shape[1], cos.shape[0]
+        _need_cuda(cos, sin, positions, status)
+        if rot > dims or cos.dtype != torch.float32 or not cos.is_contiguous() or not sin.is_contiguous() \
+                or x_col + (heads - 1) * x_head + tx + dims > x.shape[1] or y_col + (heads - 1) * y_head + ty + dims > y.shape[1]:
+            raise KernelError("head_linear: the rotated parts do not fit the rows, or their tables the parts")
     f = _fn(_latent(), "rl_head_linear", [c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int,
-                                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p])
+                                          c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                                          c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p])
     _check(f(_code(x.dtype), _code(w.dtype), _ptr(x), x.stride(0), x_col, x_head, _ptr(w), heads, n, k, _ptr(y),
-             y.stride(0), y_col, y_head, tokens if tokens is not None else x.shape[0], impl, _stream()), "head_linear")
+             y.stride(0), y_col, y_head, tokens if tokens is not None else x.shape[0], impl, dims, rot, 1 if pairs else 0, tx,
+             ty, _ptr(cos), _ptr(sin), max_pos, _ptr(positions), _ptr(status), _stream()), "head_linear")
 
 
 # ------------------------------------------------------- linear attention with a decaying state
@@ -1310,6 +1371,32 @@ def moe_route(x: torch.Tensor, router: Optional[torch.Tensor], choice: torch.Ten
            "moe_route")
 
 
+MOE_ROUTE_GROUP_PAIRS = 256
+
+
+def moe_route_group(logits: torch.Tensor, choice: torch.Tensor, weight: torch.Tensor, tokens: int, groups: int, keep: int,
+                    group_top: int, top: int, order: torch.Tensor, tile_expert: torch.Tensor, tile_begin: torch.Tensor,
+                    tile_rows: torch.Tensor, meta: torch.Tensor, softmax: bool = False, renorm: bool = False,
+                    bias: Optional[torch.Tensor] = None, choice_bias: Optional[torch.Tensor] = None,
+                    weight_scale: float = 1.0, renorm_floor: float = 0.0, tiled: Optional[int] = None) -> None:
+    """``moe_route`` from float32 logits and ``moe_group`` in one launch, for up to MOE_ROUTE_GROUP_PAIRS pairs."""
+    _need_cuda(logits, choice, weight, order, tile_expert, tile_begin, tile_rows, meta, bias, choice_bias)
+    experts = logits.shape[1]
+    for t in (bias, choice_bias):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or t.numel() != experts):
+            raise KernelError("moe_route_group: biases are contiguous float32 [experts]")
+    if logits.dtype != torch.float32 or logits.stride(1) != 1 or experts % max(groups, 1) != 0 \
+            or choice.dtype != torch.int32 or weight.dtype != torch.float32 or tokens * top > MOE_ROUTE_GROUP_PAIRS:
+        raise KernelError("moe_route_group: float32 logits of few tokens; choice int32, weight float32")
+    f = _fn(_moe(), "rl_moe_route_group", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                                            c_void_p, c_float, c_float, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                                            c_void_p, c_void_p, c_void_p, c_void_p])
+    _check(f(_ptr(logits), logits.stride(0), tokens, experts, max(groups, 1), keep, group_top, top, 1 if softmax else 0,
+             1 if renorm else 0, _ptr(bias), _ptr(choice_bias), float(weight_scale), float(renorm_floor),
+             experts if tiled is None else tiled, _ptr(choice), _ptr(weight), _ptr(order), _ptr(tile_expert),
+             _ptr(tile_begin), _ptr(tile_rows), _ptr(meta), _stream()), "moe_route_group")
+
+
 def moe_group(choice: torch.Tensor, pairs: int, experts: int, order: torch.Tensor, tile_expert: torch.Tensor,
               tile_begin: torch.Tensor, tile_rows: torch.Tensor, meta: torch.Tensor, tiled: Optional[int] = None) -> None:
     """Lists the (token, slot) pairs expert by expert (``order``) and cuts every expert's list into tiles of
@@ -1324,22 +1411,28 @@ def moe_group(choice: torch.Tensor, pairs: int, experts: int, order: torch.Tenso
 
 def moe_gemm(src: torch.Tensor, src_div: int, w: torch.Tensor, dst: torch.Tensor, order: torch.Tensor,
              tile_expert: torch.Tensor, tile_begin: torch.Tensor, tile_rows: torch.Tensor, meta: torch.Tensor,
-             max_tiles: int, act: int = ACT_NONE, few_pairs: Optional[bool] = None) -> None:
+             max_tiles: int, act: int = ACT_NONE, few_pairs: Optional[bool] = None, gated: bool = False,
+             limit: float = 0.0, slope: float = 1.0) -> None:
     """dst[pair] = act(w[expert of the pair] @ src[pair // src_div]) for every listed pair: w [experts, n, k]
     (or [experts * n, k]) with ``n = dst.shape[1]``, src [*, k], dst [pairs, n].  ``few_pairs`` chooses the
-    kernel that streams the weights for a handful of pairs (default: up to MOE_FEW_PAIRS rows of dst)."""
+    kernel that streams the weights for a handful of pairs (default: up to MOE_FEW_PAIRS rows of dst).  ``gated``
+    (that kernel only): w [experts * 2 n, k], gate rows and then up rows, dst[pair] = act(gate) * up (``limit`` and
+    ``slope`` as in ``gated_act``)."""
     _need_cuda(src, w, dst)
     n, k = dst.shape[1], src.shape[1]
     if w.shape[-1] != k or not w.is_contiguous() or src.stride(1) != 1 or dst.stride(1) != 1 or src.dtype != dst.dtype \
             or w.dtype != src.dtype:
         raise KernelError(f"moe_gemm: shapes src{tuple(src.shape)} w{tuple(w.shape)} dst{tuple(dst.shape)}, one type")
     f = _fn(_moe(), "rl_moe_gemm", [c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p,
-                                     c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
+                                     c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
+                                     c_void_p])
     if few_pairs is None:
         few_pairs = dst.shape[0] <= MOE_FEW_PAIRS
+    if gated and not few_pairs:
+        raise KernelError("moe_gemm: the gated form is for a handful of pairs")
     _check(f(_code(src.dtype), _ptr(src), src.stride(0), src_div, _ptr(w), n, k, _ptr(dst), dst.stride(0), _ptr(order),
              _ptr(tile_expert), _ptr(tile_begin), _ptr(tile_rows), _ptr(meta), max_tiles, 1 if few_pairs else 0, act,
-             _stream()), "moe_gemm")
+             1 if gated else 0, float(limit), float(slope), _stream()), "moe_gemm")
 
 
 def moe_combine(y: torch.Tensor, weight: torch.Tensor, shared: Optional[torch.Tensor], out: torch.Tensor,

@@ -257,9 +257,26 @@ class Mixer(Part):
         return False
 
 
+@dataclass
+class WeightedTerms:
+    """A sublayer's output as the sum that it is: ``top`` rows per token times their weights, plus a shared row
+    (times the sigmoid of a number per token, if given).  A kernel that reads the output anyway may form it."""
+
+    rows: torch.Tensor                       # [T * top, H]
+    weight: torch.Tensor                     # float32 [T * top]
+    top: int
+    shared: Optional[torch.Tensor] = None    # [T, H]
+    shared_gate: Optional[torch.Tensor] = None
+
+
 class FeedForward(Part):
     def forward(self, x: torch.Tensor, ctx) -> torch.Tensor:
         raise NotImplementedError
+
+    def forward_terms(self, x: torch.Tensor, ctx) -> Optional[WeightedTerms]:
+        """``forward`` with its closing sum left to the caller, for parts that end in one; None (and nothing done)
+        otherwise."""
+        return None
 
     def forward_into(self, residual: torch.Tensor, norm: Norm, ctx) -> bool:
         """Optional fused form: residual += ffn(norm(residual)); see ``Mixer.forward_into``."""

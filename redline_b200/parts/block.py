@@ -165,10 +165,12 @@ class OutNormBlock(Block):
         self.mixer_post_norm.add_post_cast(residual, a, x if nxt else None, rows=T)
         op_mark(ctx, self.closing_op, nbytes=PreNormBlock._norm_bytes(residual, a, x))
         if not last:
-            f = self.ffn.forward(x, ctx)
             nxt = copy and isinstance(ctx.block_next, OutNormBlock)
-            self.ffn_post_norm.add_post_cast(residual, f, x if nxt else None, rows=T)
-            op_mark(ctx, self.closing_op, nbytes=PreNormBlock._norm_bytes(residual, f, x))
+            terms = self.ffn.forward_terms(x, ctx) if getattr(self.ffn_post_norm, "sums_terms", False) else None
+            f = terms.rows if terms is not None else self.ffn.forward(x, ctx)
+            self.ffn_post_norm.add_post_cast(residual, f if terms is None else terms, x if nxt else None, rows=T)
+            op_mark(ctx, self.closing_op if terms is None else "combine+" + self.closing_op,
+                    nbytes=PreNormBlock._norm_bytes(residual, f, x))
         if nxt:
             ctx.block_normed = (self.AS_IS, x)
         return None

@@ -155,8 +155,9 @@ class LatentAttention(Mixer):
         latent = proj[:, self.c_col:self.c_col + self.key_size] if p.own_latent and cache.write else None
         head = (p.num_heads, p.dim, p.rot_dim, p.kv_rank, self.rot_dims)
         cached = (g.slots if latent is not None else None, k_cache, rt.page_size, ctx.status, self.pairs)
+        turn = None
         if p.q_rank > 0:
-            # the latent into the cache beside the norm of the queries' latent; then the queries and their rotation
+            # the latent into the cache beside the norm of the queries' latent; then the queries, whose rotated parts go along with the product below
             c_q = ws.get("latent.cq", (rt.max_tokens, p.q_rank), rt.dtype)[:T]
             kernels.latent_prep(None, latent, ctx.positions, T, *head, self.w_norm if latent is not None else None, p.eps,
                                 self.cos, self.sin, None, *cached, dq=proj[:, :p.q_rank], dq_w=self.w_dq_norm, dq_out=c_q)
@@ -165,15 +166,13 @@ class LatentAttention(Mixer):
             linear(c_q, self.w_uq, q)
             op_mark(ctx, "q_up_proj", self.w_uq, T)
             if p.rot_dim > 0:
-                kernels.latent_prep(q, None, ctx.positions, T, *head, None, p.eps, self.cos, self.sin, qa, None, None,
-                                    rt.page_size, ctx.status, self.pairs)
-                op_mark(ctx, "rotate_queries", nbytes=float(2 * T * p.num_heads * p.rot_dim * elem))
+                turn = (p.rot_dim, p.dim, p.kv_rank, self.cos, self.sin, ctx.positions, self.pairs, ctx.status)
         else:
             q = proj[:, :self.q_size]
             kernels.latent_prep(q, latent, ctx.positions, T, *head, self.w_norm, p.eps, self.cos, self.sin, qa, *cached)
             op_mark(ctx, "latent_norm+rotate+write", nbytes=float(T * (self.proj_size + 2 * self.key_size
                                                                        + p.num_heads * p.rot_dim) * elem))
-        kernels.head_linear(q, 0, self.q_head, self.w_uk_t, qa, 0, self.key_size, tokens=T)
+        kernels.head_linear(q, 0, self.q_head, self.w_uk_t, qa, 0, self.key_size, tokens=T, turn=turn)
         op_mark(ctx, "q_absorb", nbytes=float(T * p.num_heads * (p.dim + p.kv_rank) * elem + self.w_uk_t.numel() * elem),
                 flops=2.0 * T * p.num_heads * p.dim * p.kv_rank)
         gate = dict(gate=proj[:, self.g_col:], gate_mode=1) if p.gated else {}

@@ -25,8 +25,11 @@ import torch
 
 from ..ops import kernels
 from ..ops.linear import linear
-from .base import FeedForward, op_mark, register
+from .base import FeedForward, WeightedTerms, op_mark, register
 from .spec import TensorSpec
+
+
+MAX_ROUTE_GROUP_TOKENS = 16      # up to so many tokens the choice and the grouping are one launch
 
 
 @dataclass(frozen=True)
@@ -175,6 +178,10 @@ class RoutedExperts(FeedForward):
         if p.shared_gate:
             self.w_router = tensors["router_all"] if "router_all" in tensors else torch.cat(
                 [tensors["router"], tensors["shared_sg"].to(tensors["router"].dtype)], dim=0).contiguous()
+        # (rows of zeros up to a multiple of 8: the library's products of odd heights are several times slower)
+        pad = -self.w_router.shape[0] % 8
+        if pad:
+            self.w_router = torch.cat([self.w_router, self.w_router.new_zeros(pad, p.hidden_size)], dim=0).contiguous()
         if self.shared is not None and p.gated:
             self.shared.load({"gate": tensors["shared_gate"], "up": tensors["shared_up"], "down": tensors["shared_down"]})
         elif self.shared is not None:
@@ -185,6 +192,25 @@ class RoutedExperts(FeedForward):
         return n + (self.shared.nbytes() if self.shared is not None else 0)
 
     def forward(self, x, ctx) -> torch.Tensor:
+        p, rt = self.params, self.rt
+        T = ctx.T
+        t, choice = self._terms(x, ctx)
+        out = rt.workspace.get("ffn.out", (rt.max_tokens, p.hidden_size), rt.dtype)[:T]
+        if p.identity > 0:
+            kernels.moe_combine(t.rows, t.weight, t.shared, out, T, p.top, choice=choice, real_experts=p.num_experts, x=x,
+                                shared_gate=t.shared_gate)
+        else:
+            kernels.moe_combine(t.rows, t.weight, t.shared, out, T, p.top, shared_gate=t.shared_gate)
+        op_mark(ctx, "combine", nbytes=float((T * p.top + 2 * T) * p.hidden_size * x.element_size()))
+        return out
+
+    def forward_terms(self, x, ctx) -> Optional[WeightedTerms]:
+        if self.params.identity > 0:             # (an identity expert's term is the input row: ``moe_combine`` knows)
+            return None
+        return self._terms(x, ctx)[0]
+
+    def _terms(self, x, ctx):
+        """(the chosen experts' outputs with their weights and the shared expert's, the choices)."""
         p, rt = self.params, self.rt
         T = ctx.T
         ws = rt.workspace
@@ -204,18 +230,24 @@ class RoutedExperts(FeedForward):
         scored = ws.get("moe.logits", (rt.max_tokens, self.w_router.shape[0]), torch.float32)[:T]
         linear(x, self.w_router, scored)
         logits = scored[:, :self.outputs]
-        kernels.moe_route(logits, None, choice, weight, T, p.groups, p.group_keep, p.group_top, p.top,
-                          softmax=p.score == "softmax", renorm=p.renormalize, bias=self.b_router,
-                          choice_bias=self.b_choice, weight_scale=p.weight_scale, renorm_floor=p.renorm_floor)
-        kernels.moe_group(choice, pairs, self.outputs, order, tile_expert, tile_begin, tile_rows, meta,
-                          tiled=p.num_experts)
+        how = dict(softmax=p.score == "softmax", renorm=p.renormalize, bias=self.b_router, choice_bias=self.b_choice,
+                   weight_scale=p.weight_scale, renorm_floor=p.renorm_floor)
+        lists = (order, tile_expert, tile_begin, tile_rows, meta)
+        if T <= MAX_ROUTE_GROUP_TOKENS and pairs <= kernels.MOE_ROUTE_GROUP_PAIRS and self.outputs <= 256:
+            kernels.moe_route_group(logits, choice, weight, T, p.groups, p.group_keep, p.group_top, p.top, *lists,
+                                    tiled=p.num_experts, **how)
+        else:
+            kernels.moe_route(logits, None, choice, weight, T, p.groups, p.group_keep, p.group_top, p.top, **how)
+            kernels.moe_group(choice, pairs, self.outputs, *lists, tiled=p.num_experts)
         op_mark(ctx, "route", self.w_router, T)
         if x.dtype != self.w_up.dtype:
             raise kernels.KernelError("routed_experts: expert weights must have the activation type")
         act = ws.get("moe.act", (max_pairs, p.intermediate_size), rt.dtype)[:pairs]
         y = ws.get("moe.y", (max_pairs, p.hidden_size), rt.dtype)[:pairs]
-        lists = (order, tile_expert, tile_begin, tile_rows, meta, max_tiles)
-        if p.gated:
+        lists = lists + (max_tiles,)
+        if p.gated and pairs <= kernels.MOE_FEW_PAIRS:
+            kernels.moe_gemm(x, p.top, self.w_up, act, *lists, act=self.act, gated=True, limit=p.limit, slope=p.slope)
+        elif p.gated:
             gu = ws.get("moe.gate_up", (max_pairs, 2 * p.intermediate_size), rt.dtype)[:pairs]
             kernels.moe_gemm(x, p.top, self.w_up, gu, *lists)
             kernels.gated_act(gu, act, self.act, p.limit, p.slope)
@@ -230,12 +262,5 @@ class RoutedExperts(FeedForward):
         shared = None
         if self.shared is not None:
             shared = self.shared.run(x, ctx, "moe.shared")
-        out = ws.get("ffn.out", (rt.max_tokens, p.hidden_size), rt.dtype)[:T]
         gate = scored[:, self.outputs] if p.shared_gate else None
-        if p.identity > 0:
-            kernels.moe_combine(y, weight, shared, out, T, p.top, choice=choice, real_experts=p.num_experts, x=x,
-                                shared_gate=gate)
-        else:
-            kernels.moe_combine(y, weight, shared, out, T, p.top, shared_gate=gate)
-        op_mark(ctx, "combine", nbytes=float((pairs + 2 * T) * p.hidden_size * elem))
-        return out
+        return WeightedTerms(y, weight[:pairs], p.top, shared, gate), choice

@@ -13,7 +13,7 @@ from typing import Dict, Optional
 import torch
 
 from ..ops import kernels
-from .base import Norm, register
+from .base import Norm, WeightedTerms, register
 from .spec import TensorSpec
 
 
@@ -57,6 +57,8 @@ class RMSNormSumParams:
 class RMSNormSum(Norm):
     """stream = rmsnorm(alpha * stream + scale * delta) * weight: the norm after the sum ("postnorm" blocks)."""
 
+    sums_terms = True
+
     def tensors(self) -> Dict[str, TensorSpec]:
         t = {"weight": TensorSpec((self.params.size,))}
         if self.params.scaled:
@@ -75,6 +77,11 @@ class RMSNormSum(Norm):
 
     def add_post_cast(self, residual: torch.Tensor, delta: torch.Tensor, out: Optional[torch.Tensor],
                       rows: Optional[int] = None) -> None:
-        """The norm of the sum in place on the stream; with ``out`` also out = the new stream rows in out's type."""
+        """The norm of the sum in place on the stream; with ``out`` also out = the new stream rows in out's type.
+        ``delta`` may be ``WeightedTerms``: the same kernel then forms their sum."""
         p = self.params
-        kernels.sum_norm(residual, delta, self.weight, self.scale, p.alpha, p.eps, out, rows=rows)
+        terms = {}
+        if isinstance(delta, WeightedTerms):
+            terms = dict(top=delta.top, mix_weight=delta.weight, shared=delta.shared, shared_gate=delta.shared_gate)
+            delta = delta.rows
+        kernels.sum_norm(residual, delta, self.weight, self.scale, p.alpha, p.eps, out, rows=rows, **terms)

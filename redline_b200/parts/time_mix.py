@@ -12,7 +12,8 @@ square, the joined heads multiplied by a weight and by the gate, then projected 
 
 The per-request state is S (float32 [heads, dim, dim]) and the last row h (float32 [width]): two pools.  Where
 the block's sublayers read the residual stream itself, the mixes are formed from its float32 rows
-(``ctx.block_stream``).  The decays' two products have float32 results; mixes, tanh, decays, the recurrence,
+(``ctx.block_stream``).  Products of at most 8 rows run as one launch (groups of features with an input each).  The
+decays' two products have float32 results; mixes, tanh, decays, the recurrence,
 norm and gate are float32 (csrc/stream_ops.cu, csrc/linear_attention.cu).
 """
 
@@ -99,18 +100,27 @@ class TimeMix(Mixer):
         mixes = ws.get("tmix.mixes", (len(MIXES), rt.max_tokens, p.hidden_size), rt.dtype)
         kernels.token_shift(stream, self.mu, mixes, ctx.seq_of_token, ctx.state_slot, shift_state, T)
         op_mark(ctx, "token_shift", nbytes=T * p.hidden_size * (stream.element_size() + len(MIXES) * elem))
-        rkvg = ws.get("tmix.rkvg", (4, rt.max_tokens, n), rt.dtype)
+        w4 = self.w_in[:4 * n]
+        if kernels.gemm_skinny_grouped_ok(T, mixes, w4, n):          # a few rows: the four products are one launch
+            rkvg = ws.get("tmix.rkvg", (rt.max_tokens, 4 * n), rt.dtype)[:T]
+            kernels.gemm_skinny_grouped(mixes, w4, rkvg, T, n)
+            r, k, v, g = (rkvg[:, i * n:(i + 1) * n] for i in range(4))
+        else:
+            rkvg = ws.get("tmix.rkvg", (4, rt.max_tokens, n), rt.dtype)
+            for i in range(4):
+                linear(mixes[i, :T], self.w_each[i], rkvg[i, :T])
+            r, k, v, g = (rkvg[i, :T] for i in range(4))
         low = ws.get("tmix.low", (rt.max_tokens, p.decay_rank), torch.float32)[:T]
-        inner = ws.get("tmix.inner", (rt.max_tokens, p.decay_rank), rt.dtype)[:T]
-        for i in range(4):
-            linear(mixes[i, :T], self.w_each[i], rkvg[i, :T])
         linear(mixes[4, :T], self.w_each[4], low)
-        kernels.act_cast(low, inner, kernels.ACT_TANH)
         op_mark(ctx, "rkvgw_proj", self.w_in, T)
         z = ws.get("tmix.z", (rt.max_tokens, n), torch.float32)[:T]
-        linear(inner, self.w_2, z)
+        if T <= kernels.LOW_RANK_ROWS and p.decay_rank <= kernels.LOW_RANK_MAX:
+            kernels.low_rank(low, self.w_2, z, kernels.ACT_TANH)
+        else:
+            inner = ws.get("tmix.inner", (rt.max_tokens, p.decay_rank), rt.dtype)[:T]
+            kernels.act_cast(low, inner, kernels.ACT_TANH)
+            linear(inner, self.w_2, z)
         op_mark(ctx, "decay_proj", self.w_2, T)
-        r, k, v, g = (rkvg[i, :T] for i in range(4))
         y = ws.get("tmix.y", (rt.max_tokens, n), rt.dtype)[:T]
         run_recurrence(self, ctx, r, k, v, z, s_state, y, heads=p.num_heads, dim=p.dim, vdim=p.dim, decay_bias=self.w_0,
                        bonus=self.u, gate=g, gate_mode=kernels.GATE_SILU, norm_w=self.w_norm, eps=p.eps)

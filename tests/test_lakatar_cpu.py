@@ -98,7 +98,7 @@ def test_random_weights_are_what_the_model_expects(tmp_path):
     mix = m.blocks[1].mixer
     assert torch.equal(mix.w_each[2], w["l1.mix.v"]) and torch.equal(mix.mu[4], w["l1.mix.mu.w"])
     moe = m.blocks[0].ffn
-    assert torch.equal(moe.w_router[-1:], w["l0.mlp.shared.sg"]) and moe.w_router.shape[0] == 7
+    assert torch.equal(moe.w_router[6:7], w["l0.mlp.shared.sg"]) and torch.equal(moe.w_router[:6], w["l0.mlp.router"])
     lat = m.blocks[4].mixer
     assert lat.w_norm is None and torch.equal(lat.w_proj, torch.cat([w["l4.mix.dq"], w["l4.mix.g"]]))
     logits = P.forward(C.MIX, w, [1, 5, 9])

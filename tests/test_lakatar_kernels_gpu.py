@@ -2,7 +2,9 @@
 the recurrence with a decay per token and channel and with one decay per head (token by token and in blocks on
 the tensor cores, cut into chunks, from a given state, heads finished by the kernel or behind it), the token
 shift and its state, the norm after the sum, the latent's preparation with rotated neighbours and a latent of
-the queries, groups of experts scored by their best choice score, the gated shared expert."""
+the queries, groups of experts scored by their best choice score, the gated shared expert, and the fused forms
+for a few rows (choice and grouping in one launch, gated experts, several products at once, the decays' second
+product) and for the sum of terms that is normed."""
 
 import math
 
@@ -240,6 +242,21 @@ def test_latent_prep_with_neighbours_and_a_latent_of_the_queries(dtype, tol, H, 
             assert rel(flat[int(slots[t])], torch.cat([c[t], kr[t]])) < tol
     got = qa.view(T, H, key)
     assert rel(got[:, :, rank:], rq) < tol and torch.isnan(got[:, :, :rank].float()).all()
+    # the same parts beside the per-head product that fills the rest, on both of its kernels
+    w = torch.randn(H, rank, dn, generator=g).to(dtype)
+    want = torch.einsum("hrd,thd->thr", w.double(), q.double().view(T, H, dn + dr)[:, :, :dn])
+    for impl in (0, 1, 2):
+        both = torch.full((T, H * key), float("nan"), dtype=dtype, device=DEV)
+        kernels.head_linear(q.to(DEV), 0, dn + dr, w.to(DEV), both, 0, key, impl=impl,
+                            turn=(dr, dn, rank, cos, sin, pos.to(DEV), True, status))
+        assert rel(both.view(T, H, key)[:, :, :rank], want) < tol
+        assert torch.equal(both.view(T, H, key)[:, :, rank:], got[:, :, rank:])
+        few = torch.full((9, H * key), float("nan"), dtype=dtype, device=DEV)
+        kernels.head_linear(q[:9].to(DEV), 0, dn + dr, w.to(DEV), few, 0, key, impl=impl,
+                            turn=(dr, dn, rank, cos, sin, pos[:9].to(DEV), True, status))
+        assert rel(few.view(9, H, key)[:, :, :rank], want[:9]) < tol
+        assert torch.equal(few.view(9, H, key)[:, :, rank:], got[:9, :, rank:])
+    assert int(status.item()) == 0
     # another layer's rows are attended over: only the queries' latent is normed, nothing is written
     before = cache.clone()
     cq.zero_()
@@ -290,3 +307,130 @@ def test_a_gated_shared_expert_in_the_weighted_sum(dtype, tol):
     kernels.moe_combine(y.to(DEV), weight.to(DEV), sh.to(DEV), out, T, top, shared_gate=logits.to(DEV)[:, 4])
     want = (weight.double().view(T, top, 1) * y.double().view(T, top, W)).sum(1) + P.sigmoid(logits[:, 4:].double()) * sh.double()
     assert rel(out, want) < tol
+
+
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-6), (torch.bfloat16, 1e-2)])
+@pytest.mark.parametrize("width,top,gated", [(96, 2, True), (101, 3, True), (2048, 4, False), (4100, 1, None)])
+def test_norm_after_a_sum_of_terms(dtype, tol, width, top, gated):
+    """The routed experts' weighted sum formed by the kernel that norms (gated None: no shared expert)."""
+    from redline_b200.ops import kernels
+    g = torch.Generator().manual_seed(width + top)
+    T, alpha, eps = 6, 1.3, 1e-5
+    res = torch.randn(T, width, generator=g)
+    y, sh = torch.randn(T * top, width, generator=g).to(dtype), torch.randn(T, width, generator=g).to(dtype)
+    weight, logits = torch.rand(T * top, generator=g), torch.randn(T, 4, generator=g) * 2
+    w, sc = 1.0 + 0.3 * torch.randn(width, generator=g), 1.0 + 0.3 * torch.randn(width, generator=g)
+    d = (weight.double().view(T, top, 1) * y.double().view(T, top, width)).sum(1)
+    if gated is not None:
+        d = d + (P.sigmoid(logits[:, 2:3].double()) if gated else 1.0) * sh.double()
+    want = P.unit(alpha * res.double() + sc.double() * d, eps) * w.double()
+    r, out = res.clone().to(DEV), torch.empty(T, width, dtype=dtype, device=DEV)
+    kernels.sum_norm(r, y.to(DEV), w.to(DEV), sc.to(DEV), alpha, eps, out, top=top, mix_weight=weight.to(DEV),
+                     shared=sh.to(DEV) if gated is not None else None, shared_gate=logits.to(DEV)[:, 2] if gated else None)
+    assert rel(r, want) < 3e-6 and rel(out, want) < tol
+
+
+@pytest.mark.parametrize("tokens,experts,count,keep,top", [(1, 12, 3, 1, 2), (7, 32, 4, 2, 4), (16, 100, 1, 1, 16), (5, 6, 6, 3, 3), (3, 1, 1, 1, 1)])
+def test_choice_and_grouping_in_one_launch(tokens, experts, count, keep, top):
+    """The same choice, weights, order and tiles as the two kernels that do it one after the other."""
+    from redline_b200.ops import kernels
+    g = torch.Generator().manual_seed(tokens * experts)
+    z = (torch.randn(tokens, experts + 1, generator=g) * 2).to(DEV)[:, :experts]
+    corr = (torch.randn(experts, generator=g) * 0.3).to(DEV)
+    pairs, cap = tokens * top, kernels.moe_max_tiles(tokens * top, experts)
+    for tiled in (experts, max(experts - 2, 0)):
+        got = []
+        for fused in (False, True):
+            i32 = lambda n: torch.full((n,), -7, dtype=torch.int32, device=DEV)  # noqa: E731
+            choice, weight, lists = i32(pairs), torch.zeros(pairs, device=DEV), (i32(pairs), i32(cap), i32(cap), i32(cap), i32(4))
+            how = dict(softmax=True, choice_bias=corr, weight_scale=1.5)
+            if fused:
+                kernels.moe_route_group(z, choice, weight, tokens, count, keep, 1, top, *lists, tiled=tiled, **how)
+            else:
+                kernels.moe_route(z, None, choice, weight, tokens, count, keep, 1, top, **how)
+                kernels.moe_group(choice, pairs, experts, *lists, tiled=tiled)
+            n = int(lists[4][0])
+            got.append((choice, weight, lists[0], lists[1][:n], lists[2][:n], lists[3][:n]))
+        for a, b in zip(*got):
+            assert torch.equal(a, b)
+
+
+@pytest.mark.parametrize("dtype,tol", [(torch.float32, 3e-6), (torch.bfloat16, 2e-2)])
+@pytest.mark.parametrize("ff,width", [(24, 64), (17, 33), (704, 256)])
+@pytest.mark.parametrize("act", ["silu", "clamped_swish"])
+def test_gated_experts_of_a_few_pairs(dtype, tol, ff, width, act):
+    from redline_b200.ops import kernels
+    g = torch.Generator().manual_seed(ff)
+    experts, tokens, top, limit, slope = 5, 6, 2, 1.2, 1.702
+    x = torch.randn(tokens, width, generator=g).to(dtype)
+    w = (torch.randn(experts, 2 * ff, width, generator=g) / math.sqrt(width)).to(dtype)
+    choice = torch.stack([torch.randperm(experts, generator=g)[:top] for _ in range(tokens)]).to(torch.int32).reshape(-1).to(DEV)
+    pairs, cap = tokens * top, kernels.moe_max_tiles(tokens * top, experts)
+    i32 = lambda n: torch.zeros(n, dtype=torch.int32, device=DEV)  # noqa: E731
+    lists = (i32(pairs), i32(cap), i32(cap), i32(cap), i32(4))
+    kernels.moe_group(choice, pairs, experts, *lists)
+    out = torch.empty(pairs, ff, dtype=dtype, device=DEV)
+    mode = kernels.ACT_CLAMPED_SWISH if act == "clamped_swish" else kernels.ACT_SILU
+    kernels.moe_gemm(x.to(DEV), top, w.to(DEV).view(experts * 2 * ff, width), out, *lists, cap, act=mode, gated=True, limit=limit, slope=slope)
+    for p in range(pairs):
+        z = w[int(choice[p])].double() @ x[p // top].double()
+        gate, up = z[:ff], z[ff:]
+        if act == "silu":
+            want = P.silu(gate) * up
+        else:
+            c = gate.clamp(max=limit)
+            want = c * P.sigmoid(slope * c) * (up.clamp(-limit, limit) + 1.0)
+        assert rel(out[p], want) < tol
+
+
+@pytest.mark.parametrize("rows,n,groups,k", [(1, 64, 4, 96), (8, 48, 3, 256), (3, 2048, 4, 2048), (5, 16, 5, 136)])
+def test_several_products_of_a_few_rows_in_one_launch(rows, n, groups, k):
+    from redline_b200.ops import kernels
+    g = torch.Generator().manual_seed(rows + n)
+    x = torch.randn(groups, rows + 2, k, generator=g).to(torch.bfloat16).to(DEV)
+    w = (torch.randn(groups * n, k, generator=g) / math.sqrt(k)).to(torch.bfloat16).to(DEV)
+    y = torch.empty(rows, groups * n, dtype=torch.bfloat16, device=DEV)
+    assert kernels.gemm_skinny_grouped_ok(rows, x, w, n)
+    kernels.gemm_skinny_grouped(x, w, y, rows, n)
+    for i in range(groups):
+        want = x[i, :rows].double().cpu() @ w[i * n:(i + 1) * n].double().cpu().T
+        assert rel(y[:, i * n:(i + 1) * n], want) < 1e-2
+    assert not kernels.gemm_skinny_grouped_ok(9, x, w, n) and not kernels.gemm_skinny_grouped_ok(rows, x, w, n + 8)
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("rows,n,rank", [(1, 100, 5), (16, 257, 64), (9, 64, 24)])
+def test_low_rank_second_product(dtype, rows, n, rank):
+    from redline_b200.ops import kernels
+    g = torch.Generator().manual_seed(n)
+    x = torch.randn(rows, rank, generator=g)
+    w = torch.randn(n, rank, generator=g).to(dtype)
+    z = torch.empty(rows, n, device=DEV)
+    kernels.low_rank(x.to(DEV), w.to(DEV), z, kernels.ACT_TANH)
+    assert rel(z, torch.tanh(x.double()) @ w.double().T) < (2e-6 if dtype == torch.float32 else 5e-3)
+    y = torch.empty(rows, rank, dtype=dtype, device=DEV)
+    kernels.act_cast(x.to(DEV), y, kernels.ACT_TANH)
+    assert rel(z, y.double().cpu() @ w.double().T) < 2e-6
+
+
+@pytest.mark.parametrize("pairs,experts,tiled", [(5, 3, 3), (64, 12, 10), (1000, 7, 7), (4097, 130, 128), (20000, 256, 256), (9000, 2000, 2000)])
+def test_grouping_of_many_pairs(pairs, experts, tiled):
+    """Every expert's pairs in ascending order, one expert after another, in tiles of up to 64 (few experts chosen
+    often, many never)."""
+    from redline_b200.ops import kernels
+    g = torch.Generator().manual_seed(pairs)
+    choice = (torch.rand(pairs, generator=g) ** 3 * experts).to(torch.int32).clamp(max=experts - 1)
+    cap = kernels.moe_max_tiles(pairs, experts)
+    i32 = lambda n: torch.full((n,), -7, dtype=torch.int32, device=DEV)  # noqa: E731
+    order, te, tb, tr, meta = i32(pairs), i32(cap), i32(cap), i32(cap), i32(4)
+    kernels.moe_group(choice.to(DEV), pairs, experts, order, te, tb, tr, meta, tiled=tiled)
+    want = torch.sort(choice, stable=True).indices
+    assert torch.equal(order.cpu().long(), want)
+    tiles, at = [], 0
+    for e, n in enumerate(torch.bincount(choice.long(), minlength=experts).tolist()):
+        if e < tiled:
+            tiles += [(e, at + r, min(64, n - r)) for r in range(0, n, 64)]
+        at += n
+    n = int(meta[0])
+    assert n == len(tiles)
+    assert [tuple(t) for t in torch.stack([te[:n], tb[:n], tr[:n]], 1).tolist()] == tiles

@@ -270,8 +270,8 @@ def test_the_comparison_model_of_the_bench():
     of as many layers, the same width, heads, window and experts."""
     from redline_b200.apps import design_bench as D
     from redline_b200.config.registry import config_from_dict, model_spec
-    sizes, make, beside, make_beside = D.DESIGNS["venezen"]
-    assert beside == "kapitar"
+    sizes, make, ((beside, beside_sizes, make_beside),) = D.DESIGNS["venezen"]
+    assert beside == "kapitar" and beside_sizes is sizes
     for s in sizes.values():
         v, k = config_from_dict(make(s)), config_from_dict(make_beside(s))
         assert [(l.type, l.mlp.kind) for l in v.layers] == [("latent_attention", "dense"), ("attention", "moe"),

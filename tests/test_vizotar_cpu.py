@@ -339,11 +339,12 @@ def test_the_comparison_models_of_the_bench_parse():
     many layers, the same width and vocabulary."""
     from redline_b200.apps import design_bench as D
     from redline_b200.config.registry import config_from_dict, model_spec
-    for design, (sizes, make, beside, make_beside) in D.DESIGNS.items():
-        for s in sizes.values():
-            a, b = config_from_dict(make(s)), config_from_dict(make_beside(s))
-            sa, sb = model_spec(a), model_spec(b)
-            assert (sa.hidden_size, sa.vocab_size, len(sa.order)) == (sb.hidden_size, sb.vocab_size, len(sb.order)), design
+    for design, (sizes, make, besides) in D.DESIGNS.items():
+        for name, s in sizes.items():
+            sa = model_spec(config_from_dict(make(s)))
+            for _, beside_sizes, make_beside in besides:
+                sb = model_spec(config_from_dict(make_beside(beside_sizes[name])))
+                assert (sa.hidden_size, sa.vocab_size, len(sa.order)) == (sb.hidden_size, sb.vocab_size, len(sb.order)), design
     v = config_from_dict(D.vizotar_config(D.VIZOTAR_SIZES["s"]))
     assert [l.type for l in v.layers] == ["parallel", "channel_delta", "parallel", "channel_delta"]
     assert [l.mlp.kind for l in v.layers] == ["dense", "moe", "moe", "dense"] and v.streams == 4
