@@ -48,6 +48,9 @@ __device__ __forceinline__ float exp2_of(float x) {
   return r;
 }
 constexpr float kLog2E = 1.4426950408889634f;
+// log2 of exp(-exp(z)).  Bounded where 2^x is zero anyway, so that the sums along a block stay small numbers whose
+// differences are exact to rounding (and finite).
+__device__ __forceinline__ float log_of_decay(float z) { return fmaxf(-kLog2E * exp2_of(kLog2E * z), -160.f); }
 
 struct TcLayout {                              // bytes from the start of the dynamic shared memory
   int raw_bytes, q, k, v, g, z, cs, sn;        // a raw buffer's size, its parts; rows of qk_row, v_row, ... bytes
@@ -260,7 +263,7 @@ linear_attention_tc_kernel(const LinArgs<bf16> a) {
               const float2 u = load2(bonus + d);
               own = fmaf(qv.x * u.x, kv.x, fmaf(qv.y * u.y, kv.y, own));
             }
-            lw = make_float2(-kLog2E * exp2_of(kLog2E * (z.x + zb.x)), -kLog2E * exp2_of(kLog2E * (z.y + zb.y)));
+            lw = make_float2(log_of_decay(z.x + zb.x), log_of_decay(z.y + zb.y));
           }
         }
         *reinterpret_cast<float2*>(kf + tt * kFS + d) = kv;

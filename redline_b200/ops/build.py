@@ -29,6 +29,7 @@ ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 BASE_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "--shared", "-Xcompiler", "-fPIC", "-Xcompiler", "-fno-gnu-unique"]
 
 _lock = threading.Lock()
+_locks: Dict[str, threading.Lock] = {}         # one per object, so that different ones may be compiled side by side
 _build_dir: Optional[str] = None
 
 
@@ -102,6 +103,8 @@ def compile_module(name: str, source: str, defines: Optional[Dict[str, object]] 
     if os.path.exists(out):
         return out
     with _lock:
+        own = _locks.setdefault(out, threading.Lock())
+    with own:
         if os.path.exists(out):
             return out
         tmp = f"{out}.{os.getpid()}.tmp"

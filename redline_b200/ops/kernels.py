@@ -9,6 +9,7 @@ from __future__ import annotations
 
 import ctypes
 import os
+from concurrent.futures import ThreadPoolExecutor
 from ctypes import c_float, c_int, c_longlong, c_uint, c_void_p
 from typing import Dict, Optional, Tuple
 
@@ -1493,34 +1494,18 @@ def build_all(head_dims=(64, 128), maps_dims=((64, 128, 2), (128, 128, 1)), line
     """Compiles every kernel family (attention for the given head sizes, attention with score maps for the
     given (key size, value size, maps), linear attention and the matrix memory for the given key sizes) and
     removes built files of these modules that belong to other versions of the sources."""
-    built = [
-        build.compile_module("elementwise", "elementwise.cu", verbose=verbose),
-        build.compile_module("gemm_simt", "gemm_simt.cu", verbose=verbose),
-        build.compile_module("gemm_skinny", "gemm_skinny.cu", verbose=verbose),
-        build.compile_module("gemm_tc", "gemm_tc.cu", verbose=verbose),
-        build.compile_module("gemm_mid", "gemm_mid.cu", verbose=verbose),
-        build.compile_module("sampling", "sampling.cu", verbose=verbose),
-        build.compile_module("rowwise", "rowwise.cu", verbose=verbose),
-        build.compile_module("moe", "moe.cu", verbose=verbose),
-        build.compile_module("latent", "latent.cu", verbose=verbose),
-        build.compile_module("stream_ops", "stream_ops.cu", verbose=verbose),
-        build.compile_module("host_core", "host_core.cpp", verbose=verbose),   # host-only: cache manager, batch filler
-    ]
-    for d in head_dims:
-        built.append(build.compile_module(f"attention_d{d}", "attention.cu", {"RL_HEAD_DIM": d}, verbose=verbose))
+    jobs = [(m, f"{m}.cu", None) for m in ("elementwise", "gemm_simt", "gemm_skinny", "gemm_tc", "gemm_mid", "sampling", "rowwise",
+                                           "moe", "latent", "stream_ops")]
+    jobs.append(("host_core", "host_core.cpp", None))              # host-only: cache manager, batch filler
+    jobs += [(f"attention_d{d}", "attention.cu", {"RL_HEAD_DIM": d}) for d in head_dims]
     for d, v, m, *stride in maps_dims:         # (key size, value size, maps[, length of a value row if longer])
+        name, defines = f"attention_maps_d{d}_v{v}_m{m}", {"RL_QK_DIM": d, "RL_V_DIM": v, "RL_MAPS": m}
         if stride and stride[0] not in (0, v):
-            built.append(build.compile_module(f"attention_maps_d{d}_v{v}_m{m}_s{stride[0]}", "attention_maps.cu",
-                                              {"RL_QK_DIM": d, "RL_V_DIM": v, "RL_MAPS": m, "RL_V_STRIDE": stride[0]},
-                                              verbose=verbose))
-            continue
-        built.append(build.compile_module(f"attention_maps_d{d}_v{v}_m{m}", "attention_maps.cu",
-                                          {"RL_QK_DIM": d, "RL_V_DIM": v, "RL_MAPS": m}, verbose=verbose))
-    for d in linear_dims:
-        built.append(build.compile_module(f"linear_attention_d{d}", "linear_attention.cu", {"RL_LIN_DIM": d},
-                                          verbose=verbose))
-    for d in memory_dims:
-        built.append(build.compile_module(f"matrix_memory_d{d}", "matrix_memory.cu", {"RL_MM_DIM": d}, verbose=verbose))
-    for d in delta_dims:
-        built.append(build.compile_module(f"delta_rule_d{d}", "delta_rule.cu", {"RL_DELTA_DIM": d}, verbose=verbose))
+            name, defines = f"{name}_s{stride[0]}", dict(defines, RL_V_STRIDE=stride[0])
+        jobs.append((name, "attention_maps.cu", defines))
+    jobs += [(f"linear_attention_d{d}", "linear_attention.cu", {"RL_LIN_DIM": d}) for d in linear_dims]
+    jobs += [(f"matrix_memory_d{d}", "matrix_memory.cu", {"RL_MM_DIM": d}) for d in memory_dims]
+    jobs += [(f"delta_rule_d{d}", "delta_rule.cu", {"RL_DELTA_DIM": d}) for d in delta_dims]
+    with ThreadPoolExecutor(max(1, min(8, os.cpu_count() or 1))) as pool:
+        built = list(pool.map(lambda job: build.compile_module(*job, verbose=verbose), jobs))
     build.remove_other_versions(built)

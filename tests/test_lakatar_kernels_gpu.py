@@ -130,6 +130,7 @@ def test_recurrence_with_extreme_decays(longest):
     z = torch.full((T, D), -30.0)
     z[:, :8] = 6.0                               # exp(-exp(6)) = 0
     z[::7, 8:16] = 3.0                           # now and then
+    z[5::9, 16:20] = 120.0                       # exp(120) is no float32
     u = torch.randn(D, generator=g)
     w = torch.exp(-torch.exp(z.double())).view(T, 1, D)
     want, S = recurrence(q.double().view(T, 1, D), k.double().view(T, 1, D), v.double().view(T, 1, D),
