@@ -15,10 +15,9 @@
 //                 token's position (entry i with entry i + dims/2 of the first `dims` rotated entries, or
 //                 neighbours, cos and sin from tables), [c | k_r] into the paged cache, q_r into the
 //                 attention's query rows; the norm of the queries' latent
-//   head_linear   y[t, h, :] = W_h x[t, h, :] for every head h, W [heads, n, k], float32 sums in ascending k
-//                 (a row's result does not depend on what else is in the launch); the heads' rotated query
-//                 parts may go along; FFMA for float32, and
-//                 mma.sync.m16n8k16 for bfloat16 operands whose sizes allow it
+//   head_linear   y[t, h, :] = W_h x[t, h, :] for every head h, W [heads, n, k], float32 sums; the heads'
+//                 rotated query parts may go along; FFMA for float32, mma.sync.m16n8k16 for bfloat16
+//                 operands whose sizes allow it, and a kernel that streams the weights for up to 16 tokens
 #include "common.cuh"
 
 namespace rl {

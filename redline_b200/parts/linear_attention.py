@@ -138,7 +138,8 @@ class LinearAttention(Mixer):
         rotation = dict(cos=self.cos, sin=self.sin, positions=ctx.positions) if self.cos is not None else {}
         o = run_recurrence(self, ctx, q, k, v, self.decay, state, y, heads=p.num_heads, dim=p.dim, vdim=p.vdim, gate=g,
                            gate_mode=self.gate_mode, eps=p.eps, finish=p.head_norm, k_scale=p.k_scale, **rotation)
-        op_mark(ctx, "linear_attention", nbytes=T * (self.proj_size * proj.element_size() + 4.0 * self.v_size),
+        nbytes = T * (self.proj_size * proj.element_size() + 4.0 * self.v_size) + 8.0 * ctx.S * n * p.vdim
+        op_mark(ctx, "linear_attention", nbytes=nbytes,
                 flops=4.0 * T * p.num_heads * p.dim * p.vdim)
         if not p.head_norm:
             kernels.gated_rmsnorm(o, g, self.w_norm, y, p.eps, rows=T)

@@ -124,7 +124,7 @@ class TimeMix(Mixer):
         y = ws.get("tmix.y", (rt.max_tokens, n), rt.dtype)[:T]
         run_recurrence(self, ctx, r, k, v, z, s_state, y, heads=p.num_heads, dim=p.dim, vdim=p.dim, decay_bias=self.w_0,
                        bonus=self.u, gate=g, gate_mode=kernels.GATE_SILU, norm_w=self.w_norm, eps=p.eps)
-        op_mark(ctx, "time_mix", nbytes=T * n * (5.0 * elem + 4.0), flops=6.0 * T * n * p.dim)
+        op_mark(ctx, "time_mix", nbytes=T * n * (5.0 * elem + 4.0) + 8.0 * ctx.S * n * p.dim, flops=6.0 * T * n * p.dim)
         out = ws.get("mixer.out", (rt.max_tokens, p.hidden_size), rt.dtype)[:T]
         linear(y, self.w_o, out)
         op_mark(ctx, "o_proj", self.w_o, T)
