@@ -9,7 +9,8 @@ and slots of fixed size for per-request state.
   (reference: src/core/block_allocator.cpp:7-35).
 * Pages go back when a request is closed (finished or preempted), when a
   reservation cannot be completed (all or nothing), and, in a window group, as soon
-  as every key on a page is older than the window of all tokens still to come.
+  as every key on a page is older than the window of all tokens still to come (in a
+  chunk group: lies in an earlier chunk than all of them).
 * A request also holds one state slot (an index into per-layer state pools of fixed
   size) from opening to closing, whether or not any layer keeps state.
 
@@ -96,7 +97,8 @@ class GroupInfo:
 
     @property
     def window(self) -> int:
-        return self.spec.window if self.spec.kind == "window" else 0
+        """The window, or the chunk size of a "chunk" group."""
+        return self.spec.window if self.spec.kind in ("window", "chunk") else 0
 
     @property
     def keep_first(self) -> int:
@@ -156,6 +158,8 @@ class CacheManager:
         for gi, g in enumerate(self.groups):
             if g.keep_first > 0 and self._lib.rl_hc_set_keep_first(self._h, gi, g.keep_first) != 0:
                 raise CacheError(f"group {gi}: the kept first tokens could not be set")
+            if g.spec.kind == "chunk" and self._lib.rl_hc_set_chunked(self._h, gi) != 0:
+                raise CacheError(f"group {gi}: chunks need a positive size")
         self._open: Dict[object, RequestCache] = {}
         self.on_open = None   # called with the RequestCache of every newly opened request
 
@@ -236,9 +240,10 @@ class CacheManager:
         return code == 1
 
     def release_passed(self, rc: RequestCache, num_computed: int) -> int:
-        """After ``num_computed`` positions are in the cache: in window groups, frees the
+        """After ``num_computed`` positions are in the cache: in window and chunk groups, frees the
         pages whose keys no later token can see (key j is dead when j <= n - window for
-        the next position n; the pages of the group's kept first tokens stay).  Returns how many pages were freed."""
+        the next position n, or when it lies before n's chunk; the pages of the group's kept first tokens stay).
+        Returns how many pages were freed."""
         n = self._lib.rl_hc_release_passed(self._h, rc.rid, num_computed)
         if n < 0:
             raise CacheError(f"request {rc.key!r}: releasing pages failed ({n})")

@@ -1255,3 +1255,193 @@ class LakatarConfig(ModelConfig):
         if self.eos_token_ids:
             out["eos_token_id"] = list(self.eos_token_ids)
         return out
+
+
+# ------------------------------------------------------------------------------------------------ Vogolix
+
+@dataclass(frozen=True)
+class VogolixRotation:
+    base: float
+    dims: int                 # the first so many entries of what is rotated turn
+
+
+@dataclass(frozen=True)
+class VogolixAttention:
+    """An 'attention' mixer: softmax attention with a sink within chunks of positions; with ``kv_from`` over the keys
+    and values that layer has cached."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    chunk: int                # mask.size; 0: every earlier key
+    rot: Optional[VogolixRotation]       # neighbours turn together
+    kv_from: Optional[int] = None
+
+
+@dataclass(frozen=True)
+class VogolixLatent:
+    """A 'latent_attention' mixer: keys and values of all heads come from one cached latent vector per token."""
+
+    heads: int
+    dim: int                  # unrotated entries of a head's query and key
+    rot_dim: int              # rotated entries (the key's are one vector for all heads), entry i turns with i + dims / 2
+    vdim: int
+    kv_rank: int              # size of the latent
+    scale: float
+    window: int               # mask.size; 0: every earlier key
+    rot: Optional[VogolixRotation]
+
+
+@dataclass(frozen=True)
+class VogolixStateSpace:
+    """A 'mamba2' mixer."""
+
+    heads: int
+    vdim: int                 # channels of a head
+    state: int                # state entries per channel
+    groups: int               # heads that share their B and C are neighbours
+    norm_groups: int          # equal parts of the joined heads that are normed one by one
+    conv: int                 # taps
+
+
+@dataclass(frozen=True)
+class VogolixLayer:
+    type: str                 # attention | latent_attention | mamba2
+    mixer: Any
+    ff: int                   # width of the dense feed-forward; 0: the layer has none
+
+
+@dataclass(frozen=True)
+class VogolixConfig(ModelConfig):
+    """``Vogolix``: pre-norm layers (RMS norm) on one float32 stream.  Mixers: state-space layers (Mamba-2), attention
+    over a cached latent within a window with a gate per output entry, and grouped attention within chunks of
+    positions (normed and partly rotated queries and keys, biases, a sink; a layer may use an earlier one's keys and
+    values).  Feed-forwards: dense, gated by a ReLU.  The head has a matrix of its own, its logits are multiplied by
+    a constant.  config.json lists the layers under ``layers``."""
+
+    norm_eps: float = 1e-6
+    logit_scale: float = 1.0
+    layers: Tuple[VogolixLayer, ...] = ()
+
+    @classmethod
+    def from_hf(cls, cfg: Dict[str, Any], model_dir: Optional[str] = None) -> "VogolixConfig":
+        layers: List[VogolixLayer] = []
+        for i, entry in enumerate(_need(cfg, "layers")):
+            where = f"layers[{i}]"
+            kind = _need(entry, "type", where)
+            m = _need(entry, "mixer", where)
+            mw = where + ".mixer"
+            heads = int(_need(m, "heads", mw))
+            span = int((m.get("mask") or {}).get("size") or 0)
+            r = m.get("rot")
+            rot = VogolixRotation(float(_need(r, "base", mw + ".rot")), int(_need(r, "dims", mw + ".rot"))) if r else None
+            if kind == "attention":
+                src = m.get("kv_from")
+                mixer: Any = VogolixAttention(
+                    heads=heads, kv_heads=int(m.get("kv_heads") or heads), dim=int(_need(m, "dim", mw)),
+                    vdim=int(_need(m, "vdim", mw)), scale=float(_need(m, "scale", mw)), chunk=span, rot=rot,
+                    kv_from=int(src) if src is not None else None)
+            elif kind == "latent_attention":
+                mixer = VogolixLatent(
+                    heads=heads, dim=int(_need(m, "dim", mw)), rot_dim=int(_need(m, "rot_dim", mw)),
+                    vdim=int(_need(m, "vdim", mw)), kv_rank=int(_need(m, "kv_rank", mw)), scale=float(_need(m, "scale", mw)),
+                    window=span, rot=rot)
+            elif kind == "mamba2":
+                mixer = VogolixStateSpace(
+                    heads=heads, vdim=int(_need(m, "vdim", mw)), state=int(_need(m, "state", mw)),
+                    groups=int(_need(m, "groups", mw)), norm_groups=int(_need(m, "norm_groups", mw)),
+                    conv=int(_need(m, "conv", mw)))
+            else:
+                raise ConfigError(f"{where}: mixer type '{kind}' is not supported (attention, latent_attention, mamba2)")
+            mlp = entry.get("mlp")
+            ff = 0
+            if mlp is not None:
+                if _need(mlp, "kind", where + ".mlp") != "dense":
+                    raise ConfigError(f"{where}.mlp: kind '{mlp['kind']}' is not supported (dense)")
+                ff = int(_need(mlp, "ff", where + ".mlp"))
+                if ff <= 0:
+                    raise ConfigError(f"{where}.mlp: ff must be positive")
+            layers.append(VogolixLayer(kind, mixer, ff))
+        eos = cfg.get("eos_token_id")
+        eos = [] if eos is None else ([eos] if isinstance(eos, int) else list(eos))
+        bos = cfg.get("bos_token_id")
+        c = cls(architecture="Vogolix", vocab_size=int(_need(cfg, "vocab")), hidden_size=int(_need(cfg, "width")),
+                max_position_embeddings=int(cfg.get("max_positions", 1 << 30)),
+                bos_token_id=int(bos) if bos is not None else -1, eos_token_ids=tuple(int(e) for e in eos),
+                norm_eps=float(_need(_need(cfg, "norm"), "eps", "norm")), logit_scale=float(cfg.get("logit_scale", 1.0)),
+                layers=tuple(layers))
+        c.validate()
+        return c
+
+    def validate(self) -> None:
+        if self.vocab_size <= 0 or self.hidden_size <= 0 or not self.layers:
+            raise ConfigError("vocab, width and the number of layers must be positive")
+        if not self.norm_eps > 0:
+            raise ConfigError(f"norm.eps must be positive, got {self.norm_eps}")
+        for i, layer in enumerate(self.layers):
+            m = layer.mixer
+            mw = f"layers[{i}].mixer"
+            if m.heads <= 0 or m.vdim <= 0:
+                raise ConfigError(f"{mw}: heads and vdim must be positive")
+            rot = getattr(m, "rot", None)
+            if rot is not None and (rot.dims <= 0 or rot.dims % 2 != 0 or not rot.base > 0):
+                raise ConfigError(f"{mw}: rot.dims must be even and positive, rot.base positive")
+            if layer.type == "attention":
+                if m.kv_heads <= 0 or m.heads % m.kv_heads != 0 or m.dim <= 0:
+                    raise ConfigError(f"{mw}: heads must be a multiple of kv_heads, dim positive")
+                if m.chunk < 0:
+                    raise ConfigError(f"{mw}: mask.size must not be negative")
+                if rot is not None and rot.dims > m.dim:
+                    raise ConfigError(f"{mw}: rot.dims must be at most dim")
+                if m.kv_from is not None:
+                    src = self.layers[m.kv_from] if 0 <= m.kv_from < i else None
+                    if src is None or src.type != "attention" or src.mixer.kv_from is not None:
+                        raise ConfigError(f"{mw}: kv_from must name an earlier attention layer with keys of its own")
+                    if (src.mixer.kv_heads, src.mixer.dim, src.mixer.vdim, src.mixer.rot) != (m.kv_heads, m.dim, m.vdim, m.rot):
+                        raise ConfigError(f"{mw}: kv_heads, dim, vdim and rot must equal those of layer {m.kv_from}")
+            elif layer.type == "latent_attention":
+                if m.dim <= 0 or m.kv_rank <= 0 or m.rot_dim < 0 or m.window < 0:
+                    raise ConfigError(f"{mw}: dim and kv_rank must be positive, mask.size not negative")
+                if m.rot_dim > 0 and rot is None:
+                    raise ConfigError(f"{mw} has no 'rot'")
+                if rot is not None and rot.dims > m.rot_dim:
+                    raise ConfigError(f"{mw}: rot.dims must be at most rot_dim")
+            else:
+                if min(m.state, m.groups, m.norm_groups, m.conv) <= 0:
+                    raise ConfigError(f"{mw}: state, groups, norm_groups and conv must be positive")
+                if m.heads % m.groups != 0:
+                    raise ConfigError(f"{mw}: heads must be a multiple of groups")
+                if (m.heads * m.vdim) % m.norm_groups != 0:
+                    raise ConfigError(f"{mw}: the joined heads must form norm_groups equal parts")
+
+    def to_hf(self) -> Dict[str, Any]:
+        layers = []
+        for layer in self.layers:
+            m = layer.mixer
+            if layer.type == "attention":
+                mixer: Dict[str, Any] = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale}
+                span = m.chunk
+            elif layer.type == "latent_attention":
+                mixer = {"heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank,
+                         "scale": m.scale}
+                span = m.window
+            else:
+                mixer = {"heads": m.heads, "vdim": m.vdim, "state": m.state, "groups": m.groups, "norm_groups": m.norm_groups,
+                         "conv": m.conv}
+                span = 0
+            if span > 0:
+                mixer["mask"] = {"size": span}
+            if getattr(m, "rot", None) is not None:
+                mixer["rot"] = {"base": m.rot.base, "dims": m.rot.dims}
+            if getattr(m, "kv_from", None) is not None:
+                mixer["kv_from"] = m.kv_from
+            layers.append({"type": layer.type, "mixer": mixer, "mlp": {"kind": "dense", "ff": layer.ff} if layer.ff > 0 else None})
+        out: Dict[str, Any] = {"architecture": "Vogolix", "vocab": self.vocab_size, "width": self.hidden_size,
+                               "norm": {"eps": self.norm_eps}, "logit_scale": self.logit_scale, "layers": layers}
+        if self.bos_token_id >= 0:
+            out["bos_token_id"] = self.bos_token_id
+        if self.eos_token_ids:
+            out["eos_token_id"] = list(self.eos_token_ids)
+        return out

@@ -6,6 +6,7 @@
 //
 //   query row (h, m) of token i:   s_j = cap * tanh(scale * q_{h,m} . k_{g,m,j} / cap),  g = h / (H / G)
 //   key j is visible from i when    j <= i and (i - j < window or j < keep_first)      (window 0: all)
+//                      or, chunked, j <= i and floor(j / chunk) = floor(i / chunk)
 //   a_{h,m} = softmax_j(s) V_g
 //   M = 1:  o_h = a_{h,0};          M = 2:  o_h = a_{h,0} - lambda * a_{h,1}
 //   sink:       a learned number per head joins the softmax's denominator, exp(sink_h) once, with no key and
@@ -55,6 +56,7 @@ constexpr int kRows = 4;                     // query rows per pass over the key
 
 struct MaskArgs {
   int window, keep_first;
+  int chunk;             // > 0: positions see the keys of their own chunk only (no window then)
 };
 
 // What follows the softmax: a sink in the denominator, a gate on the output.
@@ -72,19 +74,23 @@ __device__ __forceinline__ float gate_factor(const TailArgs<T>& t, size_t tok, i
   return 1.f / (1.f + expf(-g));
 }
 
-__device__ __forceinline__ bool key_visible(int j, int i, const MaskArgs& mk) {
-  return j <= i && (mk.window <= 0 || i - j < mk.window || j < mk.keep_first);
+// The first key that position i sees (apart from kept first ones); it never falls as i grows.
+__device__ __forceinline__ int first_key(int i, const MaskArgs& mk) {
+  if (mk.chunk > 0) return i / mk.chunk * mk.chunk;
+  return mk.window > 0 ? max(i - mk.window + 1, 0) : 0;
 }
-// Whether key j is behind the window of position i and of every later one, and not kept: its page may have
-// been given back, so it is not read at all (a masked weight of zero times a stray NaN would be NaN).
-__device__ __forceinline__ bool dead_key(int j, int i, const MaskArgs& mk) {
-  return mk.window > 0 && j >= mk.keep_first && j <= i - mk.window;
+// Whether position i, whose first key is `first`, sees key j.
+__device__ __forceinline__ bool key_visible(int j, int i, int first, const MaskArgs& mk) {
+  return j <= i && (j >= first || j < mk.keep_first);
 }
-// Whether keys [lo, hi) hold one that position i sees.
-__device__ __forceinline__ bool range_visible(int lo, int hi, int i, const MaskArgs& mk) {
-  if (lo > i || lo >= hi) return false;
-  if (mk.window <= 0) return true;
-  return lo < mk.keep_first || hi > i - mk.window + 1;
+// Whether key j lies before the first key of a position and so of every later one, and is not kept: its page may
+// have been given back, so it is not read at all (a masked weight of zero times a stray NaN would be NaN).
+__device__ __forceinline__ bool dead_key(int j, int first, const MaskArgs& mk) {
+  return j >= mk.keep_first && j < first;
+}
+// Whether keys [lo, hi) hold one that position i, whose first key is `first`, sees.
+__device__ __forceinline__ bool range_visible(int lo, int hi, int i, int first, const MaskArgs& mk) {
+  return lo <= i && lo < hi && (lo < mk.keep_first || hi > first);
 }
 
 template <typename T>
@@ -135,7 +141,8 @@ maps_decode_kernel(const MapsDecodeArgs<T> a) {
   const int me = ctx - 1;                                // the query's position
   const int base = part * kPart;
   const int j_hi = min(ctx, base + kPart);
-  if (!range_visible(base, j_hi, me, a.mask)) return;
+  const int first = first_key(me, a.mask);
+  if (!range_visible(base, j_hi, me, first, a.mask)) return;
   const int lane8 = threadIdx.x % kLPK, slot = threadIdx.x / kLPK;
   const int warp = threadIdx.x >> 5;
   const int32_t* bt = a.block_table + static_cast<size_t>(seq) * a.max_blocks;
@@ -145,7 +152,7 @@ maps_decode_kernel(const MapsDecodeArgs<T> a) {
 #pragma unroll
   for (int it = 0; it < kPart / kKeysPerIter; ++it) {
     const int j = base + it * kKeysPerIter + slot;
-    pages[it] = (j < j_hi && key_visible(j, me, a.mask)) ? bt[j / a.page_size] : 0;
+    pages[it] = (j < j_hi && key_visible(j, me, first, a.mask)) ? bt[j / a.page_size] : 0;
   }
 
   for (int m = 0; m < kM; ++m) {
@@ -164,7 +171,7 @@ maps_decode_kernel(const MapsDecodeArgs<T> a) {
 #pragma unroll
       for (int it = 0; it < kPart / kKeysPerIter; ++it) {
         const int j = base + it * kKeysPerIter + slot;
-        const bool live = j < j_hi && key_visible(j, me, a.mask);
+        const bool live = j < j_hi && key_visible(j, me, first, a.mask);
         const size_t page = live ? pages[it] : 0;
         const T* kp = a.kcache + ((page * (a.kv_heads * kM) + khead) * a.page_size + j % a.page_size) * kD;
         float dot[kRows];
@@ -227,7 +234,7 @@ maps_decode_kernel(const MapsDecodeArgs<T> a) {
 #pragma unroll
       for (int it = 0; it < kPart / kKeysPerIter; ++it) {
         const int j = base + it * kKeysPerIter + slot;
-        if (j >= j_hi || !key_visible(j, me, a.mask)) continue;
+        if (j >= j_hi || !key_visible(j, me, first, a.mask)) continue;
         const size_t page = pages[it];
         const T* vp = a.vcache + ((page * a.kv_heads + kvh) * a.page_size + j % a.page_size) * kVS;
         float p[kRows];
@@ -302,21 +309,22 @@ maps_merge_kernel(const MapsDecodeArgs<T> a) {
   const int4 info = a.items[item];
   const int tok = info.x, ctx = info.z;
   const int me = ctx - 1;
-  const int p_hi = me / kPart;
+  const int p_hi = me / kPart, first = first_key(me, a.mask);
+  const int p_lo = a.mask.keep_first > 0 ? 0 : first / kPart;
   for (int d = threadIdx.x; d < kDV; d += kThreads) o[d] = 0.f;
   __syncthreads();
   for (int m = 0; m < kM; ++m) {
     const size_t row0 = (static_cast<size_t>(item) * (a.heads * kM) + head * kM + m) * a.max_parts;
     float mx = -INFINITY;
-    for (int p = 0; p <= p_hi; ++p)
-      if (range_visible(p * kPart, min(ctx, (p + 1) * kPart), me, a.mask)) mx = fmaxf(mx, a.part_ml[(row0 + p) * 2]);
+    for (int p = p_lo; p <= p_hi; ++p)
+      if (range_visible(p * kPart, min(ctx, (p + 1) * kPart), me, first, a.mask)) mx = fmaxf(mx, a.part_ml[(row0 + p) * 2]);
     const float coef = m == 0 ? 1.f : -a.lambda;
     const bool sunk = kM == 1 && a.tail.sink != nullptr;
     if (sunk) mx = fmaxf(mx, a.tail.sink[head]);
     for (int d = threadIdx.x; d < kDV; d += kThreads) {
       float num = 0.f, den = sunk ? expf(a.tail.sink[head] - mx) : 0.f;
-      for (int p = 0; p <= p_hi; ++p) {
-        if (!range_visible(p * kPart, min(ctx, (p + 1) * kPart), me, a.mask)) continue;
+      for (int p = p_lo; p <= p_hi; ++p) {
+        if (!range_visible(p * kPart, min(ctx, (p + 1) * kPart), me, first, a.mask)) continue;
         const float w = expf(a.part_ml[(row0 + p) * 2] - mx);
         num += w * a.part_o[(row0 + p) * kDV + d];
         den += w * a.part_ml[(row0 + p) * 2 + 1];
@@ -382,6 +390,7 @@ maps_prefill_kernel(const MapsPrefillArgs<T> a) {
   const int32_t* bt = a.block_table + static_cast<size_t>(seq) * a.max_blocks;
   const int r = threadIdx.x >> 2, cq = threadIdx.x & 3;
   const int my_pos = pos0 + r;
+  const int first0 = first_key(pos0, a.mask), my_first = first_key(my_pos, a.mask);      // of the CTA's rows, of this row
   const int k_end = pos0 + rows;     // exclusive
   const float inv_cap = a.softcap > 0.f ? 1.f / a.softcap : 0.f;
   const float slope = a.tail.slopes != nullptr ? a.tail.slopes[head] : 0.f;
@@ -404,16 +413,18 @@ maps_prefill_kernel(const MapsPrefillArgs<T> a) {
     for (int i = 0; i < kVQ; ++i) acc[i] = 0.f;
 
     for (int k0 = 0; k0 < k_end; k0 += kBK) {
-      // a tile that no row of this CTA sees is skipped: the rows' windows together reach back to
-      // pos0 - window + 1, and the kept first tokens are seen by all
-      const int t_hi = min(k0 + kBK, k_end);
-      if (a.mask.window > 0 && k0 >= a.mask.keep_first && t_hi <= pos0 - a.mask.window + 1) continue;
+      // a tile that no row of this CTA sees is skipped: the rows together reach back to the first row's first
+      // key, and the kept first tokens are seen by all
+      if (k0 >= a.mask.keep_first && min(k0 + kBK, k_end) <= first0) {
+        k0 = first0 / kBK * kBK - kBK;
+        continue;
+      }
       __syncthreads();
       for (int i = threadIdx.x; i < kBK * kD; i += kThreads) {
         const int key = i / kD, d = i - key * kD;
         const int j = k0 + key;
         float v = 0.f;
-        if (j < k_end && !dead_key(j, pos0, a.mask)) {
+        if (j < k_end && !dead_key(j, first0, a.mask)) {
           const size_t page = bt[j / a.page_size];
           v = to_float(a.kcache[((page * (a.kv_heads * kM) + kvh * kM + m) * a.page_size + j % a.page_size) * kD + d]);
         }
@@ -423,7 +434,7 @@ maps_prefill_kernel(const MapsPrefillArgs<T> a) {
         const int key = i / kDV, d = i - key * kDV;
         const int j = k0 + key;
         float v = 0.f;
-        if (j < k_end && !dead_key(j, pos0, a.mask)) {
+        if (j < k_end && !dead_key(j, first0, a.mask)) {
           const size_t page = bt[j / a.page_size];
           v = to_float(a.vcache[((page * a.kv_heads + kvh) * a.page_size + j % a.page_size) * kVS + d]);
         }
@@ -442,7 +453,7 @@ maps_prefill_kernel(const MapsPrefillArgs<T> a) {
 #pragma unroll
       for (int i = 0; i < kBK / 4; ++i) {
         const int kp = k0 + cq + 4 * i;
-        const bool ok = (r < rows) && key_visible(kp, my_pos, a.mask);
+        const bool ok = (r < rows) && key_visible(kp, my_pos, my_first, a.mask);
         float v = s[i];
         if (a.softcap > 0.f) v = a.softcap * tanhf(v * inv_cap);
         v -= slope * static_cast<float>(my_pos - kp);
@@ -573,6 +584,8 @@ maps_prefill_mma_kernel(const MapsPrefillArgs<bf16> a) {
   const int r0 = warp * 16 + gid, r1 = r0 + 8;                   // this thread's two rows within the CTA's 64
   const int p0 = pos0 + r0, p1 = pos0 + r1;
   const bool ok0 = r0 < rows, ok1 = r1 < rows;
+  const int first0 = first_key(pos0, a.mask);                    // of the CTA's rows; and of this thread's
+  const int f0 = first_key(p0, a.mask), f1 = first_key(p1, a.mask);
   const float inv_cap = a.softcap > 0.f ? 1.f / a.softcap : 0.f;
   const float slope = a.tail.slopes != nullptr ? a.tail.slopes[head] : 0.f;
   const int ps_shift = __ffs(a.page_size) - 1, ps_mask = a.page_size - 1;      // (pages hold a power of two of tokens)
@@ -598,10 +611,7 @@ maps_prefill_mma_kernel(const MapsPrefillArgs<bf16> a) {
 
     // the visible key tiles in turn; the next one is on its way (cp.async) while this one is worked on
     auto next_visible = [&](int k0) {
-      while (k0 < k_end && a.mask.window > 0 && k0 >= a.mask.keep_first &&
-             min(k0 + kTK, k_end) <= pos0 - a.mask.window + 1)
-        k0 += kTK;
-      return k0;
+      return (k0 >= a.mask.keep_first && min(k0 + kTK, k_end) <= first0) ? max(first0 / kTK * kTK, k0) : k0;
     };
     auto issue = [&](int stage, int k0) {
       bf16* Kd = Kst + stage * kTK * kLDK;
@@ -610,7 +620,7 @@ maps_prefill_mma_kernel(const MapsPrefillArgs<bf16> a) {
         const int key = i / (kD / 8), c = i - key * (kD / 8);
         const int j = k0 + key;
         bf16* d = Kd + key * kLDK + c * 8;
-        if (j < k_end && !dead_key(j, pos0, a.mask)) {
+        if (j < k_end && !dead_key(j, first0, a.mask)) {
           const size_t page = bt[j >> ps_shift];
           cp_async16(d, a.kcache + ((page * (a.kv_heads * kM) + kvh * kM + m) * a.page_size + (j & ps_mask)) * kD + c * 8);
         } else {
@@ -621,7 +631,7 @@ maps_prefill_mma_kernel(const MapsPrefillArgs<bf16> a) {
         const int key = i / (kDV / 8), c = i - key * (kDV / 8);
         const int j = k0 + key;
         bf16* d = Vd + key * kLDV + c * 8;
-        if (j < k_end && !dead_key(j, pos0, a.mask)) {
+        if (j < k_end && !dead_key(j, first0, a.mask)) {
           const size_t page = bt[j >> ps_shift];
           cp_async16(d, a.vcache + ((page * a.kv_heads + kvh) * a.page_size + (j & ps_mask)) * kVS + c * 8);
         } else {
@@ -671,7 +681,7 @@ maps_prefill_mma_kernel(const MapsPrefillArgs<bf16> a) {
           float v = s[nt][e] * a.scale;
           if (a.softcap > 0.f) v = a.softcap * tanh_fast(v * inv_cap);
           v -= slope * static_cast<float>(((e < 2) ? p0 : p1) - j);
-          const bool vis = (e < 2) ? (ok0 && key_visible(j, p0, a.mask)) : (ok1 && key_visible(j, p1, a.mask));
+          const bool vis = (e < 2) ? (ok0 && key_visible(j, p0, f0, a.mask)) : (ok1 && key_visible(j, p1, f1, a.mask));
           v = vis ? v : -INFINITY;
           s[nt][e] = v;
           if (e < 2) t0 = fmaxf(t0, v);
@@ -831,7 +841,7 @@ static bool g_simt_attr_set[2] = {false, false};
 template <typename T>
 int launch_maps_decode(const void* q, int q_stride, const void* kc, const void* vc, const int32_t* bt, int max_blocks,
                        const int32_t* items, float* part_o, float* part_ml, int max_parts, void* out, int out_stride,
-                       int nitems, int heads, int kv_heads, int page_size, int window, int keep_first, float scale,
+                       int nitems, int heads, int kv_heads, int page_size, int window, int keep_first, int chunk, float scale,
                        float softcap, float lambda, float post_scale, float eps, int unit_norm, const float* sink,
                        const float* slopes, const void* gate, int gate_stride, int gate_mode, cudaStream_t stream) {
   MapsDecodeArgs<T> a;
@@ -857,6 +867,7 @@ int launch_maps_decode(const void* q, int q_stride, const void* kc, const void* 
   a.page_size = page_size;
   a.mask.window = window;
   a.mask.keep_first = keep_first;
+  a.mask.chunk = chunk;
   a.scale = scale;
   a.softcap = softcap;
   a.lambda = lambda;
@@ -875,7 +886,7 @@ template <typename T>
 int launch_maps_prefill(const void* q, int q_stride, const void* kc, const void* vc, const int32_t* bt, int max_blocks,
                         const int32_t* tile_seq, const int32_t* tile_tok, const int32_t* tile_rows,
                         const int32_t* positions, void* out, int out_stride, int tiles, int tile_rows_max, int heads,
-                        int kv_heads, int page_size, int window, int keep_first, float scale, float softcap,
+                        int kv_heads, int page_size, int window, int keep_first, int chunk, float scale, float softcap,
                         float lambda, float post_scale, float eps, int unit_norm, const float* sink,
                         const float* slopes, const void* gate, int gate_stride, int gate_mode, int impl,
                         cudaStream_t stream) {
@@ -903,6 +914,7 @@ int launch_maps_prefill(const void* q, int q_stride, const void* kc, const void*
   a.tile_quarters = (tile_rows_max + kBQ - 1) / kBQ;
   a.mask.window = window;
   a.mask.keep_first = keep_first;
+  a.mask.chunk = chunk;
   a.scale = scale;
   a.softcap = softcap;
   a.lambda = lambda;
@@ -948,34 +960,34 @@ int rl_maps_partition() { return kPart; }
 int rl_maps_decode(int dtype, const void* q, int q_stride, const void* kc, const void* vc, const int32_t* bt,
                    int max_blocks, const int32_t* items, float* part_o, float* part_ml, int max_parts, void* out,
                    int out_stride, int nitems, int heads, int kv_heads, int page_size, int window, int keep_first,
-                   float scale, float softcap, float lambda, float post_scale, float eps, int unit_norm,
+                   int chunk, float scale, float softcap, float lambda, float post_scale, float eps, int unit_norm,
                    const float* sink, const float* slopes, const void* gate, int gate_stride, int gate_mode,
                    cudaStream_t stream) {
   if (nitems <= 0 || max_parts <= 0) return 0;
   if (dtype == 0)
     return launch_maps_decode<float>(q, q_stride, kc, vc, bt, max_blocks, items, part_o, part_ml, max_parts, out,
-                                     out_stride, nitems, heads, kv_heads, page_size, window, keep_first, scale, softcap,
+                                     out_stride, nitems, heads, kv_heads, page_size, window, keep_first, chunk, scale, softcap,
                                      lambda, post_scale, eps, unit_norm, sink, slopes, gate, gate_stride, gate_mode, stream);
   return launch_maps_decode<bf16>(q, q_stride, kc, vc, bt, max_blocks, items, part_o, part_ml, max_parts, out,
-                                  out_stride, nitems, heads, kv_heads, page_size, window, keep_first, scale, softcap,
+                                  out_stride, nitems, heads, kv_heads, page_size, window, keep_first, chunk, scale, softcap,
                                   lambda, post_scale, eps, unit_norm, sink, slopes, gate, gate_stride, gate_mode, stream);
 }
 
 int rl_maps_prefill(int dtype, const void* q, int q_stride, const void* kc, const void* vc, const int32_t* bt,
                     int max_blocks, const int32_t* tile_seq, const int32_t* tile_tok, const int32_t* tile_rows,
                     const int32_t* positions, void* out, int out_stride, int tiles, int tile_rows_max, int heads,
-                    int kv_heads, int page_size, int window, int keep_first, float scale, float softcap, float lambda,
+                    int kv_heads, int page_size, int window, int keep_first, int chunk, float scale, float softcap, float lambda,
                     float post_scale, float eps, int unit_norm, const float* sink, const float* slopes, const void* gate,
                     int gate_stride, int gate_mode, int impl, cudaStream_t stream) {
   if (tiles <= 0) return 0;
   if (dtype == 0)
     return launch_maps_prefill<float>(q, q_stride, kc, vc, bt, max_blocks, tile_seq, tile_tok, tile_rows, positions,
                                       out, out_stride, tiles, tile_rows_max, heads, kv_heads, page_size, window,
-                                      keep_first, scale, softcap, lambda, post_scale, eps, unit_norm, sink, slopes, gate, gate_stride,
+                                      keep_first, chunk, scale, softcap, lambda, post_scale, eps, unit_norm, sink, slopes, gate, gate_stride,
                                       gate_mode, impl, stream);
   return launch_maps_prefill<bf16>(q, q_stride, kc, vc, bt, max_blocks, tile_seq, tile_tok, tile_rows, positions,
                                    out, out_stride, tiles, tile_rows_max, heads, kv_heads, page_size, window,
-                                   keep_first, scale, softcap, lambda, post_scale, eps, unit_norm, sink, slopes, gate, gate_stride,
+                                   keep_first, chunk, scale, softcap, lambda, post_scale, eps, unit_norm, sink, slopes, gate, gate_stride,
                                       gate_mode, impl, stream);
 }
 

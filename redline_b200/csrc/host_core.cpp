@@ -75,6 +75,7 @@ struct Core {
   std::vector<Pool> pools;
   std::vector<int> windows;                    // per group; 0: every key is kept
   std::vector<int> keep_first;                 // per group: a window never passes the first so many keys
+  std::vector<int> chunked;                    // per group: 1 if its "window" is a chunk size (visible keys begin at a multiple of it)
   std::vector<int> free_slots;
   int num_state_slots = 0;
   std::vector<Request> reqs;
@@ -123,12 +124,22 @@ void* rl_hc_create(int num_groups, const int32_t* pages_per_group, const int32_t
   c->pools.resize(num_groups);
   c->windows.assign(windows, windows + num_groups);
   c->keep_first.assign(num_groups, 0);
+  c->chunked.assign(num_groups, 0);
   for (int g = 0; g < num_groups; ++g) c->pools[g].init(pages_per_group[g], 1);
   c->num_state_slots = num_state_slots;
   for (int s = num_state_slots - 1; s >= 0; --s) c->free_slots.push_back(s);   // slot 0 first
   return c;
 }
 void rl_hc_destroy(void* h) { delete static_cast<Core*>(h); }
+
+// The window of group `group` is a chunk of positions: a token sees the keys of its own chunk only, so that a
+// chunk's keys are dead as a whole once the next one begins.  To be called before any request is opened.
+int rl_hc_set_chunked(void* h, int group) {
+  Core* c = static_cast<Core*>(h);
+  if (group < 0 || group >= static_cast<int>(c->chunked.size()) || c->windows[group] <= 0) return -1;
+  c->chunked[group] = 1;
+  return 0;
+}
 
 // The first `keys` keys of every sequence stay visible in window group `group`: their pages are not
 // released when the window passes them.  To be called before any request is opened.
@@ -221,7 +232,8 @@ int rl_hc_reserve(void* h, int rid, int new_len) {
 }
 
 // After num_computed positions are in the cache: in window groups, frees the pages whose keys no
-// later token can see (key j is dead when j <= n - window for the next position n).  Pages freed.
+// later token can see (key j is dead when j <= n - window for the next position n, or with chunks when it lies
+// before n's chunk).  Pages freed.
 int rl_hc_release_passed(void* h, int rid, int num_computed) {
   Core* c = static_cast<Core*>(h);
   Request* r = c->get(rid);
@@ -230,7 +242,8 @@ int rl_hc_release_passed(void* h, int rid, int num_computed) {
   for (size_t g = 0; g < c->pools.size(); ++g) {
     const int w = c->windows[g];
     if (w <= 0) continue;
-    const int dead_keys = num_computed - w + 1;               // keys 0 .. dead_keys-1 are dead
+    // keys 0 .. dead_keys-1 are dead
+    const int dead_keys = c->chunked[g] ? num_computed / w * w : num_computed - w + 1;
     int dead_blocks = std::max(0, dead_keys) / c->page_size;
     dead_blocks = std::min<int>(dead_blocks, static_cast<int>(r->tables[g].size()));
     if (dead_blocks > std::max(r->released_upto[g], c->kept_blocks(g))) {

@@ -15,8 +15,8 @@
 //                 token's position (entry i with entry i + dims/2 of the first `dims` rotated entries, or
 //                 neighbours, cos and sin from tables), [c | k_r] into the paged cache, q_r into the
 //                 attention's query rows; the norm of the queries' latent
-//   head_linear   y[t, h, :] = W_h x[t, h, :] for every head h, W [heads, n, k], float32 sums; the heads'
-//                 rotated query parts may go along; FFMA for float32, mma.sync.m16n8k16 for bfloat16
+//   head_linear   y[t, h, :] = W_h x[t, h, :] for every head h, W [heads, n, k], float32 sums, times
+//                 sigmoid(gate[t, h, :]) where a gate is given; the heads' rotated query parts may go along; FFMA for float32, mma.sync.m16n8k16 for bfloat16
 //                 operands whose sizes allow it, and a kernel that streams the weights for up to 16 tokens
 #include "common.cuh"
 
@@ -128,7 +128,17 @@ struct HeadLinearArgs {
   int x_ld, x_col, x_head;
   int y_ld, y_col, y_head;
   Turn turn;
+  const void* gate;        // [tokens, heads * n] in rows of gate_ld entries of the activation type, or null
+  int gate_ld;
 };
+
+// The factor of output j of head h for token t.
+template <typename TA>
+__device__ __forceinline__ float gate_of(const HeadLinearArgs& a, int t, int h, int j) {
+  if (a.gate == nullptr) return 1.f;
+  const float g = to_float(static_cast<const TA*>(a.gate)[static_cast<size_t>(t) * a.gate_ld + h * a.n + j]);
+  return 1.f / (1.f + expf(-g));
+}
 
 // The rotated parts of tokens t0 .. t0 + rows - 1 of head h, by all threads of a CTA.
 template <typename TA>
@@ -194,7 +204,8 @@ head_linear_kernel(const TA* __restrict__ x, const TW* __restrict__ w, TA* __res
 #pragma unroll
     for (int r = 0; r < kHlRows; ++r)
       if (t0 + r < a.tokens)
-        y[static_cast<size_t>(t0 + r) * a.y_ld + a.y_col + h * a.y_head + j] = from_float<TA>(acc[r]);
+        y[static_cast<size_t>(t0 + r) * a.y_ld + a.y_col + h * a.y_head + j] =
+            from_float<TA>(acc[r] * gate_of<TA>(a, t0 + r, h, j));
   }
 }
 
@@ -253,10 +264,10 @@ head_linear_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, b
     if (j0 + nt * 8 >= a.n) continue;
     if (ok0)
       *reinterpret_cast<__nv_bfloat162*>(y + static_cast<size_t>(r0) * a.y_ld + a.y_col + h * a.y_head + j) =
-          __floats2bfloat162_rn(acc[nt][0], acc[nt][1]);
+          __floats2bfloat162_rn(acc[nt][0] * gate_of<bf16>(a, r0, h, j), acc[nt][1] * gate_of<bf16>(a, r0, h, j + 1));
     if (ok1)
       *reinterpret_cast<__nv_bfloat162*>(y + static_cast<size_t>(r1) * a.y_ld + a.y_col + h * a.y_head + j) =
-          __floats2bfloat162_rn(acc[nt][2], acc[nt][3]);
+          __floats2bfloat162_rn(acc[nt][2] * gate_of<bf16>(a, r1, h, j), acc[nt][3] * gate_of<bf16>(a, r1, h, j + 1));
   }
 }
 
@@ -319,7 +330,8 @@ head_linear_few_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, b
     for (int t = 0; t < kHfTokens; ++t) {
       const float v = warp_sum(acc[f][t]);
       if (lane == 0 && t < nt && j0 + f < a.n)
-        y[static_cast<size_t>(t0 + t) * a.y_ld + a.y_col + h * a.y_head + j0 + f] = __float2bfloat16_rn(v);
+        y[static_cast<size_t>(t0 + t) * a.y_ld + a.y_col + h * a.y_head + j0 + f] =
+            __float2bfloat16_rn(v * gate_of<bf16>(a, t0 + t, h, j0 + f));
     }
 }
 
@@ -368,9 +380,11 @@ int rl_latent_prep(int act_dtype, int w_dtype, const void* q, int q_src_ld, cons
 int rl_head_linear(int act_dtype, int w_dtype, const void* x, int x_ld, int x_col, int x_head, const void* w, int heads,
                    int n, int k, void* y, int y_ld, int y_col, int y_head, int tokens, int impl, int turn_dims,
                    int rot_dims, int pairs, int turn_x, int turn_y, const float* cos_t, const float* sin_t, int max_pos,
-                   const int32_t* positions, int* status, cudaStream_t stream) {
+                   const int32_t* positions, int* status, const void* gate, int gate_ld, cudaStream_t stream) {
   if (tokens <= 0 || heads <= 0 || n <= 0) return 0;
   HeadLinearArgs a;
+  a.gate = gate;
+  a.gate_ld = gate_ld;
   a.tokens = tokens;
   a.heads = heads;
   a.n = n;

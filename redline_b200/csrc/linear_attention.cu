@@ -4,8 +4,11 @@
 //   one decay per head           S_t = a_h S_(t-1) + k_t v_t^T,            o_t = S_t^T q_t
 //   a decay per token and key    o_t = S_(t-1)^T q_t + (sum_i q_i u_i k_i) v_t,
 //   channel, with a bonus        S_t = diag(a_t) S_(t-1) + k_t v_t^T,      a_t = exp(-exp(z_t + b))
+//   a decay per token (state     S_t = exp(-exp(A_h) d_t) S_(t-1) + d_t k_t v_t^T,   d_t = softplus(z_t + b_h),
+//   space), with a skip          o_t = S_t^T q_t + D_h v_t;   neighbouring heads share their q and k
 //
-// (the second form's read-out sees the token's own write through the bonus u only).  One kernel serves prompt
+// (the second form's read-out sees the token's own write through the bonus u only).  The third form is a module of
+// its own (compiled with -DRL_LIN_TOKEN=1).  One kernel serves prompt
 // portions and single tokens: a CTA takes one sequence of the step, one head and a block of value columns.
 // Columns of S never mix.  A thread keeps four neighbouring columns of a group of eight rows in registers, as
 // pairs of rows (fma.rn.f32x2: two rows per instruction, each rounded as a single fma); the G = 1 to 32 groups
@@ -50,6 +53,7 @@ constexpr int kMaxThreads = 256;
 constexpr int kTcMinTokens = 16, kTcMaxCols = 128;                     // blocks of tokens on the tensor cores: from so many on
 
 enum { GATE_NONE = 0, GATE_SIGMOID = 1, GATE_SILU = 2 };
+enum { PER_HEAD = 0, PER_CHANNEL = 1, PER_TOKEN = 2 };                 // the kind of decay
 
 template <typename T>
 struct LinArgs {
@@ -76,6 +80,9 @@ struct LinArgs {
   float* chunk_state;            // [sequences, chunks, heads, D, DV] (chunked passes only)
   float* chunk_decay;            // per channel: [sequences, chunks, heads, D]
   int* status;
+  const T* steps;                // per token: z, head h of token t at steps + t * steps_ld + h
+  int steps_ld, qk_heads;        // heads of q and k (head h reads h / (heads / qk_heads))
+  const float *step_bias, *a_log, *skip;         // per token: b, A and D of every head
   int tokens, heads, dv, chunk, max_chunks;
   int quads_ok;                  // column quadruples of the state start on 16-byte boundaries
   int qk_ok, v_ok, g_ok, z_ok, rot_ok; // rows of q and k / values / gates / decays / tables are made of 16-byte pieces
@@ -105,6 +112,9 @@ __device__ __forceinline__ float gate_value(float g, int mode) {
 }
 // (the inner exponential's relative error is that of the distance of the decay from 1)
 __device__ __forceinline__ float channel_decay(float z) { return expf(-__expf(z)); }
+
+// ln(1 + e^z)
+__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 __device__ __forceinline__ void async_copy16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<unsigned>(__cvta_generic_to_shared(dst))), "l"(src));
@@ -167,9 +177,10 @@ __device__ __forceinline__ float2 load2(const bf16* p) { return __bfloat1622floa
 // mode 3: chunk c from its starting state as pass 2 left it (chunk_state[seq][c - 1]: the state after chunk
 //         c - 1; for c = 0 the slot's state, which pass 2 has copied to the entry of the last chunk, since
 //         the last chunk's CTA overwrites the slot), outputs written; the last chunk writes the slot
-template <typename T, int MODE, bool CHANNEL>
+template <typename T, int MODE, int KIND>
 __global__ void __launch_bounds__(kMaxThreads, 2)
 linear_attention_kernel(const LinArgs<T> a) {
+  constexpr bool CHANNEL = KIND == PER_CHANNEL, TOKEN = KIND == PER_TOKEN;
   pdl_launch();
   pdl_wait();
   __shared__ __align__(16) float qs[MODE == 1 ? 1 : kTok][kSm];
@@ -177,9 +188,11 @@ linear_attention_kernel(const LinArgs<T> a) {
   __shared__ __align__(16) float as[CHANNEL ? kTok : 1][kSm];
   __shared__ __align__(8) float us[CHANNEL && MODE != 1 ? kD : 1], db[CHANNEL ? kD : 1];      // per channel: the head's bonus and decay bias
   __shared__ float bs[kTok];                       // per channel: sum_i q_i u_i k_i of every staged token
+  __shared__ float ds[2][TOKEN ? kTok : 1], es[2][TOKEN ? kTok : 1];      // per token: d and the decay of every staged token
   extern __shared__ __align__(16) unsigned char raw[];     // two buffers, the values, the read-outs (RawLayout)
   const int seq = blockIdx.z, head = blockIdx.y % a.heads, c = blockIdx.y / a.heads;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+  const int qk_head = TOKEN ? head / (a.heads / a.qk_heads) : head;
   const int group = lane / kSlots;
   const int block_cols = nwarps * kSlots * kCols;
   const int col0 = blockIdx.x * block_cols;                               // the CTA's first column
@@ -211,8 +224,10 @@ linear_attention_kernel(const LinArgs<T> a) {
 
   // tokens tb .. tb + nt - 1 on their way into buffer b: a warp takes one token at a time, its lanes the pieces of
   // the token's parts, one part after another
+  float z_ahead = 0.f;               // per token: this thread's token's z of the batch on its way
   auto stage = [&](int b, int tb, int nt) {
     constexpr int E = sizeof(T);
+    if (TOKEN && threadIdx.x < nt) z_ahead = to_float(a.steps[static_cast<size_t>(tb + threadIdx.x) * a.steps_ld + head]);
     for (int tt = warp; tt < nt; tt += nwarps) {
       unsigned char* buf = raw + b * lay.bytes;
       const size_t t = tb + tt;
@@ -225,8 +240,8 @@ linear_attention_kernel(const LinArgs<T> a) {
           for (int e = lane; e < bytes / 2; e += 32) reinterpret_cast<bf16*>(to)[e] = static_cast<const bf16*>(from)[e];
         }
       };
-      if (MODE != 1) part(buf + lay.q + tt * lay.qk_row, a.q + t * a.q_ld + head * kD, kD * E, a.qk_ok, E);
-      part(buf + lay.k + tt * lay.qk_row, a.k + t * a.k_ld + head * kD, kD * E, a.qk_ok, E);
+      if (MODE != 1) part(buf + lay.q + tt * lay.qk_row, a.q + t * a.q_ld + qk_head * kD, kD * E, a.qk_ok, E);
+      part(buf + lay.k + tt * lay.qk_row, a.k + t * a.k_ld + qk_head * kD, kD * E, a.qk_ok, E);
       const int cols = min(block_cols, a.dv - col0);
       part(buf + lay.v + tt * lay.v_row, a.v + t * a.v_ld + head * a.dv + col0, cols * E, a.v_ok, E);
       if (gated) part(buf + lay.g + tt * lay.v_row, a.gate + t * a.gate_ld + head * a.dv, a.dv * E, a.g_ok, E);
@@ -284,8 +299,11 @@ linear_attention_kernel(const LinArgs<T> a) {
       if (CHANNEL) (&as[0][0])[i] = 0.f;
     }
   }
-  const float decay = CHANNEL ? 0.f : a.decay[head];
+  const float decay = KIND == PER_HEAD ? a.decay[head] : 0.f;
   const f32x2 decay2 = pack2(decay, decay);
+  const float rate = TOKEN ? expf(a.a_log[head]) : 0.f, step_bias = TOKEN ? a.step_bias[head] : 0.f;
+  const float skip = TOKEN ? a.skip[head] : 0.f;
+  float all_decays = 1.f;                          // per token, mode 1, thread 0: the product of the decays
   constexpr int kPer = (kD + 31) / 32;             // channels of a lane
   float prod[CHANNEL && MODE == 1 ? kPer : 1];     // per channel, mode 1, warp 0: the products of its channels' decays
   if (CHANNEL) {
@@ -302,6 +320,11 @@ linear_attention_kernel(const LinArgs<T> a) {
   int b = 0;
   for (int tb = t0; tb < t1; tb += kTok, b ^= 1) {
     const int nt = min(kTok, t1 - tb);
+    if (TOKEN && threadIdx.x < nt) {           // (the other buffer of these is what the batch before reads)
+      const float d = softplus(z_ahead + step_bias);
+      ds[b][threadIdx.x] = d;
+      es[b][threadIdx.x] = expf(-rate * d);
+    }
     async_copies_done();
     __syncthreads();               // this batch has arrived, and the one before has been worked on
     if (tb + kTok < t1) stage(b ^ 1, tb + kTok, min(kTok, t1 - tb - kTok));
@@ -314,6 +337,7 @@ linear_attention_kernel(const LinArgs<T> a) {
       const float* cs = reinterpret_cast<const float*>(buf + lay.cs + tt * lay.rot_row);
       const float* sn = reinterpret_cast<const float*>(buf + lay.sn + tt * lay.rot_row);
       float bonus = 0.f;
+      const float k_scale = TOKEN ? ds[b][tt] : a.k_scale;
       if (kD % 2 == 0 && a.rot_pairs % 2 == 0) {
 #pragma unroll
         for (int j = 0; j < (kD + 63) / 64; ++j) {
@@ -335,7 +359,7 @@ linear_attention_kernel(const LinArgs<T> a) {
               qv = make_float2(qv.x * cv.x + qo.x * sv.x, qv.y * cv.y + qo.y * sv.y);
             }
           }
-          kv = make_float2(kv.x * a.k_scale, kv.y * a.k_scale);
+          kv = make_float2(kv.x * k_scale, kv.y * k_scale);
           *reinterpret_cast<float2*>(&ks[tt][sm]) = kv;
           if (MODE != 1) *reinterpret_cast<float2*>(&qs[tt][sm]) = qv;
           if (CHANNEL) {
@@ -358,7 +382,7 @@ linear_attention_kernel(const LinArgs<T> a) {
             kv = kv * cv + to_float(kr[other]) * sv;
             if (MODE != 1) qv = qv * cv + to_float(qr[other]) * sv;
           }
-          kv *= a.k_scale;
+          kv *= k_scale;
           ks[tt][sm] = kv;
           if (MODE != 1) qs[tt][sm] = qv;
           if (CHANNEL) {
@@ -386,6 +410,8 @@ linear_attention_kernel(const LinArgs<T> a) {
           if (d < kD) prod[j] *= as[tt][(d / kRows) * kStride + d % kRows];
         }
     }
+    if (TOKEN && MODE == 1 && threadIdx.x == 0)
+      for (int tt = 0; tt < nt; ++tt) all_decays *= es[b][tt];
     auto token = [&](int tt) {
       const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(&ks[tt][group * kStride]);
       const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(&qs[MODE == 1 ? 0 : tt][group * kStride]);
@@ -395,13 +421,14 @@ linear_attention_kernel(const LinArgs<T> a) {
       const f32x2 v2[kCols] = {va.x, va.y, vb.x, vb.y};
       f32x2 o2[kCols];
       // (the bonus counts once: in the first half of the first group's pairs)
-      const f32x2 bonus = pack2((CHANNEL && MODE != 1 && group == 0) ? bs[tt] : 0.f, 0.f);
+      const f32x2 bonus = pack2(MODE != 1 && group == 0 ? (CHANNEL ? bs[tt] : (TOKEN ? skip : 0.f)) : 0.f, 0.f);
+      const f32x2 own_decay = TOKEN ? pack2(es[b][tt], es[b][tt]) : decay2;
 #pragma unroll
-      for (int j = 0; j < kCols; ++j) o2[j] = CHANNEL && MODE != 1 ? mul2(bonus, v2[j]) : 0;
+      for (int j = 0; j < kCols; ++j) o2[j] = KIND != PER_HEAD && MODE != 1 ? mul2(bonus, v2[j]) : 0;
 #pragma unroll
       for (int i = 0; i < kRows / 4; ++i) {
         const ulonglong2 kv = k4[i];
-        ulonglong2 qv = make_ulonglong2(0, 0), av = make_ulonglong2(decay2, decay2);
+        ulonglong2 qv = make_ulonglong2(0, 0), av = make_ulonglong2(own_decay, own_decay);
         if (MODE != 1) qv = q4[i];
         if (CHANNEL) av = a4[i];
 #pragma unroll
@@ -485,6 +512,8 @@ linear_attention_kernel(const LinArgs<T> a) {
     for (int j = 0; j < kPer; ++j)
       if (j * 32 + lane < kD) cd[j * 32 + lane] = prod[j];
   }
+  if (TOKEN && MODE == 1 && blockIdx.x == 0 && threadIdx.x == 0)
+    a.chunk_decay[(static_cast<size_t>(seq) * a.max_chunks + c) * a.heads + head] = all_decays;
   float* to = MODE == 1 ? chunk_state : ((MODE == 0 || last_chunk) ? slot_state : nullptr);
   if (to != nullptr) {
 #pragma unroll
@@ -512,18 +541,23 @@ linear_attention_kernel(const LinArgs<T> a) {
 }  // namespace rl
 
 #if RL_LIN_DIM % 16 == 0
+#ifdef RL_LIN_TOKEN
+#include "linear_attention_ssd.cuh"
+#else
 #include "linear_attention_tc.cuh"
+#endif
 #endif
 
 namespace rl {
 
 // Pass 2: chunk_state[seq][c] <- A_c * (state after chunk c - 1) + chunk_state[seq][c], in order of c; A_c is the
-// product of chunk c's decays (every chunk before the last is full).  One thread per element of a head's state.
+// product of chunk c's decays (every chunk before the last is full; `decays` of them per head).  One thread per
+// element of a head's state.
 __global__ void linear_attention_chain_kernel(const int32_t* __restrict__ seq_of_token,
                                               const int32_t* __restrict__ state_slot, const float* __restrict__ decay,
                                               const float* __restrict__ chunk_decay, const float* __restrict__ state,
                                               long long slot_stride, float* __restrict__ chunk_state, int tokens,
-                                              int heads, int dv, int chunk, int max_chunks) {
+                                              int heads, int dv, int chunk, int max_chunks, int decays) {
   pdl_launch();
   pdl_wait();
   const int seq = blockIdx.z, head = blockIdx.y;
@@ -540,7 +574,7 @@ __global__ void linear_attention_chain_kernel(const int32_t* __restrict__ seq_of
   float dpow = 1.f;                                    // decay^chunk by repeated multiplication, as the recurrence applies it
   const float* cd = nullptr;
   if (chunk_decay != nullptr) {
-    cd = chunk_decay + (static_cast<size_t>(seq) * max_chunks * heads + head) * kD + e / dv;
+    cd = chunk_decay + (static_cast<size_t>(seq) * max_chunks * heads + head) * decays + (decays > 1 ? e / dv : 0);
   } else {
     const float dc = decay[head];
     for (int i = 0; i < chunk; ++i) dpow *= dc;
@@ -552,7 +586,7 @@ __global__ void linear_attention_chain_kernel(const int32_t* __restrict__ seq_of
     for (int i = 0; i < kAhead; ++i) {
       const bool in = c0 + i + 1 < chunks;
       own[i] = in ? p[(c0 + i) * step] : 0.f;
-      dec[i] = (in && cd != nullptr) ? cd[static_cast<size_t>(c0 + i) * heads * kD] : dpow;
+      dec[i] = (in && cd != nullptr) ? cd[static_cast<size_t>(c0 + i) * heads * decays] : dpow;
     }
 #pragma unroll
     for (int i = 0; i < kAhead; ++i) {
@@ -597,28 +631,29 @@ inline int lin_threads(int dv) {
   return need >= kMaxThreads ? kMaxThreads : (need + 31) / 32 * 32;
 }
 
-template <typename T, int MODE, bool CHANNEL>
+template <typename T, int MODE, int KIND>
 cudaError_t launch_pass(const LinArgs<T>& a, dim3 grid, int th, cudaStream_t stream) {
   const int cols = th / 32 * kSlots * kCols;
   const bool finish = MODE != 1 && a.y != nullptr;
-  const RawLayout lay = raw_layout(sizeof(T), cols, a.rot_pairs, CHANNEL, MODE != 1, finish && a.gate_mode != GATE_NONE,
+  const RawLayout lay = raw_layout(sizeof(T), cols, a.rot_pairs, KIND == PER_CHANNEL, MODE != 1, finish && a.gate_mode != GATE_NONE,
                                    finish ? a.dv : 0);
   const size_t smem = 2 * static_cast<size_t>(lay.bytes) + lay.pairs + lay.sums;
   static size_t set_for = 0;
   if (smem > set_for) {                  // (the kernel also has static shared memory: beyond 48 KB in all the limit must be raised)
-    const cudaError_t e = cudaFuncSetAttribute(linear_attention_kernel<T, MODE, CHANNEL>,
+    const cudaError_t e = cudaFuncSetAttribute(linear_attention_kernel<T, MODE, KIND>,
                                                cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     if (e != cudaSuccess) return e;
     set_for = smem;
   }
-  return launch_kernel(linear_attention_kernel<T, MODE, CHANNEL>, grid, dim3(th), smem, stream, a);
+  return launch_kernel(linear_attention_kernel<T, MODE, KIND>, grid, dim3(th), smem, stream, a);
 }
 
-#if RL_LIN_DIM % 16 == 0
+#if RL_LIN_DIM % 16 == 0 && !defined(RL_LIN_TOKEN)
 inline int tc_warps(int dv) { return min(kTcMaxWarps, dv / 16); }
 
-template <typename T, int MODE, bool CHANNEL>
+template <typename T, int MODE, int KIND>
 cudaError_t launch_tc_pass(const LinArgs<bf16>& a, dim3 grid, int warps, cudaStream_t stream) {
+  constexpr bool CHANNEL = KIND == PER_CHANNEL;
   const bool finish = MODE != 1 && a.y != nullptr;
   const TcLayout lay = tc_layout(warps * 16, a.rot_pairs, CHANNEL, MODE != 1, finish && a.gate_mode != GATE_NONE, finish);
   static int set_for = 0;
@@ -633,19 +668,23 @@ cudaError_t launch_tc_pass(const LinArgs<bf16>& a, dim3 grid, int warps, cudaStr
 #endif
 
 // One pass of the recurrence in the form that fits: blocks of tokens on the tensor cores, or token by token.
-template <typename T, int MODE, bool CHANNEL>
+template <typename T, int MODE, int KIND>
 cudaError_t launch_either(const LinArgs<T>& a, int rows, int sequences, bool tc, cudaStream_t stream) {
 #if RL_LIN_DIM % 16 == 0
   if constexpr (sizeof(T) == 2) {
     if (tc) {
+#ifdef RL_LIN_TOKEN
+      return launch_ssd_pass<MODE>(a, rows, sequences, stream);
+#else
       const int warps = tc_warps(a.dv);
-      return launch_tc_pass<T, MODE, CHANNEL>(a, dim3((a.dv + warps * 16 - 1) / (warps * 16), rows, sequences), warps, stream);
+      return launch_tc_pass<T, MODE, KIND>(a, dim3((a.dv + warps * 16 - 1) / (warps * 16), rows, sequences), warps, stream);
+#endif
     }
   }
 #endif
   const int th = lin_threads(a.dv);
   const int cols = th / 32 * kSlots * kCols;
-  return launch_pass<T, MODE, CHANNEL>(a, dim3((a.dv + cols - 1) / cols, rows, sequences), th, stream);
+  return launch_pass<T, MODE, KIND>(a, dim3((a.dv + cols - 1) / cols, rows, sequences), th, stream);
 }
 
 template <typename T>
@@ -656,27 +695,27 @@ cudaError_t launch_output(const LinArgs<T>& a, cudaStream_t stream) {
                        a.heads, a.dv, a.eps);
 }
 
-template <typename T, bool CHANNEL>
+template <typename T, int KIND>
 int launch_linear_attention(const LinArgs<T>& a0, int sequences, bool tc, cudaStream_t stream) {
   // finished heads: by the recurrence itself where one CTA has all columns of a head, else by a kernel behind it
   LinArgs<T> a = a0;
   const int th = lin_threads(a.dv);
-  const bool one_block = a.dv <= (tc ? kTcMaxCols : th / 32 * kSlots * kCols);
+  const bool one_block = KIND != PER_TOKEN && a.dv <= (tc ? kTcMaxCols : th / 32 * kSlots * kCols);
   const bool behind = a.y != nullptr && !one_block;
   if (behind) a.y = nullptr;
   cudaError_t e;
   if (a.chunk_state == nullptr || a.max_chunks <= 1) {
-    e = launch_either<T, 0, CHANNEL>(a, a.heads, sequences, tc, stream);
+    e = launch_either<T, 0, KIND>(a, a.heads, sequences, tc, stream);
   } else {
-    e = launch_either<T, 1, CHANNEL>(a, a.heads * a.max_chunks, sequences, tc, stream);
+    e = launch_either<T, 1, KIND>(a, a.heads * a.max_chunks, sequences, tc, stream);
     if (e != cudaSuccess) return static_cast<int>(e);
     const int plane = kD * a.dv;
     e = launch_kernel(linear_attention_chain_kernel, dim3((plane + 255) / 256, a.heads, sequences), dim3(256), 0, stream,
-                      a.seq_of_token, a.state_slot, a.decay, static_cast<const float*>(CHANNEL ? a.chunk_decay : nullptr),
+                      a.seq_of_token, a.state_slot, a.decay, static_cast<const float*>(KIND != PER_HEAD ? a.chunk_decay : nullptr),
                       static_cast<const float*>(a.state), a.slot_stride, a.chunk_state, a.tokens, a.heads, a.dv, a.chunk,
-                      a.max_chunks);
+                      a.max_chunks, KIND == PER_CHANNEL ? kD : 1);
     if (e != cudaSuccess) return static_cast<int>(e);
-    e = launch_either<T, 3, CHANNEL>(a, a.heads * a.max_chunks, sequences, tc, stream);
+    e = launch_either<T, 3, KIND>(a, a.heads * a.max_chunks, sequences, tc, stream);
   }
   if (e == cudaSuccess && behind) e = launch_output(a0, stream);
   return static_cast<int>(e);
@@ -687,6 +726,42 @@ int launch_linear_attention(const LinArgs<T>& a0, int sequences, bool tc, cudaSt
 using namespace rl;
 
 extern "C" {
+
+#ifdef RL_LIN_TOKEN
+
+// The state-space form: q and k of qk_heads heads, z of every token and head in the activation type (row length
+// steps_ld), step_bias, a_log and skip float32 [heads].  out [tokens, heads * DV] float32.  longest, chunk_state, chunk
+// and max_chunks as below; chunk_decay holds [sequences, max_chunks, heads].
+int rl_state_space(int dtype, const void* q, int q_ld, const void* k, int k_ld, int qk_heads, const void* v, int v_ld,
+                   const void* steps, int steps_ld, const float* step_bias, const float* a_log, const float* skip,
+                   const int32_t* seq_of_token, const int32_t* state_slot, float* state, long long slot_stride, float* out,
+                   float* chunk_state, float* chunk_decay, int tokens, int sequences, int heads, int dv, int chunk,
+                   int max_chunks, int longest, cudaStream_t stream) {
+  if (tokens <= 0 || sequences <= 0) return 0;
+  if (out == nullptr || qk_heads <= 0 || heads % qk_heads != 0 || (max_chunks > 1 && chunk_state != nullptr && chunk_decay == nullptr))
+    return static_cast<int>(cudaErrorInvalidValue);
+#define RL_CASE(T)                                                                                                \
+  do {                                                                                                            \
+    LinArgs<T> a = {};                                                                                            \
+    a.q = static_cast<const T*>(q); a.k = static_cast<const T*>(k); a.v = static_cast<const T*>(v);               \
+    a.q_ld = q_ld; a.k_ld = k_ld; a.v_ld = v_ld; a.qk_heads = qk_heads; a.k_scale = 1.f;                          \
+    a.steps = static_cast<const T*>(steps); a.steps_ld = steps_ld; a.step_bias = step_bias; a.a_log = a_log;      \
+    a.skip = skip; a.seq_of_token = seq_of_token; a.state_slot = state_slot; a.state = state;                     \
+    a.slot_stride = slot_stride; a.out = out; a.chunk_state = chunk_state; a.chunk_decay = chunk_decay;           \
+    a.tokens = tokens; a.heads = heads; a.dv = dv; a.chunk = chunk; a.max_chunks = max_chunks;                    \
+    a.quads_ok = dv % 4 == 0 && slot_stride % 4 == 0 && on16(state) && on16(chunk_state);                         \
+    constexpr int E = 16 / sizeof(T);      /* elements of a 16-byte piece */                                      \
+    a.qk_ok = kD % E == 0 && q_ld % E == 0 && k_ld % E == 0 && on16(q) && on16(k);                                \
+    a.v_ok = dv % E == 0 && v_ld % E == 0 && on16(v);                                                             \
+    const bool tc = longest >= kTcMinTokens && sizeof(T) == 2 && kD % 16 == 0 && dv % 16 == 0 && a.qk_ok && a.v_ok; \
+    return launch_linear_attention<T, PER_TOKEN>(a, sequences, tc, stream);                                       \
+  } while (0)
+  if (dtype == 0) RL_CASE(float);
+  else RL_CASE(bf16);
+#undef RL_CASE
+}
+
+#else
 
 // With y the finished heads are asked for, and out [tokens, heads * DV] is scratch that may be used on the way.
 // longest: the most tokens any sequence of the step brings (from kTcMinTokens on, and where sizes allow, bfloat16
@@ -708,7 +783,7 @@ int rl_linear_attention(int dtype, const void* q, int q_ld, const void* k, int k
     return static_cast<int>(cudaErrorInvalidValue);
 #define RL_CASE(T)                                                                                                \
   do {                                                                                                            \
-    LinArgs<T> a;                                                                                                 \
+    LinArgs<T> a = {};                                                                                            \
     a.q = static_cast<const T*>(q); a.k = static_cast<const T*>(k); a.v = static_cast<const T*>(v);               \
     a.q_ld = q_ld; a.k_ld = k_ld; a.v_ld = v_ld; a.k_scale = k_scale; a.cos_t = cos_t; a.sin_t = sin_t;           \
     a.positions = positions; a.rot_pairs = rot_pairs; a.max_pos = max_pos; a.seq_of_token = seq_of_token;         \
@@ -727,12 +802,14 @@ int rl_linear_attention(int dtype, const void* q, int q_ld, const void* k, int k
     const bool tc = longest >= kTcMinTokens && sizeof(T) == 2 && kD % 16 == 0 && dv % 16 == 0 && a.qk_ok &&       \
                     a.v_ok && (a.g_ok || gate_mode == GATE_NONE || y == nullptr) && (a.z_ok || !channel) &&       \
                     (a.rot_ok || rot_pairs == 0);                                                                 \
-    if (channel) return launch_linear_attention<T, true>(a, sequences, tc, stream);                               \
-    return launch_linear_attention<T, false>(a, sequences, tc, stream);                                           \
+    if (channel) return launch_linear_attention<T, PER_CHANNEL>(a, sequences, tc, stream);                        \
+    return launch_linear_attention<T, PER_HEAD>(a, sequences, tc, stream);                                        \
   } while (0)
   if (dtype == 0) RL_CASE(float);
   else RL_CASE(bf16);
 #undef RL_CASE
 }
+
+#endif
 
 }  // extern "C"

@@ -2,7 +2,8 @@
 // bias) fused with the add to the float32 residual stream and with the norm that follows; the norm of the
 // weighted sum of stream and output, for blocks that norm after the sum; bias +
 // activation over a range of columns; the write of any per-token tensor into its paged cache; the
-// gated unit-RMS norm that closes a linear-attention mixer; a gated activation act(gate) * up; and what
+// gated unit-RMS norm that closes a linear-attention mixer, and the one that gates first and norms in parts; a gated
+// activation act(gate) * up; and what
 // attention heads may need between their projection and the cache: an RMS norm of queries and keys
 // (per head or over the whole projection), a rotation of pairs (neighbours, or entry i with entry
 // i + half), a mix of the values with those of an earlier layer.
@@ -15,7 +16,7 @@
 namespace rl {
 
 enum { ACT_NONE = 0, ACT_RELU_SQ = 1, ACT_GELU_ERF = 2, ACT_SILU = 3, ACT_GELU_TANH = 4, ACT_SIGMOID = 5,
-       ACT_CLAMPED_SWISH = 6, ACT_TANH = 7 };
+       ACT_CLAMPED_SWISH = 6, ACT_TANH = 7, ACT_RELU = 8 };
 
 __device__ __forceinline__ float activate(float z, int mode) {
   switch (mode) {
@@ -25,6 +26,7 @@ __device__ __forceinline__ float activate(float z, int mode) {
     case ACT_GELU_TANH: return 0.5f * z * (1.f + tanhf(0.79788456080286536f * (z + 0.044715f * z * z * z)));
     case ACT_SIGMOID: return 1.f / (1.f + expf(-z));
     case ACT_TANH: return tanhf(z);
+    case ACT_RELU: return fmaxf(z, 0.f);
     default: return z;
   }
 }
@@ -432,6 +434,77 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const TA* __re
   }
 }
 
+// ------------------------------------------------ u = o * silu(gate);  out = u / rms(u's part) * w
+// The gate first, then the norm of every one of blockIdx.y = 0 .. groups - 1 equal parts of `size` entries by itself.
+// o is the float32 output of a recurrence [T, groups * size].  A part lives in registers, NV pieces of four neighbouring
+// entries per thread (VEC: parts and rows start on a piece's boundary; else entry by entry).
+template <typename TA, typename TW, int NV, bool VEC>
+__global__ void group_gated_norm_kernel(const float* __restrict__ o, const TA* __restrict__ gate, int ld_gate,
+                                        const TW* __restrict__ w, TA* __restrict__ out, int ld_out, int size, float eps) {
+  __shared__ float scratch[32];
+  const size_t r = blockIdx.x;
+  const int part = blockIdx.y * size;
+  const float* orow = o + r * (static_cast<size_t>(gridDim.y) * size) + part;
+  const TA* g = gate + r * ld_gate + part;
+  TA* y = out + r * ld_out + part;
+  w += part;
+  auto piece = [&](int i) { return (threadIdx.x + i * blockDim.x) * 4; };
+  float wv[NV][4], u[NV][4];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {           // (the weight comes from no earlier kernel of the step)
+    const int c = piece(i);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) wv[i][j] = u[i][j] = 0.f;
+    if (VEC) {
+      if (c < size) load4(w + c, wv[i]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < size) wv[i][j] = to_float(w[c + j]);
+    }
+  }
+  pdl_launch();
+  pdl_wait();
+  float q = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = piece(i);
+    float gv[4] = {0.f, 0.f, 0.f, 0.f};
+    if (VEC) {
+      if (c < size) {
+        load4(orow + c, u[i]);
+        load4(g + c, gv);
+      }
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < size) {
+          u[i][j] = orow[c + j];
+          gv[j] = to_float(g[c + j]);
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      u[i][j] *= gv[j] / (1.f + expf(-gv[j]));
+      q = fmaf(u[i][j], u[i][j], q);
+    }
+  }
+  const float rstd = rsqrtf(block_sum(q, scratch) / static_cast<float>(size) + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = piece(i);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) u[i][j] *= rstd * wv[i][j];
+    if (VEC) {
+      if (c < size) store4(y + c, u[i]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c + j < size) y[c + j] = from_float<TA>(u[i][j]);
+    }
+  }
+}
+
 // ------------------------------------------------ out[r, i] = act(gu[r, i]) * gu[r, inter + i]
 // mode ACT_CLAMPED_SWISH: g = min(gate, limit), u = clamp(up, -limit, limit), out = g sigmoid(slope g) (u + 1).
 template <typename TA>
@@ -468,6 +541,8 @@ __global__ void gated_act_kernel(const TA* __restrict__ gu, int ld, TA* __restri
 // With `slots` the finished keys and values also go to their paged caches ([pages, k_heads, page_size, dim]
 // and [pages, v_heads, page_size, v_size / v_heads]) at slots[t] = page * page_size + offset (negative: no
 // write; beyond the pool: not written, bit 2 of *status).
+// `bias` (float32 over queries, keys and values, which then lie one after another from q_col on) is added first:
+// what the norms see is the biased projection as it would be stored.
 // Two neighbouring entries as one access (the address is a multiple of the pair's size).
 __device__ __forceinline__ void load2(const float* p, float& a, float& b) {
   const float2 v = *reinterpret_cast<const float2*>(p);
@@ -484,6 +559,12 @@ __device__ __forceinline__ void store2(bf16* p, float a, float b) {
   *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
 }
 
+// An entry with its bias, rounded as it would be stored.
+template <typename TA>
+__device__ __forceinline__ float biased(TA x, const float* bias, int i) {
+  return bias != nullptr ? to_float(from_float<TA>(to_float(x) + bias[i])) : to_float(x);
+}
+
 struct HeadPrepArgs {
   int ld, q_col, q_heads, k_col, k_heads, dim, norm_mode;
   float eps;
@@ -494,6 +575,7 @@ struct HeadPrepArgs {
   long long num_slots;
   int pairs_ok;       // every head starts on a pair's boundary in the buffer, the weights and the caches
   int rot_half;       // 1: entry i < rot_pairs is paired with entry i + rot_pairs instead of its neighbour
+  const float* bias;  // or null
 };
 
 template <typename TA, typename TW>
@@ -523,9 +605,10 @@ __global__ void head_prep_kernel(TA* __restrict__ x, const int32_t* __restrict__
   if (a.norm_mode != 0) {
     for (int h = warp; h < all_heads; h += nwarps) {
       const TA* p = h < a.q_heads ? row + a.q_col + h * a.dim : row + a.k_col + (h - a.q_heads) * a.dim;
+      const float* bp = a.bias != nullptr ? a.bias + h * a.dim : nullptr;
       float q = 0.f;
       for (int d = lane; d < a.dim; d += 32) {
-        const float v = to_float(p[d]);
+        const float v = biased(p[d], bp, d);
         q += v * v;
       }
       q = warp_sum(q);
@@ -538,6 +621,7 @@ __global__ void head_prep_kernel(TA* __restrict__ x, const int32_t* __restrict__
     const int h0 = sec == 0 ? 0 : a.q_heads;
     TA* p = row + (sec == 0 ? a.q_col : a.k_col);
     const TW* w = sec == 0 ? q_w : k_w;
+    const float* bp = a.bias != nullptr ? a.bias + h0 * a.dim : nullptr;
     float whole = 1.f;
     if (a.norm_mode == 2) {        // every thread adds the section's heads in the same order
       float q = 0.f;
@@ -553,6 +637,10 @@ __global__ void head_prep_kernel(TA* __restrict__ x, const int32_t* __restrict__
                         : (a.norm_mode == 1 ? rsqrtf(head_sq[h0 + h] / static_cast<float>(a.dim) + a.eps) : 1.f);
         float u, v;
         load2(p + i, u, v);
+        if (bp != nullptr) {
+          u = to_float(from_float<TA>(u + bp[i]));
+          v = to_float(from_float<TA>(v + bp[i + 1]));
+        }
         if (a.norm_mode != 0) {
           float wu, wv;
           load2(w + (a.norm_mode == 2 ? i : d), wu, wv);
@@ -565,7 +653,7 @@ __global__ void head_prep_kernel(TA* __restrict__ x, const int32_t* __restrict__
           const float ru = u * cs - v * sn, rv = v * cs + u * sn;
           u = ru;
           v = rv;
-        } else if (a.norm_mode == 0 && kc == nullptr) {
+        } else if (a.norm_mode == 0 && kc == nullptr && bp == nullptr) {
           continue;                  // nothing changes and nothing is cached
         }
         store2(p + i, u, v);
@@ -586,16 +674,16 @@ __global__ void head_prep_kernel(TA* __restrict__ x, const int32_t* __restrict__
       const float r = a.norm_mode == 2 ? whole
                       : (a.norm_mode == 1 ? rsqrtf(head_sq[h0 + h] / static_cast<float>(a.dim) + a.eps) : 1.f);
       const int wi = a.norm_mode == 2 ? i : d;
-      float u = to_float(p[i]) * r;
+      float u = biased(p[i], bp, i) * r;
       if (a.norm_mode != 0) u *= to_float(w[wi]);
       TA* c = kc != nullptr ? kc + ((page * heads + h) * a.page_size + off) * a.dim + d : nullptr;
       if (!paired) {
         const TA o = from_float<TA>(u);
-        if (a.norm_mode != 0) p[i] = o;
+        if (a.norm_mode != 0 || bp != nullptr) p[i] = o;
         if (c != nullptr) c[0] = o;
         continue;
       }
-      float v = to_float(p[i + other]) * r;
+      float v = biased(p[i + other], bp, i + other) * r;
       if (a.norm_mode != 0) v *= to_float(w[wi + other]);
       const float cs = cos_t[static_cast<size_t>(pos) * a.rot_pairs + pair];
       const float sn = sin_t[static_cast<size_t>(pos) * a.rot_pairs + pair];
@@ -609,11 +697,16 @@ __global__ void head_prep_kernel(TA* __restrict__ x, const int32_t* __restrict__
     }
   }
   if (a.vmix_mode != 0 || slot >= 0) {
+    const float* bp = a.bias != nullptr ? a.bias + all_heads * a.dim : nullptr;
     TA* v = row + a.v_col;
     TA* f = v_first != nullptr ? v_first + static_cast<size_t>(t) * a.v_size : nullptr;
     const int vdim = a.v_size / max(a.v_heads, 1);
     for (int i = threadIdx.x; i < a.v_size; i += blockDim.x) {
       TA o = v[i];
+      if (bp != nullptr) {
+        o = from_float<TA>(to_float(o) + bp[i]);
+        if (a.vmix_mode != 2) v[i] = o;
+      }
       if (a.vmix_mode == 1) f[i] = o;
       else if (a.vmix_mode == 2) {
         o = from_float<TA>((1.f - a.lam) * to_float(o) + a.lam * to_float(f[i]));
@@ -764,6 +857,42 @@ int rl_gated_rmsnorm(const float* o, const void* gate, int ld_gate, const void* 
   RL_LAUNCH_END();
 }
 
+// Parts of up to 16 x 1,024 entries (cudaErrorInvalidValue beyond).
+int rl_group_gated_norm(const float* o, const void* gate, int ld_gate, const void* w, int w_dtype, void* out, int ld_out,
+                        int act_dtype, int rows, int n, int groups, float eps, cudaStream_t stream) {
+  if (rows <= 0 || n <= 0) return 0;
+  const int size = n / groups, pieces = (size + 3) / 4;
+  if (groups <= 0 || n % groups != 0 || pieces > 4096) return static_cast<int>(cudaErrorInvalidValue);
+  const int nv = pieces <= 256 ? 1 : (pieces <= 1024 ? 2 : 4);
+  const int th = max(32, ((pieces + nv - 1) / nv + 31) / 32 * 32);
+  const size_t act = act_dtype == RL_F32 ? 16 : 8, wb = (act_dtype == RL_F32 || w_dtype == RL_F32) ? 16 : 8;
+  const bool vec = size % 4 == 0 && ld_gate % 4 == 0 && ld_out % 4 == 0 && reinterpret_cast<uintptr_t>(o) % 16 == 0 &&
+                   reinterpret_cast<uintptr_t>(w) % wb == 0 && reinterpret_cast<uintptr_t>(gate) % act == 0 &&
+                   reinterpret_cast<uintptr_t>(out) % act == 0;
+  const dim3 grid(rows, groups);
+#define RL_CASE(TA, TW, NV)                                                                                         \
+  do {                                                                                                              \
+    if (vec) launch_kernel(group_gated_norm_kernel<TA, TW, NV, true>, grid, dim3(th), 0, stream, o,                 \
+                           static_cast<const TA*>(gate), ld_gate, static_cast<const TW*>(w), static_cast<TA*>(out), \
+                           ld_out, size, eps);                                                                      \
+    else launch_kernel(group_gated_norm_kernel<TA, TW, NV, false>, grid, dim3(th), 0, stream, o,                    \
+                       static_cast<const TA*>(gate), ld_gate, static_cast<const TW*>(w), static_cast<TA*>(out),     \
+                       ld_out, size, eps);                                                                          \
+  } while (0)
+#define RL_SIZES(TA, TW)                        \
+  do {                                          \
+    if (nv == 1) RL_CASE(TA, TW, 1);            \
+    else if (nv == 2) RL_CASE(TA, TW, 2);       \
+    else RL_CASE(TA, TW, 4);                    \
+  } while (0)
+  if (act_dtype == RL_F32) RL_SIZES(float, float);
+  else if (w_dtype == RL_F32) RL_SIZES(bf16, float);
+  else RL_SIZES(bf16, bf16);
+#undef RL_SIZES
+#undef RL_CASE
+  RL_LAUNCH_END();
+}
+
 int rl_gated_act(const void* gu, int ld, void* out, int act_dtype, int rows, int inter, int mode, float limit,
                  float slope, const float* bias, cudaStream_t stream) {
   if (rows <= 0 || inter <= 0) return 0;
@@ -783,10 +912,11 @@ int rl_head_prep(void* x, int act_dtype, int ld, const int32_t* positions, int t
                  float eps, const float* cos_t, const float* sin_t, int rot_pairs, int max_pos, int v_col,
                  int v_size, void* v_first, int vmix_mode, float lam, const int32_t* slots, void* k_cache,
                  void* v_cache, int v_heads, int page_size, long long num_slots, int* status, int rot_half,
-                 cudaStream_t stream) {
+                 const float* bias, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   HeadPrepArgs a;
   a.rot_half = rot_half;
+  a.bias = bias;
   a.ld = ld; a.q_col = q_col; a.q_heads = q_heads; a.k_col = k_col; a.k_heads = k_heads; a.dim = dim;
   a.norm_mode = norm_mode; a.eps = eps; a.rot_pairs = rot_pairs; a.max_pos = max_pos; a.v_col = v_col;
   a.v_size = v_size; a.vmix_mode = vmix_mode; a.lam = lam;

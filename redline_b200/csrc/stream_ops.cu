@@ -12,7 +12,8 @@
 // pair_norm_mean_kernel, one CTA per token: out = ca * N(a + bias_a, wa) + cb * N(b + bias_b, wb), N the RMS
 // norm, the biases (float32, of the two products that made a and b) optional.
 //
-// short_conv_kernel, one thread per channel and token (eight tokens in a large step): y_t = act(sum_j w[c, j] (u_(t - taps + 1 + j) + bias_c)),
+// short_conv_kernel, one thread per channel and token (eight tokens in a large step):
+// y_t = act(sum_j w[c, j] (u_(t - taps + 1 + j) + bias_c) + out_bias_c),
 // over the tokens of the token's own sequence; tokens before the step's portion come from the request's state
 // slot, which holds the last taps - 1 inputs (bias added) in float32: [taps - 1, channels], the oldest first,
 // zeros for a new request.  short_conv_state_kernel then moves the slot on: the thread of a sequence's last
@@ -149,7 +150,8 @@ struct ConvArgs {
   int ld_x, col_x, ld_y, col_y, channels, taps, act, tokens;
   int tile;                      // consecutive tokens a thread of short_conv_kernel walks
   int own_state;                 // every sequence has one token in this step: the thread of the token moves the slot on itself
-  const float* bias;             // [channels] or null
+  const float* bias;             // [channels] or null: of the inputs
+  const float* out_bias;         // [channels] or null: of the sums
   const int32_t* seq_of_token;
   const int32_t* state_slot;
   float* state;                  // [slots] x [taps - 1, channels]
@@ -186,7 +188,7 @@ __global__ void short_conv_kernel(const ConvArgs a, const TA* __restrict__ x, co
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= a.channels) return;
   const int t_begin = blockIdx.y * a.tile, t_end = min(t_begin + a.tile, a.tokens);
-  const float bias = a.bias != nullptr ? a.bias[c] : 0.f;
+  const float bias = a.bias != nullptr ? a.bias[c] : 0.f, out_bias = a.out_bias != nullptr ? a.out_bias[c] : 0.f;
   const int keep = a.taps - 1;
   float wt[kMaxTaps], win[kMaxTaps];     // win[j]: the input j + 1 tokens back, wt[j] its weight
 #pragma unroll
@@ -211,7 +213,7 @@ __global__ void short_conv_kernel(const ConvArgs a, const TA* __restrict__ x, co
 #pragma unroll
     for (int j = kMaxTaps - 1; j >= 0; --j)                  // the oldest input first, as a sum over the taps in order
       if (j < keep) acc = fmaf(wt[j], win[j], acc);
-    acc = fmaf(w_now, u, acc);
+    acc = fmaf(w_now, u, acc) + out_bias;
 #pragma unroll
     for (int j = kMaxTaps - 1; j > 0; --j) win[j] = win[j - 1];
     win[0] = u;
@@ -381,14 +383,14 @@ int rl_pair_norm_mean(int act_dtype, const void* a, int ld_a, const void* wa, fl
 }
 
 int rl_short_conv(int act_dtype, const void* x, int ld_x, int col_x, const void* w, int w_dtype, const float* bias,
-                  void* y, int ld_y, int col_y, int channels, int taps, int act, const int32_t* seq_of_token,
+                  const float* out_bias, void* y, int ld_y, int col_y, int channels, int taps, int act, const int32_t* seq_of_token,
                   const int32_t* state_slot, float* state, long long slot_stride, int tokens, int single,
                   cudaStream_t stream) {
   if (tokens <= 0 || channels <= 0) return 0;
   if (taps < 1 || taps > kMaxTaps) return static_cast<int>(cudaErrorInvalidValue);
   ConvArgs a;
   a.ld_x = ld_x; a.col_x = col_x; a.ld_y = ld_y; a.col_y = col_y; a.channels = channels; a.taps = taps; a.act = act;
-  a.tokens = tokens; a.bias = bias; a.seq_of_token = seq_of_token; a.state_slot = state_slot; a.state = state;
+  a.tokens = tokens; a.bias = bias; a.out_bias = out_bias; a.seq_of_token = seq_of_token; a.state_slot = state_slot; a.state = state;
   a.slot_stride = slot_stride;
   a.own_state = (single && taps > 1) ? 1 : 0;
   const int th = 128;

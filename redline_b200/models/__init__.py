@@ -1,3 +1,3 @@
 """Built-in architectures; importing this package registers them."""
 
-from . import kapitar, lakatar, llama, pufevik, venezen, vizotar  # noqa: F401
+from . import kapitar, lakatar, llama, pufevik, venezen, vizotar, vogolix  # noqa: F401

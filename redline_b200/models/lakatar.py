@@ -65,7 +65,7 @@ def lakatar_spec(c: LakatarConfig) -> ModelSpec:
                 names.update({"dkv": p + "mix.dkv", "dkv_norm": p + "mix.dkv.norm"})
             mixer = PartSpec("latent_attention", LatentAttentionParams(
                 hidden_size=W, num_heads=m.heads, dim=m.dim, rot_dim=m.rot_dim, vdim=m.vdim, kv_rank=m.kv_rank,
-                scale=m.scale, eps=c.norm_eps, q_rank=m.q_rank, gated=True, own_latent=own,
+                scale=m.scale, eps=c.norm_eps, q_rank=m.q_rank, gate="head", own_latent=own,
                 position=_rotation("rope_pairs", RotaryPairsParams, m.rot, c.max_position_embeddings)
                 if m.rot_dim > 0 else None), names)
         f = layer.mlp

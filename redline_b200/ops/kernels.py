@@ -173,7 +173,8 @@ def gemm_tn_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, rows: Opti
 SKINNY_MAX_ROWS = 16
 SKINNY_UNSTAGED_ROWS = 8    # up to here bfloat16 activations are read from global memory, not staged
 EPI_BF16, EPI_F32, EPI_ADD_RESIDUAL, EPI_SWIGLU = 0, 1, 2, 3
-EPI_GEGLU_TANH = 4     # gemm_tc and gemm_skinny: as EPI_SWIGLU with the tanh form of GELU on the gate
+EPI_GEGLU_TANH, EPI_REGLU = 4, 5     # gemm_tc and gemm_skinny: as EPI_SWIGLU with the tanh form of GELU, or a ReLU, on the gate
+EPI_GATED = (EPI_SWIGLU, EPI_GEGLU_TANH, EPI_REGLU)
 _sm_count: Dict[int, int] = {}
 
 
@@ -207,8 +208,8 @@ def gemm_skinny(w: torch.Tensor, y: torch.Tensor, epilogue: int, rows: int, x: O
     x given: bfloat16 activations [rows, K].  residual + norm_w given instead: x is
     bfloat16(rmsnorm(residual[rows_idx]) * norm_w) formed inside the kernel.
     epilogue EPI_BF16 / EPI_F32: store into y; EPI_ADD_RESIDUAL: y (float32 stream) += product;
-    EPI_SWIGLU: w is [2 N, K] (gate rows, then up rows), y = silu(gate) * up, [rows, N]; EPI_GEGLU_TANH: the
-    same with the tanh form of GELU on the gate.
+    EPI_SWIGLU: w is [2 N, K] (gate rows, then up rows), y = silu(gate) * up, [rows, N]; EPI_GEGLU_TANH and
+    EPI_REGLU: the same with the tanh form of GELU, or a ReLU, on the gate.
 
     The RMSNorm between a product that ends in ``residual +=`` and the product after it can be handed
     over instead of run as a kernel: with ``hand_out = (next_norm_weight, xw, sums)`` (EPI_ADD_RESIDUAL)
@@ -222,7 +223,7 @@ def gemm_skinny(w: torch.Tensor, y: torch.Tensor, epilogue: int, rows: int, x: O
              c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
              c_void_p])
     K = w.shape[1]
-    N = w.shape[0] // 2 if epilogue in (EPI_SWIGLU, EPI_GEGLU_TANH) else w.shape[0]
+    N = w.shape[0] // 2 if epilogue in EPI_GATED else w.shape[0]
     norm = residual is not None
     if norm:
         if norm_w is None or residual.dtype != torch.float32 or residual.shape[1] != K or residual.stride(0) != K:
@@ -233,7 +234,7 @@ def gemm_skinny(w: torch.Tensor, y: torch.Tensor, epilogue: int, rows: int, x: O
             raise KernelError("gemm_skinny: x must be bfloat16 [rows, K]")
         ldx = x.stride(0)
     want = {EPI_BF16: torch.bfloat16, EPI_F32: torch.float32, EPI_ADD_RESIDUAL: torch.float32,
-            EPI_SWIGLU: torch.bfloat16, EPI_GEGLU_TANH: torch.bfloat16}[epilogue]
+            EPI_SWIGLU: torch.bfloat16, EPI_GEGLU_TANH: torch.bfloat16, EPI_REGLU: torch.bfloat16}[epilogue]
     if y.dtype != want or y.shape[1] != N or y.stride(1) != 1:
         raise KernelError(f"gemm_skinny: output must be {want} [rows, {N}]")
     next_w = xw = ss_out = None
@@ -305,17 +306,17 @@ def gemm_tc_ok(x: torch.Tensor, w: torch.Tensor) -> bool:
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, epilogue: int = EPI_BF16, tile_n: int = 0) -> None:
     """y = epilogue(x @ w^T) with tcgen05 tensor cores, TMEM accumulators and TMA loads
-    (csrc/gemm_tc.cu): bfloat16 x [M, K], w [N, K] (EPI_SWIGLU and EPI_GEGLU_TANH: [2 N, K], gate rows then
-    up rows).
+    (csrc/gemm_tc.cu): bfloat16 x [M, K], w [N, K] (EPI_SWIGLU, EPI_GEGLU_TANH and EPI_REGLU: [2 N, K],
+    gate rows then up rows).
     Epilogues as gemm_skinny's.  tile_n: 0 lets the kernel choose its tiling; 128 or 256 force one CTA per
     128-row tile of that width, 512 forces CTA pairs (tcgen05.mma.cta_group::2) on 256 x 256 tiles."""
     _need_cuda(x, w, y)
     f = _fn(_lib("gemm_tc", "gemm_tc.cu"), "rl_gemm_tc",
             [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p])
     M, K = x.shape
-    N = w.shape[0] // 2 if epilogue in (EPI_SWIGLU, EPI_GEGLU_TANH) else w.shape[0]
+    N = w.shape[0] // 2 if epilogue in EPI_GATED else w.shape[0]
     want = {EPI_BF16: torch.bfloat16, EPI_F32: torch.float32, EPI_ADD_RESIDUAL: torch.float32,
-            EPI_SWIGLU: torch.bfloat16, EPI_GEGLU_TANH: torch.bfloat16}[epilogue]
+            EPI_SWIGLU: torch.bfloat16, EPI_GEGLU_TANH: torch.bfloat16, EPI_REGLU: torch.bfloat16}[epilogue]
     if w.shape[1] != K or y.dtype != want or y.shape[1] != N or y.stride(1) != 1 or not gemm_tc_ok(x, w):
         raise KernelError(f"gemm_tc: shapes x{tuple(x.shape)} w{tuple(w.shape)} y{tuple(y.shape)} {y.dtype}")
     _check(f(_ptr(x), x.stride(0), _ptr(w), _ptr(y), y.stride(0), epilogue, M, N, K, _ptr(tc_status(x.device)),
@@ -595,8 +596,9 @@ def attn_prefill(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcache: t
 ACT_NONE, ACT_RELU_SQ, ACT_GELU_ERF, ACT_SILU, ACT_GELU_TANH, ACT_SIGMOID = 0, 1, 2, 3, 4, 5
 ACT_CLAMPED_SWISH = 6      # gated_act only: min / clamp of gate and up, g * sigmoid(slope * g) * (up + 1)
 ACT_TANH = 7               # act_cast and bias_act
+ACT_RELU = 8
 ACTIVATIONS = {"none": ACT_NONE, "relu_squared": ACT_RELU_SQ, "gelu": ACT_GELU_ERF, "silu": ACT_SILU,
-               "gelu_tanh": ACT_GELU_TANH}
+               "gelu_tanh": ACT_GELU_TANH, "relu": ACT_RELU}
 NORM_LAYER, NORM_RMS = 0, 1
 
 
@@ -737,6 +739,23 @@ def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, out
              rows if rows is not None else o.shape[0], o.shape[1], float(eps), _stream()), "gated_rmsnorm")
 
 
+def group_gated_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, groups: int, eps: float,
+                     rows: Optional[int] = None) -> None:
+    """u = o * silu(gate), then every one of ``groups`` equal parts of a row divided by its own root mean square, times
+    ``weight``: out = u / sqrt(mean over the part (u^2) + eps) * weight.  o float32 [T, n] contiguous, gate and out
+    (row-strided) views [T, n] of the activation type."""
+    _need_cuda(o, gate, weight, out)
+    n = o.shape[1]
+    if o.dtype != torch.float32 or not o.is_contiguous() or gate.stride(1) != 1 or out.stride(1) != 1 \
+            or gate.dtype != out.dtype or gate.shape[1] != n or out.shape[1] != n or weight.numel() != n \
+            or groups <= 0 or n % groups != 0:
+        raise KernelError("group_gated_norm: o float32 contiguous, gate and out of the activation type, equal parts")
+    f = _fn(_rw(), "rl_group_gated_norm", [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int,
+                                            c_int, c_float, c_void_p])
+    _check(f(_ptr(o), _ptr(gate), gate.stride(0), _ptr(weight), _code(weight.dtype), _ptr(out), out.stride(0),
+             _code(out.dtype), rows if rows is not None else o.shape[0], n, groups, float(eps), _stream()), "group_gated_norm")
+
+
 def gated_act(gate_up: torch.Tensor, out: torch.Tensor, act: int, limit: float = 0.0, slope: float = 1.0,
               bias: Optional[torch.Tensor] = None) -> None:
     """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i], I = out.shape[1].  ``ACT_CLAMPED_SWISH``: with
@@ -764,21 +783,30 @@ def head_prep(x: torch.Tensor, positions: torch.Tensor, tokens: int, q_col: int,
               cos: Optional[torch.Tensor] = None, sin: Optional[torch.Tensor] = None, v_col: int = 0, v_size: int = 0,
               v_first: Optional[torch.Tensor] = None, mix_mode: int = VALUE_MIX_NONE, lam: float = 0.0,
               slots: Optional[torch.Tensor] = None, k_cache: Optional[torch.Tensor] = None,
-              v_cache: Optional[torch.Tensor] = None, page_size: int = 0, halves: bool = False) -> None:
+              v_cache: Optional[torch.Tensor] = None, page_size: int = 0, halves: bool = False,
+              bias: Optional[torch.Tensor] = None) -> None:
     """In place on the rows of a projection buffer (csrc/rowwise.cu: head_prep_kernel): the query heads at
     ``q_col`` and the key heads at ``k_col`` are RMS-normed (per head with weights [dim], or over the whole
     section with weights [heads * dim]) and their first 2 * cos.shape[1] entries rotated in neighbouring
     pairs (``halves``: entry i paired with entry i + cos.shape[1]) by the tables' angles at each token's position; the values at ``v_col`` are kept in ``v_first``
     [tokens, v_size] or blended with it, v <- (1 - lam) v + lam v_first.  All in float32.  With ``slots`` the
     finished keys and values are also written to their paged caches ([pages, k_heads, page_size, dim] and
-    [pages, v_heads, page_size, vdim]; a slot beyond the pool is not written and sets bit 2 of ``status``)."""
-    _need_cuda(x, positions, q_weight, k_weight, cos, sin, v_first)
+    [pages, v_heads, page_size, vdim]; a slot beyond the pool is not written and sets bit 2 of ``status``).
+    ``k_heads`` 0: queries only (no keys, no values).  ``bias`` (float32, from column ``q_col`` on over the queries, the
+    keys and the values, which then lie one after another) is added first."""
+    _need_cuda(x, positions, q_weight, k_weight, cos, sin, v_first, bias)
+    if k_heads == 0 and (slots is not None or mix_mode != VALUE_MIX_NONE):
+        raise KernelError("head_prep: without keys there is nothing to cache or to blend")
+    if bias is not None and (bias.dtype != torch.float32 or not bias.is_contiguous()
+                             or (k_heads > 0 and (k_col != q_col + q_heads * dim or v_col != k_col + k_heads * dim))
+                             or bias.numel() != (q_heads + k_heads) * dim + (v_size if k_heads > 0 else 0)):
+        raise KernelError("head_prep: a bias is contiguous float32 over neighbouring queries, keys and values")
     if x.stride(1) != 1:
         raise KernelError("head_prep: rows must be contiguous")
     if norm_mode != HEAD_NORM_NONE:
         want = (dim, dim) if norm_mode == HEAD_NORM_EACH else (q_heads * dim, k_heads * dim)
-        if q_weight is None or k_weight is None or (q_weight.numel(), k_weight.numel()) != want \
-                or q_weight.dtype != k_weight.dtype:
+        if q_weight is None or q_weight.numel() != want[0] or (k_heads > 0 and (
+                k_weight is None or k_weight.numel() != want[1] or q_weight.dtype != k_weight.dtype)):
             raise KernelError(f"head_prep: norm weights of {want} entries and one type")
     pairs = 0
     if cos is not None:
@@ -800,12 +828,12 @@ def head_prep(x: torch.Tensor, positions: torch.Tensor, tokens: int, q_col: int,
     f = _fn(_rw(), "rl_head_prep", [c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                                      c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_int,
                                      c_int, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_int,
-                                     c_int, c_longlong, c_void_p, c_int, c_void_p])
+                                     c_int, c_longlong, c_void_p, c_int, c_void_p, c_void_p])
     _check(f(_ptr(x), _code(x.dtype), x.stride(0), _ptr(positions), tokens, q_col, q_heads, k_col, k_heads, dim,
              _ptr(q_weight), _ptr(k_weight), _code(q_weight.dtype) if q_weight is not None else 0, norm_mode,
              float(eps), _ptr(cos), _ptr(sin), pairs, cos.shape[0] if cos is not None else 0, v_col, v_size,
              _ptr(v_first), mix_mode, float(lam), _ptr(slots), _ptr(k_cache), _ptr(v_cache), v_heads, page_size,
-             num_slots, _ptr(status), 1 if halves else 0, _stream()), "head_prep")
+             num_slots, _ptr(status), 1 if halves else 0, _ptr(bias), _stream()), "head_prep")
 
 
 # ------------------------------------ attention with score maps, a capped score and kept first tokens
@@ -834,7 +862,7 @@ def maps_attn_decode(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcach
                      maps: int, page_size: int, window: int, keep_first: int, scale: float, softcap: float,
                      lam: float, post_scale: float, eps: float, unit_norm: bool,
                      sink: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                     gate_mode: int = 0, slopes: Optional[torch.Tensor] = None, v_stride: int = 0) -> None:
+                     gate_mode: int = 0, slopes: Optional[torch.Tensor] = None, v_stride: int = 0, chunk: int = 0) -> None:
     """One query token per item (``items`` as for ``attn_decode``) over the paged cache, ``maps`` score maps
     per head over shared values (csrc/attention_maps.cu): q rows (head, map) of ``dim``, key cache
     [pages, kv_heads * maps, page, dim], value cache [pages, kv_heads, page, vdim], out heads of ``vdim``.
@@ -842,12 +870,15 @@ def maps_attn_decode(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcach
     view of q's type) multiplies the output by its sigmoid, per head (``gate_mode`` 1, [tokens, heads]) or
     per entry (2, [tokens, heads * vdim]); ``post_scale`` multiplies the output too.  ``slopes`` (float32
     [heads]): slope_h times the distance between query and key is taken off every score of head h.
-    ``v_stride``: see ``_maps``."""
+    ``v_stride``: see ``_maps``.  ``chunk`` > 0 (without a window): a position sees the keys of its own chunk of so many
+    positions only."""
     _need_cuda(q, kcache, vcache, out, sink, gate, slopes)
     _check_tail(maps, heads, vdim, q, sink, gate, gate_mode, slopes)
+    if chunk < 0 or (chunk > 0 and (window > 0 or keep_first > 0)):
+        raise KernelError("attention_maps: chunks go without a window and kept first tokens")
     f = _fn(_maps(dim, vdim, maps, v_stride), "rl_maps_decode",
             [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
-             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_float, c_int,
+             c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float, c_float, c_int,
              c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p])
     need = nitems * heads * maps * max_parts
     if part_o.numel() < need * vdim or part_ml.numel() < need * 2:
@@ -856,7 +887,7 @@ def maps_attn_decode(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcach
         raise KernelError("maps_attn_decode: items must be 16-byte aligned")
     _check(f(_code(q.dtype), _ptr(q), q_stride, _ptr(kcache), _ptr(vcache), _ptr(block_table), block_table.shape[1],
              _ptr(items), _ptr(part_o), _ptr(part_ml), max_parts, _ptr(out), out.stride(0), nitems, heads, kv_heads,
-             page_size, window, keep_first, float(scale), float(softcap), float(lam), float(post_scale), float(eps),
+             page_size, window, keep_first, chunk, float(scale), float(softcap), float(lam), float(post_scale), float(eps),
              1 if unit_norm else 0, _ptr(sink), _ptr(slopes), _ptr(gate), gate.stride(0) if gate is not None else 0,
              gate_mode if gate is not None else 0, _stream()), "maps_attn_decode", 2)
 
@@ -880,19 +911,21 @@ def maps_attn_prefill(q: torch.Tensor, q_stride: int, kcache: torch.Tensor, vcac
                       window: int, keep_first: int, scale: float, softcap: float, lam: float, post_scale: float,
                       eps: float, unit_norm: bool, sink: Optional[torch.Tensor] = None,
                       gate: Optional[torch.Tensor] = None, gate_mode: int = 0, impl: int = 0,
-                      slopes: Optional[torch.Tensor] = None, v_stride: int = 0) -> None:
+                      slopes: Optional[torch.Tensor] = None, v_stride: int = 0, chunk: int = 0) -> None:
     """Tiles of up to ``tile_rows_max`` consecutive query tokens of one sequence; otherwise as
     ``maps_attn_decode``.  impl 0: the best kernel that applies (bfloat16 with sizes that are multiples of
     16: mma.sync tensor cores; else CUDA cores); 1: CUDA cores; 2: the tensor-core kernel or an error."""
     _need_cuda(q, kcache, vcache, out, sink, gate, slopes)
     _check_tail(maps, heads, vdim, q, sink, gate, gate_mode, slopes)
+    if chunk < 0 or (chunk > 0 and (window > 0 or keep_first > 0)):
+        raise KernelError("attention_maps: chunks go without a window and kept first tokens")
     f = _fn(_maps(dim, vdim, maps, v_stride), "rl_maps_prefill",
             [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
-             c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float,
+             c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_float,
              c_float, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p])
     _check(f(_code(q.dtype), _ptr(q), q_stride, _ptr(kcache), _ptr(vcache), _ptr(block_table), block_table.shape[1],
              _ptr(tile_seq), _ptr(tile_tok), _ptr(tile_rows), _ptr(positions), _ptr(out), out.stride(0), tiles,
-             tile_rows_max, heads, kv_heads, page_size, window, keep_first, float(scale), float(softcap), float(lam),
+             tile_rows_max, heads, kv_heads, page_size, window, keep_first, chunk, float(scale), float(softcap), float(lam),
              float(post_scale), float(eps), 1 if unit_norm else 0, _ptr(sink), _ptr(slopes), _ptr(gate),
              gate.stride(0) if gate is not None else 0, gate_mode if gate is not None else 0, impl, _stream()),
            "maps_attn_prefill")
@@ -952,20 +985,23 @@ def latent_prep(q: Optional[torch.Tensor], latent: Optional[torch.Tensor], posit
 
 
 def head_linear(x: torch.Tensor, x_col: int, x_head: int, w: torch.Tensor, y: torch.Tensor, y_col: int, y_head: int,
-                tokens: Optional[int] = None, impl: int = 0, turn: Optional[Tuple] = None) -> None:
+                tokens: Optional[int] = None, impl: int = 0, turn: Optional[Tuple] = None,
+                gate: Optional[torch.Tensor] = None) -> None:
     """y[t, y_col + h * y_head + j] = sum_k w[h, j, k] * x[t, x_col + h * x_head + k] for every head h:
     w [heads, n, k]; float32 sums.  impl 0: a kernel for at most 16 tokens, tensor cores or CUDA cores, whichever
     fits; 1: CUDA cores; 2: tensor cores where they apply.
     ``turn`` = (entries, first of them in x's head, in y's head, cos, sin, positions, pairs, status): that part of
     every head's row of x goes to y's turned by the token's position, the first 2 * cos.shape[1] entries as in
-    ``latent_prep``."""
-    _need_cuda(x, w, y)
+    ``latent_prep``.  ``gate`` [tokens, heads * n] (a row-strided view of x's type): every output times its sigmoid."""
+    _need_cuda(x, w, y, gate)
     heads, n, k = w.shape
     if x.dtype != y.dtype or x.stride(1) != 1 or y.stride(1) != 1 or not w.is_contiguous() \
             or (x.dtype == torch.float32 and w.dtype != torch.float32):
         raise KernelError("head_linear: x and y have one type and contiguous rows; w contiguous [heads, n, k]")
     if x_col + (heads - 1) * x_head + k > x.shape[1] or y_col + (heads - 1) * y_head + n > y.shape[1]:
         raise KernelError("head_linear: the heads do not fit the rows")
+    if gate is not None and (gate.dtype != x.dtype or gate.stride(1) != 1 or gate.shape[1] != heads * n):
+        raise KernelError("head_linear: a gate has x's type and one entry per output")
     dims = rot = tx = ty = max_pos = pairs = 0
     cos = sin = positions = status = None
     if turn is not None:
@@ -977,10 +1013,11 @@ def head_linear(x: torch.Tensor, x_col: int, x_head: int, w: torch.Tensor, y: to
             raise KernelError("head_linear: the rotated parts do not fit the rows, or their tables the parts")
     f = _fn(_latent(), "rl_head_linear", [c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_int,
                                           c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                                          c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p])
+                                          c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
     _check(f(_code(x.dtype), _code(w.dtype), _ptr(x), x.stride(0), x_col, x_head, _ptr(w), heads, n, k, _ptr(y),
              y.stride(0), y_col, y_head, tokens if tokens is not None else x.shape[0], impl, dims, rot, 1 if pairs else 0, tx,
-             ty, _ptr(cos), _ptr(sin), max_pos, _ptr(positions), _ptr(status), _stream()), "head_linear")
+             ty, _ptr(cos), _ptr(sin), max_pos, _ptr(positions), _ptr(status), _ptr(gate),
+             gate.stride(0) if gate is not None else 0, _stream()), "head_linear")
 
 
 # ------------------------------------------------------- linear attention with a decaying state
@@ -1079,6 +1116,69 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, seq_of_t
              gate_mode if gate is not None else GATE_NONE, _ptr(norm_w), float(eps),
              _ptr(chunk_state) if chunked else None, _ptr(chunk_decay) if chunked and channel else None, _ptr(status), tokens,
              sequences, heads, vdim, chunk, max_chunks if chunked else 1, longest, _stream()), "linear_attention", 3 if chunked else 1)
+
+
+def _ssm(state: int) -> ctypes.CDLL:
+    if not 1 <= state <= 256:
+        raise KernelError(f"state_space takes state sizes up to 256; got {state}")
+    return _lib(f"state_space_d{state}", "linear_attention.cu", {"RL_LIN_DIM": state, "RL_LIN_TOKEN": 1})
+
+
+SSD_CTAS = 296                     # CTAs that fill the machine: sequences are cut into chunks until there are about so many
+SSD_MIN_CHUNK = 256
+
+
+def state_space_chunks(longest: int, sequences: int, heads: int, vdim: int, blocks: bool) -> Tuple[int, int]:
+    """(chunk length, most chunks) for a step of ``sequences`` sequences of at most ``longest`` tokens; (0, 1) when
+    every sequence is run as one chain.  ``blocks``: for the form that runs blocks of 64 tokens on the tensor cores."""
+    if not blocks:
+        return linear_attention_chunks(longest)
+    ctas = heads * sequences * ((vdim + 63) // 64)
+    chunks = min(16, (SSD_CTAS + ctas - 1) // ctas, longest // SSD_MIN_CHUNK)
+    if chunks <= 1:
+        return 0, 1
+    chunk = ((longest + chunks - 1) // chunks + 63) // 64 * 64
+    return chunk, (longest + chunk - 1) // chunk
+
+
+def state_space(q: torch.Tensor, k: torch.Tensor, qk_heads: int, v: torch.Tensor, steps: torch.Tensor,
+                step_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor, seq_of_token: torch.Tensor,
+                state_slot: torch.Tensor, state: torch.Tensor, out: torch.Tensor, tokens: int, sequences: int, heads: int,
+                dim: int, vdim: int, chunk_state: Optional[torch.Tensor] = None, chunk_decay: Optional[torch.Tensor] = None,
+                chunk: int = 0, max_chunks: int = 1, longest: int = 0) -> None:
+    """The state-space recurrence over every sequence of the step, from and into the sequences' state slots
+    (csrc/linear_attention.cu): per head h, with d_t = softplus(steps_t,h + step_bias_h),
+    S_t = exp(-exp(a_log_h) d_t) S_(t-1) + d_t k_t v_t^T and out_t = S_t^T q_t + skip_h v_t.  q, k
+    [tokens, qk_heads * dim] (head h reads head h // (heads / qk_heads)), v [tokens, heads * vdim] and steps
+    [tokens, heads] are row-strided views of one type; step_bias, a_log and skip float32 [heads]; state and out as for
+    ``linear_attention``, as are ``chunk_state``, ``chunk``, ``max_chunks`` and ``longest``; ``chunk_decay`` (float32,
+    sequences * max_chunks * heads) goes with ``chunk_state``."""
+    _need_cuda(q, k, v, steps, step_bias, a_log, skip, state, out, chunk_state, chunk_decay)
+    for t in (step_bias, a_log, skip, out, chunk_state, chunk_decay):
+        if t is not None and (t.dtype != torch.float32 or not t.is_contiguous()):
+            raise KernelError("state_space: constants, sums and chunk workspace are contiguous float32")
+    flat = state.view(state.shape[0], -1) if state.is_contiguous() else state
+    if state.dtype != torch.float32 or flat.stride(1) != 1 or flat.shape[1] < heads * dim * vdim:
+        raise KernelError("state_space: the state is float32 [slots, heads * dim * vdim]")
+    if any(t.dtype != q.dtype or t.stride(1) != 1 for t in (q, k, v, steps)) or heads % qk_heads != 0 \
+            or q.shape[1] != qk_heads * dim or k.shape[1] != qk_heads * dim or v.shape[1] != heads * vdim \
+            or steps.shape[1] != heads or out.shape[1] != heads * vdim:
+        raise KernelError("state_space: q, k [tokens, qk_heads * dim], v [tokens, heads * vdim] and steps [tokens, heads] of one type")
+    if any(t.numel() != heads for t in (step_bias, a_log, skip)):
+        raise KernelError("state_space: one constant per head")
+    chunked = chunk_state is not None and max_chunks > 1
+    if chunked and (chunk_decay is None or chunk_state.numel() < sequences * max_chunks * heads * dim * vdim
+                    or chunk_decay.numel() < sequences * max_chunks * heads):
+        raise KernelError("state_space: chunk workspace too small")
+    f = _fn(_ssm(dim), "rl_state_space",
+            [c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
+             c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+             c_int, c_void_p])
+    _check(f(_code(q.dtype), _ptr(q), q.stride(0), _ptr(k), k.stride(0), qk_heads, _ptr(v), v.stride(0), _ptr(steps),
+             steps.stride(0), _ptr(step_bias), _ptr(a_log), _ptr(skip), _ptr(seq_of_token), _ptr(state_slot), _ptr(state),
+             flat.stride(0), _ptr(out), _ptr(chunk_state) if chunked else None, _ptr(chunk_decay) if chunked else None,
+             tokens, sequences, heads, vdim, chunk, max_chunks if chunked else 1, longest, _stream()), "state_space",
+           3 if chunked else 1)
 
 
 # ------------------------------------------------------- matrix memory with exponential gates
@@ -1213,25 +1313,26 @@ def pair_norm_mean(a: torch.Tensor, wa: torch.Tensor, ca: float, b: torch.Tensor
 
 def short_conv(x: torch.Tensor, col_x: int, w: torch.Tensor, bias: Optional[torch.Tensor], y: torch.Tensor, col_y: int,
                act: int, seq_of_token: torch.Tensor, state_slot: torch.Tensor, state: torch.Tensor, tokens: int,
-               single: bool = False) -> None:
+               single: bool = False, out_bias: Optional[torch.Tensor] = None) -> None:
     """Causal convolution over time on ``w.shape[0]`` channels of x's rows, from column ``col_x``, into y's from
-    ``col_y`` (another buffer): y_t = act(sum_j w[c, j] (x_(t - taps + 1 + j) + bias_c)) within a token's own
-    sequence; what lies before the step's portion comes from the sequence's slot of ``state`` (float32
+    ``col_y`` (another buffer): y_t = act(sum_j w[c, j] (x_(t - taps + 1 + j) + bias_c) + out_bias_c) within a
+    token's own sequence; what lies before the step's portion comes from the sequence's slot of ``state`` (float32
     [slots, (taps - 1) * channels]: the last inputs, zeros for a new request), which is then moved on
     (csrc/stream_ops.cu).  ``act``: ACT_NONE or ACT_SILU.  ``single``: every sequence of the step has exactly one
     token (one launch instead of two)."""
-    _need_cuda(x, w, bias, y, state)
+    _need_cuda(x, w, bias, y, state, out_bias)
     channels, taps = w.shape
     if x.dtype != y.dtype or x.stride(1) != 1 or y.stride(1) != 1 or not w.is_contiguous() \
             or x.data_ptr() == y.data_ptr() or not 1 <= taps <= MAX_CONV_TAPS or act not in (ACT_NONE, ACT_SILU):
         raise KernelError(f"short_conv: two buffers of one type, contiguous weights [channels, taps <= {MAX_CONV_TAPS}]")
     if state.dtype != torch.float32 or state.stride(1) != 1 or state.shape[1] < (taps - 1) * channels:
         raise KernelError("short_conv: the state is float32 [slots, (taps - 1) * channels]")
-    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != channels or not bias.is_contiguous()):
-        raise KernelError("short_conv: the bias is contiguous float32 [channels]")
-    f = _fn(_so(), "rl_short_conv", [c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
+    for b in (bias, out_bias):
+        if b is not None and (b.dtype != torch.float32 or b.numel() != channels or not b.is_contiguous()):
+            raise KernelError("short_conv: a bias is contiguous float32 [channels]")
+    f = _fn(_so(), "rl_short_conv", [c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                      c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_int, c_void_p])
-    _check(f(_code(x.dtype), _ptr(x), x.stride(0), col_x, _ptr(w), _code(w.dtype), _ptr(bias), _ptr(y), y.stride(0),
+    _check(f(_code(x.dtype), _ptr(x), x.stride(0), col_x, _ptr(w), _code(w.dtype), _ptr(bias), _ptr(out_bias), _ptr(y), y.stride(0),
              col_y, channels, taps, act, _ptr(seq_of_token), _ptr(state_slot), _ptr(state), state.stride(0), tokens,
              1 if single else 0, _stream()), "short_conv", 2 if (taps > 1 and not single) else 1)
 
@@ -1490,9 +1591,10 @@ def gather_logprob(logits: torch.Tensor, rows: int, target: torch.Tensor, out: t
 
 
 def build_all(head_dims=(64, 128), maps_dims=((64, 128, 2), (128, 128, 1)), linear_dims=(64,), memory_dims=(64,),
-              delta_dims=(128,), verbose: bool = True) -> None:
+              delta_dims=(128,), state_dims=(), verbose: bool = True) -> None:
     """Compiles every kernel family (attention for the given head sizes, attention with score maps for the
-    given (key size, value size, maps), linear attention and the matrix memory for the given key sizes) and
+    given (key size, value size, maps), linear attention, the matrix memory, the delta rule and the state-space
+    recurrence for the given key sizes) and
     removes built files of these modules that belong to other versions of the sources."""
     jobs = [(m, f"{m}.cu", None) for m in ("elementwise", "gemm_simt", "gemm_skinny", "gemm_tc", "gemm_mid", "sampling", "rowwise",
                                            "moe", "latent", "stream_ops")]
@@ -1505,6 +1607,7 @@ def build_all(head_dims=(64, 128), maps_dims=((64, 128, 2), (128, 128, 1)), line
         jobs.append((name, "attention_maps.cu", defines))
     jobs += [(f"linear_attention_d{d}", "linear_attention.cu", {"RL_LIN_DIM": d}) for d in linear_dims]
     jobs += [(f"matrix_memory_d{d}", "matrix_memory.cu", {"RL_MM_DIM": d}) for d in memory_dims]
+    jobs += [(f"state_space_d{d}", "linear_attention.cu", {"RL_LIN_DIM": d, "RL_LIN_TOKEN": 1}) for d in state_dims]
     jobs += [(f"delta_rule_d{d}", "delta_rule.cu", {"RL_DELTA_DIM": d}) for d in delta_dims]
     with ThreadPoolExecutor(max(1, min(8, os.cpu_count() or 1))) as pool:
         built = list(pool.map(lambda job: build.compile_module(*job, verbose=verbose), jobs))

@@ -22,6 +22,10 @@ directly behind the projection (and its biases), whose last inputs are the mixer
 only the keys are cached and the kernels read them twice); ``distance_slopes``: one number per head, times the
 distance between query and key, is taken off every score; ``sink_value``: a constant in place of the learned
 sink (0.0 adds a one to every denominator).
+``chunk``: in place of a window, a position sees the keys of its own chunk of so many positions only (chunks are
+counted from position 0).  ``own_kv`` False: there are no keys and values of its own, the layer attends over those
+that an earlier layer has cached (its call of the run order names the other call in ``cache_of``; masks may differ:
+``keep_for`` then says what both need kept).
 
 The cache holds keys [kv_heads * maps, dim] and values [kv_heads, vdim] per token (a window group that
 keeps its first pages); sequences that bring one token go to the partitioned decode kernel, longer
@@ -70,6 +74,9 @@ class MapsAttentionParams:
     values_are_keys: bool = False            # no W_v: v = k as projected; only k is cached
     distance_slopes: Optional[tuple] = None  # per head: s_ij <- s_ij - slope_h * (i - j)
     sink_value: Optional[float] = None       # a constant sink for every head (with ``sink`` False)
+    chunk: int = 0               # > 0: positions see the keys of their own chunk of so many positions (no window)
+    own_kv: bool = True          # False: another layer's cached keys and values are attended over
+    keep_for: Optional[tuple] = None         # (cache kind, span) if the cache serves other masks than this layer's too
 
 
 @register("mixer", "maps_attention")
@@ -110,10 +117,16 @@ class MapsAttention(Mixer):
                                   or p.head_norm != "none" or p.value_mix != "none"):
             raise ValueError("values_are_keys goes with one map, vdim = dim, and no bias, convolution, position "
                              "encoding, head norm or value blend")
+        if p.chunk < 0 or (p.chunk > 0 and (p.window > 0 or p.keep_first > 0)):
+            raise ValueError("chunked attention has no window and keeps no first tokens")
+        if not p.own_kv and (p.values_are_keys or p.conv_taps > 0 or p.value_mix != "none"
+                             or (p.position is not None and self.rotary is None)):
+            raise ValueError("attention over another layer's keys goes without value options, convolutions and position "
+                             "encodings that are not rotations")
         self.scale = p.scale if p.scale is not None else 1.0 / math.sqrt(p.dim)
         self.q_size = p.num_heads * p.maps * p.dim
-        self.k_size = p.num_kv_heads * p.maps * p.dim
-        self.v_size = 0 if p.values_are_keys else p.num_kv_heads * p.vdim
+        self.k_size = p.num_kv_heads * p.maps * p.dim if p.own_kv else 0
+        self.v_size = 0 if p.values_are_keys or not p.own_kv else p.num_kv_heads * p.vdim
         self.qkv_size = self.q_size + self.k_size + self.v_size
         self.out_size = p.num_heads * p.vdim
         self.gate_size = {"none": 0, "head": p.num_heads, "entry": self.out_size}[p.gate]
@@ -139,8 +152,12 @@ class MapsAttention(Mixer):
         tensors = (CacheTensor("k", (p.num_kv_heads * p.maps, p.dim)),)
         if not p.values_are_keys:
             tensors += (CacheTensor("v", (p.num_kv_heads, p.vdim)),)
+        if p.keep_for is not None:
+            return CacheSpec(p.keep_for[0], tensors, p.keep_for[1])
         if p.window > 0:
             return CacheSpec("window", tensors, p.window, p.keep_first)
+        if p.chunk > 0:
+            return CacheSpec("chunk", tensors, p.chunk)
         return CacheSpec("full", tensors)
 
     def tiling(self):
@@ -159,12 +176,15 @@ class MapsAttention(Mixer):
         }
         if p.values_are_keys:
             del t["v"], t["v_bias"]
+        if not p.own_kv:
+            del t["k"], t["v"], t["k_bias"], t["v_bias"]
         if p.maps == 2:
             t.update({n: TensorSpec((p.dim,)) for n in ("lq1", "lk1", "lq2", "lk2")})
         if p.head_norm != "none":
             whole = p.head_norm == "whole"
             t["q_norm"] = TensorSpec((self.q_size if whole else p.dim,))
-            t["k_norm"] = TensorSpec((self.k_size if whole else p.dim,))
+            if p.own_kv:
+                t["k_norm"] = TensorSpec((self.k_size if whole else p.dim,))
         if p.sink:
             t["sink"] = TensorSpec((p.num_heads,))
         if p.gate != "none":
@@ -179,8 +199,9 @@ class MapsAttention(Mixer):
         return t
 
     def fused(self) -> Dict[str, list]:
-        out = {"qkv": ["q", "k"] + ([] if self.params.values_are_keys else ["v"])
-               + (["g"] if self.params.gate != "none" else [])}
+        p = self.params
+        out = {"qkv": ["q"] + (["k"] if p.own_kv else []) + (["v"] if p.own_kv and not p.values_are_keys else [])
+               + (["g"] if p.gate != "none" else [])}
         if self.params.conv_taps > 0:
             out["qkv_conv"] = ["q_conv", "k_conv", "v_conv"]
         return out
@@ -211,7 +232,8 @@ class MapsAttention(Mixer):
                 torch.cat([tensors[n] for n in ("q_conv", "k_conv", "v_conv")], dim=0).contiguous()
         self.b_qkv = None
         if p.bias:
-            self.b_qkv = torch.cat([tensors[n].float() for n in ("q_bias", "k_bias", "v_bias")]).contiguous()
+            names = ("q_bias", "k_bias", "v_bias") if p.own_kv else ("q_bias",)
+            self.b_qkv = torch.cat([tensors[n].float() for n in names]).contiguous()
         if p.maps == 2:
             # one number for the layer, in float32 like everything around the scores
             lq1, lk1, lq2, lk2 = (tensors[n].float() for n in ("lq1", "lk1", "lq2", "lk2"))
@@ -253,6 +275,8 @@ class MapsAttention(Mixer):
         qkv = ws.get("mattn.qkv", (rt.max_tokens, self.proj_size), rt.dtype)[:T]
         linear(x, self.w_qkv, qkv)
         gate_buf = qkv                     # where the gate's columns lie
+        prepared = self.rotary is not None or self.norm_mode != kernels.HEAD_NORM_NONE or self.mix_mode != kernels.VALUE_MIX_NONE
+        bias = self.b_qkv if self.w_conv is None else None      # the biases that the kernel behind the product adds
         if self.w_conv is not None:
             # (the biases are added on the way into the convolution, whose state keeps the biased inputs)
             conv = ws.get("mattn.qkv_conv", (rt.max_tokens, self.proj_size), rt.dtype)[:T]
@@ -261,12 +285,13 @@ class MapsAttention(Mixer):
             kernels.short_conv(qkv, 0, self.w_conv, self.b_qkv, conv, 0, kernels.ACT_NONE, ctx.seq_of_token,
                                ctx.state_slot, state, T, single=ctx.num_decode == ctx.S == T)
             qkv = conv
-        elif self.b_qkv is not None:
+        elif self.b_qkv is not None and (not prepared or (self.position is not None and self.rotary is None)):
+            bias = None
             kernels.bias_act(qkv, self.b_qkv, kernels.ACT_NONE, cols=self.qkv_size)
         op_mark(ctx, "qkv_proj", self.w_qkv, T)
         if self.position is not None and self.rotary is None:
             self.position.apply(qkv, p.num_heads * p.maps, p.num_kv_heads * p.maps, p.dim, ctx)
-        if self.rotary is not None or self.norm_mode != kernels.HEAD_NORM_NONE or self.mix_mode != kernels.VALUE_MIX_NONE:
+        if prepared:
             v_first = None
             if self.mix_mode != kernels.VALUE_MIX_NONE:
                 # (the layers run one after another within a step: the buffer holds this step's tokens)
@@ -274,11 +299,13 @@ class MapsAttention(Mixer):
             cos, sin = self.rotary if self.rotary is not None else (None, None)
             g = ctx.groups[cache.group]
             # (the same kernel puts the finished keys and values into the cache)
-            kernels.head_prep(qkv, ctx.positions, T, 0, p.num_heads * p.maps, self.q_size, p.num_kv_heads * p.maps, p.dim,
+            own = cache.write and p.own_kv
+            kernels.head_prep(qkv, ctx.positions, T, 0, p.num_heads * p.maps, self.q_size,
+                              p.num_kv_heads * p.maps if p.own_kv else 0, p.dim,
                               ctx.status, self.w_qnorm, self.w_knorm, self.norm_mode, p.eps, cos, sin,
                               self.q_size + self.k_size, self.v_size, v_first, self.mix_mode, self.mix,
-                              g.slots if cache.write else None, cache.tensors["k"], cache.tensors["v"], rt.page_size,
-                              halves=self.rotary is not None and self.halves)
+                              g.slots if own else None, cache.tensors["k"], cache.tensors["v"], rt.page_size,
+                              halves=self.rotary is not None and self.halves, bias=bias)
             op_mark(ctx, "qk_norm+rotate+kv_write", nbytes=(2.0 * self.qkv_size + self.k_size + self.v_size) * T * qkv.element_size())
             stored = True
         else:
@@ -286,7 +313,7 @@ class MapsAttention(Mixer):
         g = ctx.groups[cache.group]
         k_cache = cache.tensors["k"]
         v_cache = k_cache if p.values_are_keys else cache.tensors["v"]
-        if cache.write and not stored:
+        if cache.write and p.own_kv and not stored:
             kernels.cache_store(qkv, self.q_size, p.num_kv_heads * p.maps, p.dim, g.slots, k_cache, rt.page_size,
                                 ctx.status, tokens=T)
             if not p.values_are_keys:
@@ -302,12 +329,13 @@ class MapsAttention(Mixer):
             part_o = ws.get("mattn.part_o", (rows * p.vdim,), torch.float32)
             part_ml = ws.get("mattn.part_ml", (rows * 2,), torch.float32)
             kernels.maps_attn_decode(qkv, self.proj_size, k_cache, v_cache, g.block_table, ctx.decode_info, part_o,
-                                     part_ml, ctx.decode_parts, attn, ctx.num_decode, *common, slopes=self.slopes)
+                                     part_ml, ctx.decode_parts, attn, ctx.num_decode, *common, slopes=self.slopes,
+                                     chunk=p.chunk)
             self._mark(ctx, "attention_decode", "decode")
         if ctx.num_tiles > 0:
             kernels.maps_attn_prefill(qkv, self.proj_size, k_cache, v_cache, g.block_table, ctx.tile_seq, ctx.tile_tok,
                                       ctx.tile_rows, ctx.positions, attn, ctx.num_tiles, kernels.PREFILL_TILE_ROWS,
-                                      *common, slopes=self.slopes)
+                                      *common, slopes=self.slopes, chunk=p.chunk)
             self._mark(ctx, "attention_prefill", "prefill")
 
     def _mark(self, ctx, op: str, which: str) -> None:
@@ -316,7 +344,7 @@ class MapsAttention(Mixer):
         from ..engine.profiler import attention_work
         p = self.params
         elem = 2 if self.rt.dtype == torch.bfloat16 else 4
-        window = p.window + p.keep_first if p.window > 0 else 0
+        window = p.window + p.keep_first if p.window > 0 else p.chunk      # (of a chunk the mean token sees half)
         nbytes, flops = attention_work(ctx.host, p.num_heads * p.maps, p.num_kv_heads * p.maps, (p.dim + p.vdim) // 2,
                                        window, elem)[which]
         ctx.profiler.mark(op, nbytes, flops)

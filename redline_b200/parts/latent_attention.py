@@ -3,7 +3,7 @@
 Per token the mixer projects its input to queries (per head ``dim`` unrotated and ``rot_dim`` rotated entries)
 and to [c' | k_r]: a latent of ``kv_rank`` entries, RMS-normed with a weight into c, and one rotated key part
 of ``rot_dim`` entries that all heads share.  Head h's key is [W_uk,h c | k_r], its value W_uv,h c; scores are
-scale * q . k over every earlier token, ordinary softmax.  Only [c | k_r] is cached (one row per token, one
+scale * q . k over every earlier token (or those of a window), ordinary softmax.  Only [c | k_r] is cached (one row per token, one
 "key head" for all query heads), and the keys and values are never formed:
 
     q_n . (W_uk,h c_j) = (W_uk,h^T q_n) . c_j          sum_j p_j W_uv,h c_j = W_uv,h (sum_j p_j c_j)
@@ -16,8 +16,9 @@ first ``rot_dims`` entries of the rotated part.  Norm, rotation, scores and soft
 types.
 
 Further options: the queries may come from a latent of their own, q = W_uq rmsnorm(W_dq h) (``q_rank``); every
-head's output may be multiplied by sigmoid(W_g h)_h (``gated``; applied by the attention kernels to what they
-return, which W_uv,h maps linearly); a layer may attend over the rows that an earlier layer has cached
+head's output may be multiplied by sigmoid(W_g h)_h (``gate`` "head"; applied by the attention kernels to what they
+return, which W_uv,h maps linearly) or entry by entry ("entry": W_g h has a number per output entry; applied by the
+product with W_uv,h to its result); ``window`` > 0: a token sees itself and the ``window`` - 1 tokens before it; a layer may attend over the rows that an earlier layer has cached
 (``own_latent`` False: no W_dkv; its call of the run order names the other call in ``cache_of``).  What is
 projected from h, [q or the queries' latent | latent | key part | gate], is one product.
 """
@@ -47,8 +48,9 @@ class LatentAttentionParams:
     eps: float = 1e-6            # of the latent's RMS norm
     position: Optional[PartSpec] = None      # an encoding of the rotated part (needed if rot_dim > 0)
     q_rank: int = 0              # > 0: size of the latent the queries come from
-    gated: bool = False          # a sigmoid gate per head
+    gate: str = "none"           # none | head | entry: a sigmoid gate per head or per output entry
     own_latent: bool = True      # False: another layer's cached rows are attended over
+    window: int = 0              # 0: every earlier token
 
 
 @register("mixer", "latent_attention")
@@ -62,6 +64,8 @@ class LatentAttention(Mixer):
         if self.key_size > kernels.MAPS_MAX_DIM or p.kv_rank > kernels.MAPS_MAX_VDIM:
             raise ValueError(f"latent_attention: kv_rank + rot_dim is {self.key_size}; the attention kernels take "
                              f"rows of up to {kernels.MAPS_MAX_DIM} entries of which {kernels.MAPS_MAX_VDIM} are the latent")
+        if p.gate not in ("none", "head", "entry") or p.window < 0:
+            raise ValueError(f"latent_attention: gate '{p.gate}' is not known (none, head, entry), or a negative window")
         self.cos = self.sin = None
         self.rot_dims = 0
         self.pairs = False
@@ -82,13 +86,15 @@ class LatentAttention(Mixer):
         # columns of the projection from h: queries or their latent, then (own) latent and key part, then gates
         self.c_col = p.q_rank or self.q_size
         self.g_col = self.c_col + (self.key_size if p.own_latent else 0)
-        self.proj_size = self.g_col + (p.num_heads if p.gated else 0)
+        self.gate_size = {"none": 0, "head": p.num_heads, "entry": p.num_heads * p.vdim}[p.gate]
+        self.proj_size = self.g_col + self.gate_size
         self.qa_size = p.num_heads * self.key_size
         self.lat_size = p.num_heads * p.kv_rank
         self.out_size = p.num_heads * p.vdim
 
     def cache_spec(self) -> CacheSpec:
-        return CacheSpec("full", (CacheTensor("k", (1, self.key_size)),))
+        tensors = (CacheTensor("k", (1, self.key_size)),)
+        return CacheSpec("window", tensors, self.params.window) if self.params.window > 0 else CacheSpec("full", tensors)
 
     def tiling(self):
         return kernels.PREFILL_TILE_ROWS, kernels.DECODE_PARTITION
@@ -109,13 +115,13 @@ class LatentAttention(Mixer):
         if p.own_latent:
             t["dkv"] = TensorSpec((self.key_size, p.hidden_size))
             t["dkv_norm"] = TensorSpec((p.kv_rank,))
-        if p.gated:
-            t["g"] = TensorSpec((p.num_heads, p.hidden_size))
+        if p.gate != "none":
+            t["g"] = TensorSpec((self.gate_size, p.hidden_size))
         return t
 
     def _projected(self) -> list:
         p = self.params
-        return ["dq" if p.q_rank > 0 else "q"] + (["dkv"] if p.own_latent else []) + (["g"] if p.gated else [])
+        return ["dq" if p.q_rank > 0 else "q"] + (["dkv"] if p.own_latent else []) + (["g"] if p.gate != "none" else [])
 
     def fused(self) -> Dict[str, list]:
         return {"from_input": self._projected()}
@@ -175,10 +181,10 @@ class LatentAttention(Mixer):
         kernels.head_linear(q, 0, self.q_head, self.w_uk_t, qa, 0, self.key_size, tokens=T, turn=turn)
         op_mark(ctx, "q_absorb", nbytes=float(T * p.num_heads * (p.dim + p.kv_rank) * elem + self.w_uk_t.numel() * elem),
                 flops=2.0 * T * p.num_heads * p.dim * p.kv_rank)
-        gate = dict(gate=proj[:, self.g_col:], gate_mode=1) if p.gated else {}
+        gate = dict(gate=proj[:, self.g_col:], gate_mode=1) if p.gate == "head" else {}
         lat = ws.get("latent.out", (rt.max_tokens, self.lat_size), rt.dtype)[:T]
         v_stride = self.key_size if p.rot_dim > 0 else 0
-        common = (p.num_heads, 1, self.key_size, p.kv_rank, 1, rt.page_size, 0, 0, p.scale, 0.0, 0.0, 1.0, p.eps, False)
+        common = (p.num_heads, 1, self.key_size, p.kv_rank, 1, rt.page_size, p.window, 0, p.scale, 0.0, 0.0, 1.0, p.eps, False)
         if ctx.num_decode > 0:
             rows = ctx.max_items * p.num_heads * ctx.parts_capacity
             part_o = ws.get("mattn.part_o", (rows * p.kv_rank,), torch.float32)
@@ -192,7 +198,8 @@ class LatentAttention(Mixer):
                                       *common, v_stride=v_stride, **gate)
             self._mark(ctx, "attention_prefill", "prefill")
         heads_v = ws.get("latent.values", (rt.max_tokens, self.out_size), rt.dtype)[:T]
-        kernels.head_linear(lat, 0, p.kv_rank, self.w_uv, heads_v, 0, p.vdim, tokens=T)
+        kernels.head_linear(lat, 0, p.kv_rank, self.w_uv, heads_v, 0, p.vdim, tokens=T,
+                            gate=proj[:, self.g_col:] if p.gate == "entry" else None)
         op_mark(ctx, "v_up", nbytes=float(T * p.num_heads * (p.vdim + p.kv_rank) * elem + self.w_uv.numel() * elem),
                 flops=2.0 * T * p.num_heads * p.vdim * p.kv_rank)
         out = ws.get("mixer.out", (rt.max_tokens, p.hidden_size), rt.dtype)[:T]
@@ -206,5 +213,5 @@ class LatentAttention(Mixer):
         from ..engine.profiler import attention_work
         p = self.params
         elem = 2 if self.rt.dtype == torch.bfloat16 else 4
-        nbytes, flops = attention_work(ctx.host, p.num_heads, 1, (self.key_size + p.kv_rank) // 2, 0, elem)[which]
+        nbytes, flops = attention_work(ctx.host, p.num_heads, 1, (self.key_size + p.kv_rank) // 2, p.window, elem)[which]
         ctx.profiler.mark(op, nbytes, flops)

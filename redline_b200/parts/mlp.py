@@ -2,8 +2,8 @@
 projection [gate | up]; act is SiLU (reference: src/cuda/model/llama.cpp:134-136,
 src/cuda/kernels/elementwise.cu:66-82) unless the parameters name another activation
 (``gelu_tanh`` and the others of ``kernels.ACTIVATIONS``, or ``clamped_swish``: gate and up clamped,
-g * sigmoid(slope * g) * (up + 1)), which runs as a kernel of its own behind the product; prompt portions have the tcgen05 kernel's gated epilogue for SiLU and
-the tanh GELU, and so has the weight-streaming product for at most 16 rows; the forms that also
+g * sigmoid(slope * g) * (up + 1)), which runs as a kernel of its own behind the product; prompt portions have the tcgen05 kernel's gated epilogue for SiLU,
+the tanh GELU and ReLU, and so has the weight-streaming product for at most 16 rows; the forms that also
 fuse the norm before and the add behind are SiLU's."""
 
 from __future__ import annotations
@@ -87,7 +87,8 @@ class SwiGLUMLP(FeedForward):
         T = ctx.T
         ws = rt.workspace
         act = ws.get(name + ".act", (rt.max_tokens, p.intermediate_size), rt.dtype)[:T]
-        tc_epilogue = {"silu": kernels.EPI_SWIGLU, "gelu_tanh": kernels.EPI_GEGLU_TANH}.get(self.params.activation)
+        tc_epilogue = {"silu": kernels.EPI_SWIGLU, "gelu_tanh": kernels.EPI_GEGLU_TANH,
+                       "relu": kernels.EPI_REGLU}.get(self.params.activation)
         if (tc_epilogue is not None and T >= TC_MIN_ROWS and self.b_gate_up is None
                 and kernels.gemm_tc_ok(x, self.w_gate_up)):
             # prompt portions: gate/up product and the gated activation in one tcgen05 kernel

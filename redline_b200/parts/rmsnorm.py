@@ -1,7 +1,8 @@
 """RMSNorm fused with the residual add: y = x * rsqrt(mean(x^2) + eps) * w with the
 weight multiplying directly, sums in float32
 (reference: src/cuda/kernels/elementwise.cu:29-64); designs that store the weight around
-zero (``zero_centred``) multiply by 1 + w, formed in float32 when the weights are loaded.
+zero (``zero_centred``) multiply by 1 + w, formed in float32 when the weights are loaded, and
+so is a constant factor on the normed rows (``scale``: a factor on the logits, say).
 ``rmsnorm_sum`` norms the weighted sum of the stream and a sublayer's output, for blocks
 that norm after the sum."""
 
@@ -22,6 +23,7 @@ class RMSNormParams:
     size: int
     eps: float
     zero_centred: bool = False
+    scale: float = 1.0             # the normed rows are multiplied by this
 
 
 @register("norm", "rmsnorm")
@@ -33,6 +35,8 @@ class RMSNorm(Norm):
         self.weight = tensors["weight"]
         if self.params.zero_centred:
             self.weight = (1.0 + self.weight.float()).contiguous()
+        if self.params.scale != 1.0:
+            self.weight = (self.weight.float() * self.params.scale).contiguous()
 
     def nbytes(self) -> int:
         return self.weight.numel() * self.weight.element_size()

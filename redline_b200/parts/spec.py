@@ -109,7 +109,8 @@ class CacheSpec:
     """What a mixer needs cached for each token it has seen.
 
     kind     "full": every token stays; "window": only the last ``window`` tokens (and the first
-             ``keep_first`` ones, if the mixer's mask keeps them visible)
+             ``keep_first`` ones, if the mixer's mask keeps them visible); "chunk": only those of the chunk of
+             ``window`` positions (counted from position 0) that the next token lies in
     tensors  the tensors kept per token, each with a shape of its own (keys and values of the same
              shape for ordinary attention; one latent vector, or keys and values of different widths,
              for other mixers)
