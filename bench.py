@@ -502,10 +502,10 @@ def main() -> int:
     ap.add_argument("--profile-batch", type=int, default=BATCH)
     ap.add_argument("--profile-prompt", type=int, default=0, help="with --profile-step: prompt length (default: context - 96)")
     ap.add_argument("--profile-eager", action="store_true", help="with --profile-step: no CUDA graph")
-    ap.add_argument("--compare-design", default="", choices=["", "kapitar", "pufevik", "vizotar", "venezen", "lakatar"],
+    ap.add_argument("--compare-design", default="", choices=["", "kapitar", "pufevik", "vizotar", "venezen", "lakatar", "vogolix"],
                     help="instead of the headline run: prefill and decode throughput of this architecture beside "
                          "the closest one the package has (Llama; Pufevik for vizotar, Kapitar for venezen, Venezen and "
-                         "Vizotar for lakatar) at equal layer sizes, with the "
+                         "Vizotar for lakatar, Pufevik and Lakatar for vogolix) at equal layer sizes, with the "
                          "per-op roofline fractions of both")
     ap.add_argument("--compare-sizes", default="s,m", help="with --compare-design: which of its sizes (s, m)")
     ap.add_argument("--compare-no-ops", action="store_true", help="with --compare-design: no per-op tables")

@@ -1,5 +1,6 @@
 """Prefill and decode throughput of one architecture beside another at equal layer sizes, with the
-per-op roofline fractions of both (``bench.py --compare-design kapitar``, ``pufevik``, ``vizotar``, ``venezen`` or ``lakatar``).
+per-op roofline fractions of both (``bench.py --compare-design kapitar``, ``pufevik``, ``vizotar``, ``venezen``,
+``lakatar`` or ``vogolix``).
 
 Every size is a handful of layers whose matrices have the shapes of a real model's (random weights):
 the Kapitar model has one layer of every kind (attention + dense, lightning + routed, attention + routed,
@@ -36,6 +37,13 @@ package has (the same attention over latents of the same sizes, the same experts
 feed-forwards are dense and as wide as Lakatar's chosen and shared experts together), and Vizotar for its
 recurrence (the delta rule with a decay per key channel, as many state entries per head as Lakatar's time mixing
 has in two heads), both at the same width.
+
+The Vogolix model has five layers, all with a gated dense feed-forward: chunked attention with a sink, attention over
+its keys and values, two state-space layers, windowed attention over a cached latent.  Beside it stand Pufevik, the
+closest architecture the package has (attention with a sink, norms over the whole projection and neighbouring pairs
+rotated, through the same kernels, over a window as long as the chunk; a gated dense feed-forward of the same width),
+and Lakatar for the latent attention (the same rows) and for its recurrences (retention: as many state entries as half
+a state-space layer's), both at the same width.
 """
 
 from __future__ import annotations
@@ -82,6 +90,13 @@ LAKATAR_SIZES: Dict[str, Dict[str, int]] = {
     "m": dict(width=2048, heads=16, lat_dim=64, rot_dim=32, lat_vdim=64, kv_rank=192, q_rank=768, wkv_heads=32, wkv_dim=64,
               decay_rank=64, ret_heads=8, ret_dim=128, ret_vdim=256, experts=32, top=4, expert_ff=704, shared_ff=1408, groups=4,
               keep=2, vocab=32000),
+}
+VOGOLIX_SIZES: Dict[str, Dict[str, int]] = {
+    # PUFEVIK_SIZES' attention and feed-forward, LAKATAR_SIZES' latent attention, the state-space layers' sizes
+    "s": dict(width=1024, heads=8, kv_heads=2, dim=128, vdim=128, ff=2816, lat_dim=64, rot_dim=32, lat_vdim=64, kv_rank=192,
+              ssm_heads=32, ssm_vdim=64, ssm_state=128, ssm_groups=1, taps=4, vocab=32000),
+    "m": dict(width=2048, heads=16, kv_heads=4, dim=128, vdim=128, ff=5632, lat_dim=64, rot_dim=32, lat_vdim=64, kv_rank=192,
+              ssm_heads=64, ssm_vdim=64, ssm_state=128, ssm_groups=1, taps=4, vocab=32000),
 }
 WINDOW, KEEP_FIRST = 1024, 4
 PROMPT = 2048
@@ -174,13 +189,30 @@ def lakatar_config(s: Dict[str, int]) -> Dict[str, Any]:
                        {"type": "latent_attention", "mixer": dict(latent, kv_from=1), "mlp": moe}]}
 
 
+def vogolix_config(s: Dict[str, int]) -> Dict[str, Any]:
+    att = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["vdim"], "scale": s["dim"] ** -0.5,
+           "mask": {"size": WINDOW}, "rot": {"base": 1000000.0, "dims": s["dim"] // 2}}
+    latent = {"heads": s["heads"], "dim": s["lat_dim"], "rot_dim": s["rot_dim"], "vdim": s["lat_vdim"], "kv_rank": s["kv_rank"],
+              "scale": (s["lat_dim"] + s["rot_dim"]) ** -0.5, "mask": {"size": WINDOW},
+              "rot": {"base": 500000.0, "dims": s["rot_dim"]}}
+    ssm = {"heads": s["ssm_heads"], "vdim": s["ssm_vdim"], "state": s["ssm_state"], "groups": s["ssm_groups"], "norm_groups": 1,
+           "conv": s["taps"]}
+    dense = {"kind": "dense", "ff": s["ff"]}
+    return {"architecture": "Vogolix", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "layers": [{"type": "attention", "mixer": att, "mlp": dense}, {"type": "attention", "mixer": dict(att, kv_from=0), "mlp": dense},
+                       {"type": "mamba2", "mixer": ssm, "mlp": dense}, {"type": "mamba2", "mixer": ssm, "mlp": dense},
+                       {"type": "latent_attention", "mixer": latent, "mlp": dense}]}
+
+
 # design -> (its sizes, its configuration, [(architecture beside it, that one's sizes, its configuration at them)])
 DESIGNS = {"kapitar": (SIZES, kapitar_config, [("llama", SIZES, llama_config)]),
            "pufevik": (PUFEVIK_SIZES, pufevik_config, [("llama", PUFEVIK_SIZES, llama_beside_pufevik)]),
            "vizotar": (VIZOTAR_SIZES, vizotar_config, [("pufevik", VIZOTAR_SIZES, pufevik_config)]),
            "venezen": (VENEZEN_SIZES, venezen_config, [("kapitar", VENEZEN_SIZES, kapitar_config)]),
            "lakatar": (LAKATAR_SIZES, lakatar_config, [("venezen", VENEZEN_SIZES, venezen_config),
-                                                       ("vizotar", VIZOTAR_SIZES, vizotar_config)])}
+                                                       ("vizotar", VIZOTAR_SIZES, vizotar_config)]),
+           "vogolix": (VOGOLIX_SIZES, vogolix_config, [("pufevik", PUFEVIK_SIZES, pufevik_config),
+                                                       ("lakatar", LAKATAR_SIZES, lakatar_config)])}
 
 
 def _prefill(model: str, tokens: int, reps: int, warmup: int) -> float:
@@ -286,7 +318,7 @@ def compare(design: str, sizes: List[str], steps: int, warmup: int, batch: int, 
     with tempfile.TemporaryDirectory() as tmp:
         for name in sizes:
             s = table[name]
-            entry: Dict[str, Any] = {"shape": dict(s, layers=4, window=WINDOW)}
+            entry: Dict[str, Any] = {"shape": dict(s, layers=len(design_config(s)["layers"]), window=WINDOW)}
             if design == "kapitar":
                 entry["shape"]["keep_first"] = KEEP_FIRST
             for arch, cfg in [(design, design_config(s))] + [(b, conf(sizes_of[name])) for b, sizes_of, conf in beside]:

@@ -9,6 +9,7 @@ package, if present).
     python -m redline_b200.apps.kernel_bench head_linear --tokens 2048 --heads 16 --n 192 --k 64 [--impl 1]
     python -m redline_b200.apps.kernel_bench latent_attn --tokens 2048 --heads 16 --rank 192 --rot 32 [--impl 1]
     python -m redline_b200.apps.kernel_bench recurrence --tokens 2048 --heads 32 --head-dim 64 --vdim 64 [--channel] [--seqs 1]
+    python -m redline_b200.apps.kernel_bench state_space --tokens 2048 --heads 64 --qk-heads 1 --head-dim 128 --vdim 64 [--seqs 1]
 
 Each kernel runs over several distinct copies of its large operands (more than the
 L2 holds), captured in a CUDA graph so that launch overhead of the host is not
@@ -325,10 +326,46 @@ def bench_recurrence(args) -> None:
                       "copies": copies}))
 
 
+def bench_state_space(args) -> None:
+    """The state-space recurrence over sequences of equal length, cut as the engine cuts them, float32 sums out."""
+    dev, bf = "cuda", torch.bfloat16
+    H, G, D, DV, S = args.heads, args.qk_heads, args.head_dim, args.vdim, args.seqs
+    per = args.tokens // S
+    T = per * S
+    copies = max(2, min(args.copies, int(2e9 // (T * (2 * G * D + H * DV) * 2 + S * H * D * DV * 4))))
+    q, k = ([torch.randn(T, G * D, device=dev).to(bf) for _ in range(copies)] for _ in range(2))
+    v = [torch.randn(T, H * DV, device=dev).to(bf) for _ in range(copies)]
+    z = [torch.randn(T, H, device=dev).to(bf) for _ in range(copies)]
+    bias, a_log, skip = torch.full((H,), -3.0, device=dev), torch.ones(H, device=dev), torch.randn(H, device=dev)
+    seq = (torch.arange(T, dtype=torch.int32) // per).to(dev)
+    slot = torch.arange(S, dtype=torch.int32, device=dev)
+    state = [torch.zeros(S, H * D * DV, device=dev) for _ in range(copies)]
+    o = torch.empty(T, H * DV, device=dev)
+    blocks = args.impl == 0 and D % 16 == 0 and DV % 16 == 0
+    chunk, chunks = kernels.state_space_chunks(per, T, H, DV, blocks)
+    if args.chunk:
+        chunk, chunks = args.chunk, (per + args.chunk - 1) // args.chunk
+    kw = dict(chunk=chunk, max_chunks=chunks, longest=0 if args.impl == 1 else per)
+    if chunks > 1:
+        kw.update(chunk_state=torch.empty(S * chunks * H * D * DV, device=dev), chunk_decay=torch.empty(S * chunks * H, device=dev))
+
+    def fn(i):
+        i %= copies
+        kernels.state_space(q[i], k[i], G, v[i], z[i], bias, a_log, skip, seq, slot, state[i], o, T, S, H, D, DV, **kw)
+
+    us = graph_time_us(fn, copies, use_graph=not args.no_graph)
+    nbytes = T * (2.0 * (2 * G * D + H * DV + H) + 4.0 * H * DV) + 8.0 * S * H * D * DV
+    pk = peaks()
+    print(json.dumps({"kernel": "state_space", "tokens": T, "seqs": S, "heads": H, "qk_heads": G, "state": D, "vdim": DV,
+                      "chunk": chunk, "us": round(us, 2), "GB/s": round(nbytes / us / 1e3, 1),
+                      "TFLOP/s": round(4.0 * T * H * D * DV / us / 1e6, 2),
+                      "frac_of_measured_hbm": round(nbytes / us / 1e3 / pk["hbm_gbs"], 3), "copies": copies}))
+
+
 def main() -> int:
     ap = argparse.ArgumentParser(description=__doc__, formatter_class=argparse.RawDescriptionHelpFormatter)
     sub = ap.add_subparsers(dest="kernel", required=True)
-    for name in ("attn_decode", "attn_prefill", "skinny", "gemm_tc", "gemm_mid", "head_linear", "latent_attn", "recurrence"):
+    for name in ("attn_decode", "attn_prefill", "skinny", "gemm_tc", "gemm_mid", "head_linear", "latent_attn", "recurrence", "state_space"):
         p = sub.add_parser(name)
         p.add_argument("--heads", type=int, default=32)
         p.add_argument("--kv-heads", type=int, default=8)
@@ -348,7 +385,9 @@ def main() -> int:
             p.add_argument("--k", type=int, default=64, help="head_linear: inputs of a head")
             p.add_argument("--rank", type=int, default=192, help="latent_attn: size of the cached latent")
             p.add_argument("--rot", type=int, default=32, help="latent_attn: size of the rotated key part")
-        if name == "recurrence":
+        if name == "state_space":
+            p.add_argument("--qk-heads", type=int, default=1, help="groups of heads that share their queries and keys")
+        if name in ("recurrence", "state_space"):
             p.add_argument("--tokens", type=int, default=2048)
             p.add_argument("--vdim", type=int, default=64)
             p.add_argument("--seqs", type=int, default=1, help="sequences of equal length (tokens in all)")
@@ -390,7 +429,8 @@ def main() -> int:
         return 1
     {"attn_decode": bench_attn_decode, "attn_prefill": bench_attn_prefill, "skinny": bench_skinny,
      "gemm_tc": bench_gemm_tc, "gemm_mid": bench_gemm_mid, "head_linear": bench_head_linear,
-     "latent_attn": bench_latent_attn, "recurrence": bench_recurrence}[args.kernel](args)
+     "latent_attn": bench_latent_attn, "recurrence": bench_recurrence,
+     "state_space": bench_state_space}[args.kernel](args)
     return 0
 
 

@@ -109,7 +109,9 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
 // stream-serialization attribute, a kernel may begin (be scheduled, run its prologue, ask
 // for weights that no earlier kernel writes) while its predecessor is still draining; it
 // calls pdl_wait() before it touches anything an earlier kernel of the chain wrote, which
-// returns once the predecessor has completed and its writes are visible.  pdl_launch()
+// returns once the predecessor has completed and its writes are visible.  (In a kernel that loads constants before
+// pdl_wait(), pointers to what earlier kernels wrote are not `const __restrict__`: loads through such a pointer count
+// as loads of memory that never changes, and the compiler may move them up across the wait.)  pdl_launch()
 // tells the scheduler that the successor may be brought in.  Without the attribute both
 // are no-ops.  REDLINE_PDL=0 in the environment turns the attribute off.
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }

@@ -278,7 +278,7 @@ head_linear_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, b
 constexpr int kHfTokens = 8, kHfCols = 4;
 template <bool TURN>
 __global__ void __launch_bounds__(128)
-head_linear_few_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16* __restrict__ y, const HeadLinearArgs a) {
+head_linear_few_kernel(const bf16* x, const bf16* __restrict__ w, bf16* __restrict__ y, const HeadLinearArgs a) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y, t0 = blockIdx.z * kHfTokens;
   pdl_launch();

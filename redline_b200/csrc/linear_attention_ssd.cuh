@@ -8,8 +8,9 @@
 // Every exponent is a sum of negative numbers.  All four products run on mma.sync with float32 accumulators; q, k and v
 // are bfloat16 as they are, and what is not (the state, M, the weighted values) enters as a high and a low part, so
 // that the result is off by some 2^-16 of its terms.  A CTA takes one sequence (chunk), one head and up to 64 value
-// columns; a warp takes 16 of the block's tokens for the outputs, and every fourth 16 rows of the state, which it keeps
-// as accumulators; the state's two parts go to shared memory once per block, for the read-out of the next one.
+// columns; each of its eight warps takes 16 of the block's tokens and half of the columns for the outputs, and every
+// eighth tile of 16 rows and half of the columns of the state, which it keeps as accumulators; the state's two parts go
+// to shared memory once per block, for the read-out of the next one.
 #pragma once
 
 namespace rl {
@@ -18,8 +19,9 @@ constexpr int kSL = 64;                        // tokens of a block
 constexpr int kSV = 64;                        // value columns of a CTA
 constexpr int kSN = kD + 8;                    // elements of a row of queries or keys in shared memory (spreads the banks)
 constexpr int kSX = kSV + 8;                   // elements of a row of values; of a row of the state
-constexpr int kSTiles = (kD / 16 + 3) / 4;     // 16-row tiles of the state per warp
-constexpr int kSsdThreads = 128;
+constexpr int kSH = kSV / 2;                   // columns of a warp
+constexpr int kSTiles = (kD / 16 * 2 + 7) / 8; // tiles of the state (16 rows, half of the columns) per warp
+constexpr int kSsdThreads = 256;
 
 __device__ __forceinline__ void ssd_mma(float* d, const uint32_t* a, uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -82,6 +84,7 @@ ssd_kernel(const LinArgs<bf16> a) {
   const int qk_head = head / (a.heads / a.qk_heads);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, gid = lane >> 2, tig = lane & 3;
   const int col0 = blockIdx.x * kSV, cols = min(kSV, a.dv - col0);            // (a multiple of 16)
+  const int rows0 = (warp & 3) * 16, half0 = (warp >> 2) * kSH;               // the warp's tokens and columns for the outputs
   const SsdLayout lay = ssd_layout(MODE != 1);
   bf16* qs = reinterpret_cast<bf16*>(sm + lay.q);
   bf16* ks = reinterpret_cast<bf16*>(sm + lay.k);
@@ -139,10 +142,11 @@ ssd_kernel(const LinArgs<bf16> a) {
   float* slot_state = a.state + static_cast<size_t>(a.state_slot[seq]) * a.slot_stride + head * plane;
   float* chunk_state = MODE == 0 ? nullptr
       : a.chunk_state + ((static_cast<size_t>(seq) * a.max_chunks + c) * a.heads + head) * plane;
-  // S[i][j]: rows (4 i + warp) * 16 + gid and + 8, columns j * 8 + 2 tig and + 1
-  float S[kSTiles][kSV / 8][4];
-  auto row_of = [&](int i) { return (4 * i + warp) * 16 + gid; };
-  auto tile_in = [&](int i) { return (4 * i + warp) * 16 < kD; };
+  // S[i][j]: tile 8 i + warp (two tiles to 16 rows), rows gid and + 8 of it, columns j * 8 + 2 tig and + 1 of its half
+  float S[kSTiles][kSH / 8][4];
+  const int state_half = (warp & 1) * kSH;         // (8 i + warp and warp have the same half)
+  auto row_of = [&](int i) { return (8 * i + warp) / 2 * 16 + gid; };
+  auto tile_in = [&](int i) { return (8 * i + warp) / 2 * 16 < kD; };
   {
     const float* from = slot_state;
     if (MODE == 3 && c > 0) from = chunk_state - static_cast<size_t>(a.heads) * plane;
@@ -153,9 +157,9 @@ ssd_kernel(const LinArgs<bf16> a) {
 #pragma unroll
     for (int i = 0; i < kSTiles; ++i)
 #pragma unroll
-      for (int j = 0; j < kSV / 8; ++j) {
-        const bool in = MODE != 1 && tile_in(i) && j * 8 < cols;
-        const float* p = from + static_cast<size_t>(row_of(i)) * a.dv + col0 + j * 8 + 2 * tig;
+      for (int j = 0; j < kSH / 8; ++j) {
+        const bool in = MODE != 1 && tile_in(i) && state_half + j * 8 < cols;
+        const float* p = from + static_cast<size_t>(row_of(i)) * a.dv + col0 + state_half + j * 8 + 2 * tig;
         float2 x = make_float2(0.f, 0.f), y = x;
         if (in) {
           if (a.quads_ok) {
@@ -191,9 +195,9 @@ ssd_kernel(const LinArgs<bf16> a) {
       for (int i = 0; i < kSTiles; ++i)
         if (tile_in(i)) {
 #pragma unroll
-          for (int j = 0; j < kSV / 8; ++j)
-            if (j * 8 < cols) {
-              const int at = row_of(i) * kSX + j * 8 + 2 * tig;
+          for (int j = 0; j < kSH / 8; ++j)
+            if (state_half + j * 8 < cols) {
+              const int at = row_of(i) * kSX + state_half + j * 8 + 2 * tig;
               uint32_t hi, lo;
               ssd_split(S[i][j][0], S[i][j][1], hi, lo);
               *reinterpret_cast<uint32_t*>(sh + at) = hi;
@@ -208,12 +212,12 @@ ssd_kernel(const LinArgs<bf16> a) {
     __syncthreads();
     const float half = total[0], end = half + total[1];
     auto log_at = [&](int t) { return logs[t] + (t >= 32 ? half : 0.f); };
-    // ---- the values times d_s e^(l_end - l_s): two threads to a token
+    // ---- the values times d_s e^(l_end - l_s): four threads to a token
     {
-      const int s = threadIdx.x >> 1, c0 = (threadIdx.x & 1) * (kSV / 2);
+      const int s = threadIdx.x >> 2, c0 = (threadIdx.x & 3) * (kSV / 4);
       const float w = steps[s] * ssd_exp2(end - log_at(s));
 #pragma unroll
-      for (int e = 0; e < kSV / 2; e += 8)
+      for (int e = 0; e < kSV / 4; e += 8)
         if (c0 + e < cols) {
           float v[8];
           load16(vs + s * kSX + c0 + e, v);
@@ -224,30 +228,30 @@ ssd_kernel(const LinArgs<bf16> a) {
           *reinterpret_cast<uint4*>(wl + s * kSX + c0 + e) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
         }
     }
-    if (MODE != 1 && warp * 16 < nt) {
-      const int r0 = warp * 16 + gid, r1 = r0 + 8;               // this thread's two tokens of the block
-      float o[kSV / 8][4], g[kSL / 8][4];
+    if (MODE != 1 && rows0 < nt && half0 < cols) {
+      const int r0 = rows0 + gid, r1 = r0 + 8;                   // this thread's two tokens of the block
+      float o[kSH / 8][4], g[kSL / 8][4];
 #pragma unroll
-      for (int j = 0; j < kSV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+      for (int j = 0; j < kSH / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
 #pragma unroll
       for (int j = 0; j < kSL / 8; ++j) g[j][0] = g[j][1] = g[j][2] = g[j][3] = 0.f;
 #pragma unroll 4
       for (int kk = 0; kk < kD / 16; ++kk) {
         uint32_t qa[4];
-        ssd_ldmatrix<false>(qa, qs + (warp * 16 + (lane & 15)) * kSN + kk * 16 + (lane >> 4) * 8);
+        ssd_ldmatrix<false>(qa, qs + (rows0 + (lane & 15)) * kSN + kk * 16 + (lane >> 4) * 8);
 #pragma unroll
         for (int j = 0; j < kSL / 8; j += 2)
-          if (j * 8 < warp * 16 + 16) {                          // (tokens s <= t only)
+          if (j * 8 < rows0 + 16) {                              // (tokens s <= t only)
             uint32_t b[4];
             ssd_ldmatrix<false>(b, ks + (j * 8 + (lane & 7) + (lane >> 4) * 8) * kSN + kk * 16 + ((lane >> 3) & 1) * 8);
             ssd_mma(g[j], qa, b[0], b[1]);
             ssd_mma(g[j + 1], qa, b[2], b[3]);
           }
 #pragma unroll
-        for (int j = 0; j < kSV / 8; j += 2)
-          if (j * 8 < cols) {
+        for (int j = 0; j < kSH / 8; j += 2)
+          if (half0 + j * 8 < cols) {
             uint32_t b[4];
-            const int at = (kk * 16 + (lane & 15)) * kSX + j * 8 + (lane >> 4) * 8;
+            const int at = (kk * 16 + (lane & 15)) * kSX + half0 + j * 8 + (lane >> 4) * 8;
             ssd_ldmatrix<true>(b, sl + at);
             ssd_mma(o[j], qa, b[0], b[1]);
             ssd_mma(o[j + 1], qa, b[2], b[3]);
@@ -259,7 +263,7 @@ ssd_kernel(const LinArgs<bf16> a) {
       const float l0 = log_at(r0), l1 = log_at(r1);
       const float e0 = ssd_exp2(l0), e1 = ssd_exp2(l1);
 #pragma unroll
-      for (int j = 0; j < kSV / 8; ++j) {
+      for (int j = 0; j < kSH / 8; ++j) {
         o[j][0] *= e0;
         o[j][1] *= e0;
         o[j][2] *= e1;
@@ -267,7 +271,7 @@ ssd_kernel(const LinArgs<bf16> a) {
       }
 #pragma unroll
       for (int kk = 0; kk < kSL / 16; ++kk) {
-        if (kk > warp) continue;
+        if (kk * 16 > rows0) continue;
         uint32_t mh[4], ml[4];
 #pragma unroll
         for (int h = 0; h < 2; ++h) {                            // the 16 columns' two tiles
@@ -282,21 +286,21 @@ ssd_kernel(const LinArgs<bf16> a) {
           ssd_split(m(q[2], r1, l1, s, x0, d0), m(q[3], r1, l1, s + 1, x1, d1), mh[2 * h + 1], ml[2 * h + 1]);
         }
 #pragma unroll
-        for (int j = 0; j < kSV / 8; j += 2)
-          if (j * 8 < cols) {
+        for (int j = 0; j < kSH / 8; j += 2)
+          if (half0 + j * 8 < cols) {
             uint32_t b[4];
-            ssd_ldmatrix<true>(b, vs + (kk * 16 + (lane & 15)) * kSX + j * 8 + (lane >> 4) * 8);
+            ssd_ldmatrix<true>(b, vs + (kk * 16 + (lane & 15)) * kSX + half0 + j * 8 + (lane >> 4) * 8);
             ssd_mma(o[j], ml, b[0], b[1]);
             ssd_mma(o[j + 1], ml, b[2], b[3]);
             ssd_mma(o[j], mh, b[0], b[1]);
             ssd_mma(o[j + 1], mh, b[2], b[3]);
           }
       }
-      float* out = a.out + static_cast<size_t>(tb) * (a.heads * a.dv) + head * a.dv + col0 + 2 * tig;
+      float* out = a.out + static_cast<size_t>(tb) * (a.heads * a.dv) + head * a.dv + col0 + half0 + 2 * tig;
       const size_t row = static_cast<size_t>(a.heads) * a.dv;
 #pragma unroll
-      for (int j = 0; j < kSV / 8; ++j)
-        if (j * 8 < cols) {
+      for (int j = 0; j < kSH / 8; ++j)
+        if (half0 + j * 8 < cols) {
           if (r0 < nt) *reinterpret_cast<float2*>(out + r0 * row + j * 8) = make_float2(o[j][0], o[j][1]);
           if (r1 < nt) *reinterpret_cast<float2*>(out + r1 * row + j * 8) = make_float2(o[j][2], o[j][3]);
         }
@@ -308,7 +312,7 @@ ssd_kernel(const LinArgs<bf16> a) {
       for (int i = 0; i < kSTiles; ++i)
         if (tile_in(i)) {
 #pragma unroll
-          for (int j = 0; j < kSV / 8; ++j) {
+          for (int j = 0; j < kSH / 8; ++j) {
             S[i][j][0] *= e;
             S[i][j][1] *= e;
             S[i][j][2] *= e;
@@ -322,12 +326,12 @@ ssd_kernel(const LinArgs<bf16> a) {
 #pragma unroll
         for (int i = 0; i < kSTiles; ++i)
           if (tile_in(i))
-            ssd_ldmatrix<true>(ka[i], ks + (kk * 16 + (lane & 7) + (lane >> 4) * 8) * kSN + (4 * i + warp) * 16 + ((lane >> 3) & 1) * 8);
+            ssd_ldmatrix<true>(ka[i], ks + (kk * 16 + (lane & 7) + (lane >> 4) * 8) * kSN + (8 * i + warp) / 2 * 16 + ((lane >> 3) & 1) * 8);
 #pragma unroll
-        for (int j = 0; j < kSV / 8; j += 2)
-          if (j * 8 < cols) {
+        for (int j = 0; j < kSH / 8; j += 2)
+          if (state_half + j * 8 < cols) {
             uint32_t bh[4], bl[4];
-            const int at = (kk * 16 + (lane & 15)) * kSX + j * 8 + (lane >> 4) * 8;
+            const int at = (kk * 16 + (lane & 15)) * kSX + state_half + j * 8 + (lane >> 4) * 8;
             ssd_ldmatrix<true>(bl, wl + at);
             ssd_ldmatrix<true>(bh, wh + at);
 #pragma unroll
@@ -353,9 +357,9 @@ ssd_kernel(const LinArgs<bf16> a) {
   for (int i = 0; i < kSTiles; ++i)
     if (tile_in(i)) {
 #pragma unroll
-      for (int j = 0; j < kSV / 8; ++j)
-        if (j * 8 < cols) {
-          float* p = to + static_cast<size_t>(row_of(i)) * a.dv + col0 + j * 8 + 2 * tig;
+      for (int j = 0; j < kSH / 8; ++j)
+        if (state_half + j * 8 < cols) {
+          float* p = to + static_cast<size_t>(row_of(i)) * a.dv + col0 + state_half + j * 8 + 2 * tig;
           float* p8 = p + 8 * static_cast<size_t>(a.dv);
           if (a.quads_ok) {
             *reinterpret_cast<float2*>(p) = make_float2(S[i][j][0], S[i][j][1]);

@@ -201,9 +201,8 @@ struct RowMix {
 };
 
 template <typename TA, int NV, bool VEC>
-__global__ void sum_norm_kernel(float* __restrict__ residual, const TA* __restrict__ delta, int ld_delta,
-                                const float* __restrict__ w, const float* __restrict__ scale, float alpha, float eps,
-                                TA* __restrict__ out, int ld_out, int hidden, const RowMix<TA> mix) {
+__global__ void sum_norm_kernel(float* residual, const TA* delta, int ld_delta, const float* __restrict__ w,
+                                const float* __restrict__ scale, float alpha, float eps, TA* __restrict__ out, int ld_out, int hidden, const RowMix<TA> mix) {
   __shared__ float scratch[32];
   const int r = blockIdx.x;
   float* res = residual + static_cast<size_t>(r) * hidden;
@@ -439,7 +438,7 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ o, const TA* __re
 // o is the float32 output of a recurrence [T, groups * size].  A part lives in registers, NV pieces of four neighbouring
 // entries per thread (VEC: parts and rows start on a piece's boundary; else entry by entry).
 template <typename TA, typename TW, int NV, bool VEC>
-__global__ void group_gated_norm_kernel(const float* __restrict__ o, const TA* __restrict__ gate, int ld_gate,
+__global__ void group_gated_norm_kernel(const float* o, const TA* gate, int ld_gate,
                                         const TW* __restrict__ w, TA* __restrict__ out, int ld_out, int size, float eps) {
   __shared__ float scratch[32];
   const size_t r = blockIdx.x;

@@ -229,6 +229,76 @@ __global__ void short_conv_kernel(const ConvArgs a, const TA* __restrict__ x, co
   }
 }
 
+// The same for steps of many tokens: a thread takes four neighbouring channels of kWideTile tokens.  Where these and
+// the taps - 1 tokens before them belong to one sequence (the whole CTA sees the same tokens), all their rows are asked
+// for at once and the window is in registers; else every output gathers its own inputs.  Needs channels, columns and
+// row lengths that are multiples of four, aligned rows.
+constexpr int kWideTile = 8, kWideTaps = 4;
+
+template <typename TA, typename TW, int TAPS>
+__global__ void __launch_bounds__(128)
+short_conv_wide_kernel(const ConvArgs a, const TA* x, const TW* __restrict__ w, TA* __restrict__ y) {
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  const bool in = c < a.channels;
+  constexpr int keep = TAPS - 1;
+  float wt[4][TAPS], bias[4] = {0.f, 0.f, 0.f, 0.f}, out_bias[4] = {0.f, 0.f, 0.f, 0.f};
+  if (in) {                              // (constants come from no earlier kernel of the step)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) wt[e][j] = to_float(w[static_cast<size_t>(c + e) * TAPS + j]);
+      if (a.bias != nullptr) bias[e] = a.bias[c + e];
+      if (a.out_bias != nullptr) out_bias[e] = a.out_bias[c + e];
+    }
+  }
+  pdl_launch();
+  pdl_wait();
+  if (!in) return;
+  const int t_begin = blockIdx.y * kWideTile, t_end = min(t_begin + kWideTile, a.tokens);
+  const bool one = t_begin >= keep && a.seq_of_token[t_begin - keep] == a.seq_of_token[t_end - 1];
+  auto finish = [&](int t, float (&acc)[4]) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      acc[e] += out_bias[e];
+      if (a.act == ACT_SILU) acc[e] = sizeof(TA) == 2 ? __fdividef(acc[e], 1.f + __expf(-acc[e])) : acc[e] / (1.f + expf(-acc[e]));
+    }
+    store4(y + static_cast<size_t>(t) * a.ld_y + a.col_y + c, acc);
+  };
+  if (one) {
+    float u[keep + kWideTile][4];
+#pragma unroll
+    for (int i = 0; i < keep + kWideTile; ++i) {
+      const int t = min(t_begin - keep + i, t_end - 1);
+      load4(x + static_cast<size_t>(t) * a.ld_x + a.col_x + c, u[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < keep + kWideTile; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) u[i][e] += bias[e];
+#pragma unroll
+    for (int i = 0; i < kWideTile; ++i) {
+      if (t_begin + i >= t_end) break;
+      float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc[e] = fmaf(wt[e][j], u[i + j][e], acc[e]);
+      finish(t_begin + i, acc);
+    }
+    return;
+  }
+  for (int t = t_begin; t < t_end; ++t) {
+    const int seq = a.seq_of_token[t], first = conv_first(a.seq_of_token, t, seq, keep);
+    const float* st = a.state + static_cast<size_t>(a.state_slot[seq]) * a.slot_stride;
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[e] = fmaf(wt[e][j], conv_input(a, x, st, t - keep + j, first, c + e, bias[e]), acc[e]);
+    finish(t, acc);
+  }
+}
+
 // Moves the slots on: the thread that meets a sequence's last token of the step gathers the channel's last
 // taps - 1 inputs (from the step, or from the old slot where the portion is shorter) and writes them back.
 template <typename TA>
@@ -398,9 +468,22 @@ int rl_short_conv(int act_dtype, const void* x, int ld_x, int col_x, const void*
   a.tile = static_cast<long long>(channels) * tokens >= (1ll << 20) ? kConvTile : 1;
   const dim3 grid((channels + th - 1) / th, (tokens + a.tile - 1) / a.tile);
   const dim3 grid_state((channels + th - 1) / th, (tokens + kStateTile - 1) / kStateTile);
+  // (a step in which every sequence has one token moves the slots on in the first kernel)
+  const size_t piece = act_dtype == RL_F32 ? 16 : 8;
+  const bool wide = a.tile > 1 && !a.own_state && taps <= kWideTaps && channels % 4 == 0 && ld_x % 4 == 0 && col_x % 4 == 0 &&
+                    ld_y % 4 == 0 && col_y % 4 == 0 && reinterpret_cast<uintptr_t>(x) % piece == 0 &&
+                    reinterpret_cast<uintptr_t>(y) % piece == 0;
+  const dim3 grid_wide((channels / 4 + th - 1) / th, (tokens + kWideTile - 1) / kWideTile);
+#define RL_WIDE(TA, TW, TAPS)                                                                                  \
+  launch_kernel(short_conv_wide_kernel<TA, TW, TAPS>, grid_wide, dim3(th), 0, stream, a, static_cast<const TA*>(x), \
+                static_cast<const TW*>(w), static_cast<TA*>(y))
 #define RL_CASE(TA, TW)                                                                                        \
   do {                                                                                                         \
-    launch_kernel(short_conv_kernel<TA, TW>, grid, dim3(th), 0, stream, a, static_cast<const TA*>(x),          \
+    if (wide && taps == 1) RL_WIDE(TA, TW, 1);                                                                 \
+    else if (wide && taps == 2) RL_WIDE(TA, TW, 2);                                                            \
+    else if (wide && taps == 3) RL_WIDE(TA, TW, 3);                                                            \
+    else if (wide) RL_WIDE(TA, TW, 4);                                                                         \
+    else launch_kernel(short_conv_kernel<TA, TW>, grid, dim3(th), 0, stream, a, static_cast<const TA*>(x),          \
                   static_cast<const TW*>(w), static_cast<TA*>(y));                                             \
     if (taps > 1 && !single) launch_kernel(short_conv_state_kernel<TA>, grid_state, dim3(th), 0, stream, a, static_cast<const TA*>(x)); \
   } while (0)
@@ -408,6 +491,7 @@ int rl_short_conv(int act_dtype, const void* x, int ld_x, int col_x, const void*
   else if (w_dtype == RL_F32) RL_CASE(bf16, float);
   else RL_CASE(bf16, bf16);
 #undef RL_CASE
+#undef RL_WIDE
   RL_LAUNCH_END();
 }
 

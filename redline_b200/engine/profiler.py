@@ -134,23 +134,28 @@ def linear_work(rows: int, w: torch.Tensor, act_elem: int, out_elem: int) -> tup
     return (float(w.numel() * w.element_size() + rows * k * act_elem + rows * n * out_elem), 2.0 * rows * n * k)
 
 
-def attention_work(host, num_heads: int, num_kv_heads: int, head_dim: int, window: int, elem: int) -> dict:
+def attention_work(host, num_heads: int, num_kv_heads: int, head_dim: int, window: int, elem: int, chunk: int = 0) -> dict:
     """What the attention of a step has to read and compute, from the step's host-side description
     (``host.q_len`` / ``host.start_pos`` per sequence): {"decode": (bytes, flops), "prefill": (bytes, flops)}.
     A single token reads the keys and values of its context once per kv head; a portion of n tokens
-    after p earlier ones reads its p + n keys and values once and computes over the causal part."""
+    after p earlier ones reads its p + n keys and values once and computes over the causal part.  ``window`` > 0 or
+    ``chunk`` > 0: only the last so many keys, or those of the token's chunk of so many positions, are seen."""
+
+    def seen(pos: int) -> int:
+        return min(pos + 1, window) if window > 0 else (pos % chunk + 1 if chunk > 0 else pos + 1)
+
     dec_b = dec_f = pre_b = pre_f = 0.0
     kv_row = 2.0 * num_kv_heads * head_dim * elem            # K and V of one token
     q_row = 2.0 * num_heads * head_dim * elem                # q read, output written
     for n, p in zip(host.q_len, host.start_pos):
         if n == 1:
-            keys = p + 1 if window <= 0 else min(p + 1, window)
+            keys = seen(p)
             dec_b += keys * kv_row + q_row
             dec_f += 4.0 * num_heads * head_dim * keys
         elif n > 1:
             pairs = n * p + n * (n + 1) / 2.0                # (query, key) pairs of the causal part
-            if window > 0:
-                pairs = sum(min(p + i + 1, window) for i in range(n))
-            pre_b += (p + n) * kv_row + n * q_row
+            if window > 0 or chunk > 0:
+                pairs = sum(seen(p + i) for i in range(n))
+            pre_b += (n + seen(p) - 1) * kv_row + n * q_row
             pre_f += 4.0 * num_heads * head_dim * pairs
     return {"decode": (dec_b, dec_f), "prefill": (pre_b, pre_f)}

@@ -1124,21 +1124,25 @@ def _ssm(state: int) -> ctypes.CDLL:
     return _lib(f"state_space_d{state}", "linear_attention.cu", {"RL_LIN_DIM": state, "RL_LIN_TOKEN": 1})
 
 
-SSD_CTAS = 296                     # CTAs that fill the machine: sequences are cut into chunks until there are about so many
-SSD_MIN_CHUNK = 256
+SSD_CTAS = 296                     # CTAs of the block form that run side by side (two on each of 148 SMs)
 
 
-def state_space_chunks(longest: int, sequences: int, heads: int, vdim: int, blocks: bool) -> Tuple[int, int]:
-    """(chunk length, most chunks) for a step of ``sequences`` sequences of at most ``longest`` tokens; (0, 1) when
-    every sequence is run as one chain.  ``blocks``: for the form that runs blocks of 64 tokens on the tensor cores."""
+def state_space_chunks(longest: int, tokens: int, heads: int, vdim: int, blocks: bool) -> Tuple[int, int]:
+    """(chunk length, most chunks) for a step of ``tokens`` tokens whose longest sequence brings ``longest``; (0, 1)
+    when every sequence is run as one chain.  ``blocks``: for the form that runs blocks of 64 tokens on the tensor cores."""
     if not blocks:
         return linear_attention_chunks(longest)
-    ctas = heads * sequences * ((vdim + 63) // 64)
-    chunks = min(16, (SSD_CTAS + ctas - 1) // ctas, longest // SSD_MIN_CHUNK)
-    if chunks <= 1:
-        return 0, 1
-    chunk = ((longest + chunks - 1) // chunks + 63) // 64 * 64
-    return chunk, (longest + chunk - 1) // chunk
+    ctas = heads * max((tokens + longest - 1) // longest, 1) * ((vdim + 63) // 64)       # (short sequences hardly count)
+    total = (longest + 63) // 64
+    # time in blocks of a CTA: waves of CTAs times their blocks; chunks' own sums cost half as much again, their states some more
+    best = None
+    for chunks in range(1, min(16, total // 2) + 1):
+        per = (total + chunks - 1) // chunks
+        chunks = (total + per - 1) // per
+        cost = (ctas * chunks + SSD_CTAS - 1) // SSD_CTAS * (per if chunks == 1 else 1.5 * per + 1.5)
+        if best is None or cost < best[0]:
+            best = (cost, per * 64, chunks)
+    return (0, 1) if best is None or best[2] == 1 else best[1:]
 
 
 def state_space(q: torch.Tensor, k: torch.Tensor, qk_heads: int, v: torch.Tensor, steps: torch.Tensor,

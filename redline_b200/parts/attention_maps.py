@@ -344,7 +344,7 @@ class MapsAttention(Mixer):
         from ..engine.profiler import attention_work
         p = self.params
         elem = 2 if self.rt.dtype == torch.bfloat16 else 4
-        window = p.window + p.keep_first if p.window > 0 else p.chunk      # (of a chunk the mean token sees half)
+        window = p.window + p.keep_first if p.window > 0 else 0
         nbytes, flops = attention_work(ctx.host, p.num_heads * p.maps, p.num_kv_heads * p.maps, (p.dim + p.vdim) // 2,
-                                       window, elem)[which]
+                                       window, elem, p.chunk)[which]
         ctx.profiler.mark(op, nbytes, flops)

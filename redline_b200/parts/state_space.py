@@ -103,7 +103,7 @@ class StateSpace(Mixer):
         # (how a step is cut depends on its shape alone: single-token steps and full portions replay as graphs)
         longest = 1 if ctx.num_tiles == 0 else max(ctx.host.q_len)
         blocks = rt.dtype == torch.bfloat16 and p.state % 16 == 0 and p.vdim % 16 == 0
-        chunk, max_chunks = kernels.state_space_chunks(longest, ctx.S, H, p.vdim, blocks)
+        chunk, max_chunks = kernels.state_space_chunks(longest, T, H, p.vdim, blocks)
         work = {}
         if max_chunks > 1:
             work = dict(chunk_state=ws.get("lin.chunks", (ctx.S * max_chunks * H * p.state * p.vdim,), torch.float32),
