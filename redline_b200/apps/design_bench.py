@@ -38,8 +38,8 @@ feed-forwards are dense and as wide as Lakatar's chosen and shared experts toget
 recurrence (the delta rule with a decay per key channel, as many state entries per head as Lakatar's time mixing
 has in two heads), both at the same width.
 
-The Vogolix model has five layers, all with a gated dense feed-forward: chunked attention with a sink, attention over
-its keys and values, two state-space layers, windowed attention over a cached latent.  Beside it stand Pufevik, the
+The Vogolix model has four layers, all with a gated dense feed-forward: chunked attention with a sink, a state-space
+layer, attention over the first layer's keys and values, windowed attention over a cached latent.  Beside it stand Pufevik, the
 closest architecture the package has (attention with a sink, norms over the whole projection and neighbouring pairs
 rotated, through the same kernels, over a window as long as the chunk; a gated dense feed-forward of the same width),
 and Lakatar for the latent attention (the same rows) and for its recurrences (retention: as many state entries as half
@@ -199,8 +199,8 @@ def vogolix_config(s: Dict[str, int]) -> Dict[str, Any]:
            "conv": s["taps"]}
     dense = {"kind": "dense", "ff": s["ff"]}
     return {"architecture": "Vogolix", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-6}, "logit_scale": 0.5,
-            "layers": [{"type": "attention", "mixer": att, "mlp": dense}, {"type": "attention", "mixer": dict(att, kv_from=0), "mlp": dense},
-                       {"type": "mamba2", "mixer": ssm, "mlp": dense}, {"type": "mamba2", "mixer": ssm, "mlp": dense},
+            "layers": [{"type": "attention", "mixer": att, "mlp": dense}, {"type": "mamba2", "mixer": ssm, "mlp": dense},
+                       {"type": "attention", "mixer": dict(att, kv_from=0), "mlp": dense},
                        {"type": "latent_attention", "mixer": latent, "mlp": dense}]}
 
 
@@ -318,7 +318,7 @@ def compare(design: str, sizes: List[str], steps: int, warmup: int, batch: int, 
     with tempfile.TemporaryDirectory() as tmp:
         for name in sizes:
             s = table[name]
-            entry: Dict[str, Any] = {"shape": dict(s, layers=len(design_config(s)["layers"]), window=WINDOW)}
+            entry: Dict[str, Any] = {"shape": dict(s, layers=4, window=WINDOW)}
             if design == "kapitar":
                 entry["shape"]["keep_first"] = KEEP_FIRST
             for arch, cfg in [(design, design_config(s))] + [(b, conf(sizes_of[name])) for b, sizes_of, conf in beside]:

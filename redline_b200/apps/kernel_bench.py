@@ -6,7 +6,7 @@ package, if present).
     python -m redline_b200.apps.kernel_bench skinny --rows 8 --n 3072 --k 2048 [--norm] [--epilogue swiglu]
     python -m redline_b200.apps.kernel_bench attn_prefill --tokens 2048
     python -m redline_b200.apps.kernel_bench gemm_tc --rows 2048 --n 8192 --k 2048 --epilogue swiglu [--library]
-    python -m redline_b200.apps.kernel_bench head_linear --tokens 2048 --heads 16 --n 192 --k 64 [--impl 1]
+    python -m redline_b200.apps.kernel_bench head_linear --tokens 2048 --heads 16 --n 192 --k 64 [--impl 1] [--gate]
     python -m redline_b200.apps.kernel_bench latent_attn --tokens 2048 --heads 16 --rank 192 --rot 32 [--impl 1]
     python -m redline_b200.apps.kernel_bench recurrence --tokens 2048 --heads 32 --head-dim 64 --vdim 64 [--channel] [--seqs 1]
     python -m redline_b200.apps.kernel_bench state_space --tokens 2048 --heads 64 --qk-heads 1 --head-dim 128 --vdim 64 [--seqs 1]
@@ -235,14 +235,16 @@ def bench_head_linear(args) -> None:
     xs = [torch.randn(T, H * K, device=dev).to(torch.bfloat16) for _ in range(copies)]
     ys = [torch.empty(T, H * N, device=dev, dtype=torch.bfloat16) for _ in range(copies)]
     w = (torch.randn(H, N, K, device=dev) / math.sqrt(K)).to(torch.bfloat16)
+    gates = [torch.randn(T, H * N, device=dev).to(torch.bfloat16) for _ in range(copies if args.gate else 0)]
 
     def fn(i):
-        kernels.head_linear(xs[i % copies], 0, K, w, ys[i % copies], 0, N, impl=args.impl)
+        kernels.head_linear(xs[i % copies], 0, K, w, ys[i % copies], 0, N, impl=args.impl,
+                            gate=gates[i % copies] if args.gate else None)
 
     us = graph_time_us(fn, copies, use_graph=not args.no_graph)
-    nbytes, flops = T * H * (N + K) * 2.0 + w.numel() * 2.0, 2.0 * T * H * N * K
+    nbytes, flops = T * H * ((2 if args.gate else 1) * N + K) * 2.0 + w.numel() * 2.0, 2.0 * T * H * N * K
     pk = peaks()
-    print(json.dumps({"kernel": "head_linear", "impl": args.impl, "tokens": T, "heads": H, "n": N, "k": K, "us": round(us, 2),
+    print(json.dumps({"kernel": "head_linear", "gate": bool(args.gate), "impl": args.impl, "tokens": T, "heads": H, "n": N, "k": K, "us": round(us, 2),
                       "GB/s": round(nbytes / us / 1e3, 1), "TFLOP/s": round(flops / us / 1e6, 1),
                       "frac_of_measured_hbm": round(nbytes / us / 1e3 / pk["hbm_gbs"], 3),
                       "frac_of_measured_bf16": round(flops / us / 1e6 / pk["bf16_tflops"], 4), "copies": copies}))
@@ -381,6 +383,7 @@ def main() -> int:
         if name in ("head_linear", "latent_attn"):
             p.add_argument("--tokens", type=int, default=2048)
             p.add_argument("--impl", type=int, default=0, help="0 auto (tensor cores where they apply), 1 CUDA cores")
+            p.add_argument("--gate", action="store_true", help="head_linear: outputs times the sigmoid of a gate each")
             p.add_argument("--n", type=int, default=192, help="head_linear: outputs of a head")
             p.add_argument("--k", type=int, default=64, help="head_linear: inputs of a head")
             p.add_argument("--rank", type=int, default=192, help="latent_attn: size of the cached latent")

@@ -221,7 +221,7 @@ __device__ __forceinline__ void hl_mma(float* d, const uint32_t* a, uint32_t b0,
 
 constexpr int kHmRows = 64, kHmCols = 64;
 
-template <bool TURN>
+template <bool TURN, bool GATE>
 __global__ void __launch_bounds__(128)
 head_linear_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, bf16* __restrict__ y,
                        const HeadLinearArgs a) {
@@ -239,6 +239,17 @@ head_linear_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, b
   const bf16* x0 = x + static_cast<size_t>(ok0 ? r0 : t0) * a.x_ld + a.x_col + h * a.x_head + tig * 2;
   const bf16* x1 = x + static_cast<size_t>(ok1 ? r1 : t0) * a.x_ld + a.x_col + h * a.x_head + tig * 2;
   const bf16* wh = w + static_cast<size_t>(h) * a.n * a.k;
+  // (the gates are asked for ahead of the product; their pairs start on 4-byte boundaries as y's do)
+  uint32_t gates[GATE ? kHmCols / 8 : 1][2];
+  if (GATE) {
+    const bf16* g = static_cast<const bf16*>(a.gate) + h * a.n + j0 + tig * 2;
+#pragma unroll
+    for (int nt = 0; nt < kHmCols / 8; ++nt) {
+      const bool in = j0 + nt * 8 < a.n;
+      gates[GATE ? nt : 0][0] = in && ok0 ? *reinterpret_cast<const uint32_t*>(g + static_cast<size_t>(r0) * a.gate_ld + nt * 8) : 0u;
+      gates[GATE ? nt : 0][1] = in && ok1 ? *reinterpret_cast<const uint32_t*>(g + static_cast<size_t>(r1) * a.gate_ld + nt * 8) : 0u;
+    }
+  }
   float acc[kHmCols / 8][4];
 #pragma unroll
   for (int nt = 0; nt < kHmCols / 8; ++nt) acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f;
@@ -262,12 +273,19 @@ head_linear_mma_kernel(const bf16* __restrict__ x, const bf16* __restrict__ w, b
   for (int nt = 0; nt < kHmCols / 8; ++nt) {
     const int j = j0 + nt * 8 + tig * 2;
     if (j0 + nt * 8 >= a.n) continue;
+    if (GATE) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const uint32_t g = gates[GATE ? nt : 0][e >> 1];
+        acc[nt][e] = __fdividef(acc[nt][e], 1.f + __expf(-__uint_as_float(e & 1 ? g & 0xFFFF0000u : g << 16)));
+      }
+    }
     if (ok0)
       *reinterpret_cast<__nv_bfloat162*>(y + static_cast<size_t>(r0) * a.y_ld + a.y_col + h * a.y_head + j) =
-          __floats2bfloat162_rn(acc[nt][0] * gate_of<bf16>(a, r0, h, j), acc[nt][1] * gate_of<bf16>(a, r0, h, j + 1));
+          __floats2bfloat162_rn(acc[nt][0], acc[nt][1]);
     if (ok1)
       *reinterpret_cast<__nv_bfloat162*>(y + static_cast<size_t>(r1) * a.y_ld + a.y_col + h * a.y_head + j) =
-          __floats2bfloat162_rn(acc[nt][2] * gate_of<bf16>(a, r1, h, j), acc[nt][3] * gate_of<bf16>(a, r1, h, j + 1));
+          __floats2bfloat162_rn(acc[nt][2], acc[nt][3]);
   }
 }
 
@@ -299,6 +317,11 @@ head_linear_few_kernel(const bf16* x, const bf16* __restrict__ w, bf16* __restri
     for (int t = 0; t < kHfTokens; ++t) acc[f][t] = 0.f;
   const int nt = min(kHfTokens, a.tokens - t0);
   const bf16* xr = x + static_cast<size_t>(t0) * a.x_ld + a.x_col + h * a.x_head;
+  // lane 8 f + t writes output f of token t
+  static_assert(kHfCols * kHfTokens == 32, "a lane per output");
+  const int my_f = lane / kHfTokens, my_t = lane % kHfTokens;
+  const bool mine = my_t < nt && j0 + my_f < a.n;
+  float factor = 1.f, sum = 0.f;
   for (int c0 = 0; c0 < a.k; c0 += 256) {
     const int c = c0 + lane * 8;
     const bool in = c < a.k;
@@ -311,7 +334,10 @@ head_linear_few_kernel(const bf16* x, const bf16* __restrict__ w, bf16* __restri
         for (int i = 0; i < 8; ++i) wv[f][i] = 0.f;
       }
     }
-    if (c0 == 0) pdl_wait();                   // (the matrices come from no earlier kernel of the step)
+    if (c0 == 0) {                             // (the matrices come from no earlier kernel of the step)
+      pdl_wait();
+      if (mine) factor = gate_of<bf16>(a, t0 + my_t, h, j0 + my_f);
+    }
 #pragma unroll
     for (int t = 0; t < kHfTokens; ++t) {
       if (t < nt && in) {
@@ -329,10 +355,10 @@ head_linear_few_kernel(const bf16* x, const bf16* __restrict__ w, bf16* __restri
 #pragma unroll
     for (int t = 0; t < kHfTokens; ++t) {
       const float v = warp_sum(acc[f][t]);
-      if (lane == 0 && t < nt && j0 + f < a.n)
-        y[static_cast<size_t>(t0 + t) * a.y_ld + a.y_col + h * a.y_head + j0 + f] =
-            __float2bfloat16_rn(v * gate_of<bf16>(a, t0 + t, h, j0 + f));
+      if (f == my_f && t == my_t) sum = v;
     }
+  if (mine)
+    y[static_cast<size_t>(t0 + my_t) * a.y_ld + a.y_col + h * a.y_head + j0 + my_f] = __float2bfloat16_rn(sum * factor);
 }
 
 }  // namespace rl
@@ -382,6 +408,7 @@ int rl_head_linear(int act_dtype, int w_dtype, const void* x, int x_ld, int x_co
                    int rot_dims, int pairs, int turn_x, int turn_y, const float* cos_t, const float* sin_t, int max_pos,
                    const int32_t* positions, int* status, const void* gate, int gate_ld, cudaStream_t stream) {
   if (tokens <= 0 || heads <= 0 || n <= 0) return 0;
+  if (gate != nullptr && turn_dims > 0) return static_cast<int>(cudaErrorInvalidValue);
   HeadLinearArgs a;
   a.gate = gate;
   a.gate_ld = gate_ld;
@@ -398,7 +425,7 @@ int rl_head_linear(int act_dtype, int w_dtype, const void* x, int x_ld, int x_co
   a.turn = Turn{turn_dims, rot_dims, pairs, turn_x, turn_y, max_pos, cos_t, sin_t, positions, status};
   const bool even = ((x_ld | x_col | x_head | y_ld | y_col | y_head) & 1) == 0 &&
                     reinterpret_cast<uintptr_t>(x) % 4 == 0 && reinterpret_cast<uintptr_t>(y) % 4 == 0 &&
-                    reinterpret_cast<uintptr_t>(w) % 4 == 0;
+                    reinterpret_cast<uintptr_t>(w) % 4 == 0 && (gate == nullptr || (gate_ld % 2 == 0 && reinterpret_cast<uintptr_t>(gate) % 4 == 0));
   const int turning = turn_dims > 0 ? 1 : 0;
   const bool pieces = act_dtype == 1 && w_dtype == 1 && k % 8 == 0 && x_ld % 8 == 0 && x_col % 8 == 0 && x_head % 8 == 0 &&
                       reinterpret_cast<uintptr_t>(x) % 16 == 0 && reinterpret_cast<uintptr_t>(w) % 16 == 0;
@@ -410,8 +437,9 @@ int rl_head_linear(int act_dtype, int w_dtype, const void* x, int x_ld, int x_co
   }
   if (act_dtype == 1 && w_dtype == 1 && impl != 1 && k % 16 == 0 && n % 8 == 0 && even) {
     const dim3 grid((tokens + kHmRows - 1) / kHmRows, (n + kHmCols - 1) / kHmCols + turning, heads);
-    if (turning) launch_kernel(head_linear_mma_kernel<true>, grid, dim3(128), 0, stream, static_cast<const bf16*>(x), static_cast<const bf16*>(w), static_cast<bf16*>(y), a);
-    else launch_kernel(head_linear_mma_kernel<false>, grid, dim3(128), 0, stream, static_cast<const bf16*>(x), static_cast<const bf16*>(w), static_cast<bf16*>(y), a);
+    if (turning) launch_kernel(head_linear_mma_kernel<true, false>, grid, dim3(128), 0, stream, static_cast<const bf16*>(x), static_cast<const bf16*>(w), static_cast<bf16*>(y), a);
+    else if (gate != nullptr) launch_kernel(head_linear_mma_kernel<false, true>, grid, dim3(128), 0, stream, static_cast<const bf16*>(x), static_cast<const bf16*>(w), static_cast<bf16*>(y), a);
+    else launch_kernel(head_linear_mma_kernel<false, false>, grid, dim3(128), 0, stream, static_cast<const bf16*>(x), static_cast<const bf16*>(w), static_cast<bf16*>(y), a);
     RL_LAUNCH_END();
   }
   dim3 grid((tokens + kHlRows - 1) / kHlRows, (n + kHlCols - 1) / kHlCols + turning, heads);

@@ -1000,8 +1000,8 @@ def head_linear(x: torch.Tensor, x_col: int, x_head: int, w: torch.Tensor, y: to
         raise KernelError("head_linear: x and y have one type and contiguous rows; w contiguous [heads, n, k]")
     if x_col + (heads - 1) * x_head + k > x.shape[1] or y_col + (heads - 1) * y_head + n > y.shape[1]:
         raise KernelError("head_linear: the heads do not fit the rows")
-    if gate is not None and (gate.dtype != x.dtype or gate.stride(1) != 1 or gate.shape[1] != heads * n):
-        raise KernelError("head_linear: a gate has x's type and one entry per output")
+    if gate is not None and (gate.dtype != x.dtype or gate.stride(1) != 1 or gate.shape[1] != heads * n or turn is not None):
+        raise KernelError("head_linear: a gate has x's type and one entry per output, and goes without turned parts")
     dims = rot = tx = ty = max_pos = pairs = 0
     cos = sin = positions = status = None
     if turn is not None:

@@ -200,7 +200,7 @@ class LatentAttention(Mixer):
         heads_v = ws.get("latent.values", (rt.max_tokens, self.out_size), rt.dtype)[:T]
         kernels.head_linear(lat, 0, p.kv_rank, self.w_uv, heads_v, 0, p.vdim, tokens=T,
                             gate=proj[:, self.g_col:] if p.gate == "entry" else None)
-        op_mark(ctx, "v_up", nbytes=float(T * p.num_heads * (p.vdim + p.kv_rank) * elem + self.w_uv.numel() * elem),
+        op_mark(ctx, "v_up", nbytes=float(T * p.num_heads * ((2 if p.gate == "entry" else 1) * p.vdim + p.kv_rank) * elem + self.w_uv.numel() * elem),
                 flops=2.0 * T * p.num_heads * p.vdim * p.kv_rank)
         out = ws.get("mixer.out", (rt.max_tokens, p.hidden_size), rt.dtype)[:T]
         linear(heads_v, self.w_o, out)
